@@ -499,6 +499,10 @@ typedef struct tm_cache_sequence { /* LlamaCacheManager::Sequence, LlamaCacheMan
 } tm_cache_sequence;
 TM_API int tm_cache_manager_create(tm_cache_manager** out, size_t layer_num, size_t head_num, size_t size_per_head,
                                    size_t max_seq_len, size_t elem_bits, size_t max_entry_count, size_t chunk_size, int device);
+/* The same manager over slabs of `slab_bytes` whose layout is the model's own (tm_model_new_cache): k_cache is the start
+ * of a sequence's slab. */
+TM_API int tm_cache_manager_create_slabs(tm_cache_manager** out, size_t slab_bytes, size_t max_seq_len, size_t max_entry_count,
+                                         size_t chunk_size, int device);
 TM_API int tm_cache_manager_destroy(tm_cache_manager* m);
 TM_API int tm_cache_create(tm_cache_manager* m, uint64_t id, void* stream, tm_cache_sequence* out);
 TM_API int tm_cache_fetch(tm_cache_manager* m, uint64_t id, void* stream, tm_cache_sequence* out);
@@ -590,7 +594,122 @@ TM_API unsigned long long tm_llama_last_launches(const tm_llama* m);
 TM_API int tm_llama_check_status(tm_llama* m, void* stream, unsigned* word);
 
 /* ------------------------------------------------------------------------------------------
- * Persistent-batch scheduler over tm_cache_*, tm_llama_prefill, tm_llama_decode, tm_sample_topk / tm_sample_topp and
+ * Served models: one interface over the models of this library, which the scheduler, the command line
+ * (lmdeploy_b200/serve.py) and the trace replay (bin/trace_run) use.  tm_model_open chooses by what the folder holds:
+ *   config.json with "architecture": "Rumazen" and model.safetensors   the config-driven decoder (window attention with
+ *       pooled blocks, generalised delta rule, parallel layers); bf16, or everything in fp32
+ *   config.ini and weight files                                        a TurboMind W4A16 workspace (tm_llama)
+ * tm_model_close frees what tm_model_open and tm_decoder_create_random made; a tm_llama keeps its own functions, and
+ * tm_llama_as_model lends its tm_model.
+ */
+typedef struct tm_model tm_model;
+enum { TM_DTYPE_BF16 = 0, TM_DTYPE_F32 = 1 };
+typedef struct tm_model_options {
+    int dtype;              /* TM_DTYPE_BF16: matrix products, activations and cached rows in 16 bits; TM_DTYPE_F32: all fp32 */
+    int max_batch_size;     /* sequences of one decode step                                                                 */
+    int session_len;        /* most tokens of one sequence                                                                  */
+    int max_prefill_tokens; /* tokens that go through the layers together in a prefill; longer ones are cut (0: 4096)        */
+} tm_model_options;
+typedef struct tm_model_info {
+    int    vocab_size, max_batch_size, session_len;
+    int    can_rewind;      /* 0: a sequence cannot go back to an earlier length without running it again (recurrent state)  */
+    size_t slab_bytes;      /* cache and state of one sequence                                                              */
+} tm_model_info;
+TM_API int tm_model_open(tm_model** out, tm_handle* h, const char* dir, const tm_model_options* opt);
+TM_API int tm_model_close(tm_model* m);
+/* why the last tm_model_open / tm_decoder_create_random of this thread failed ("" when it did not) */
+TM_API const char* tm_model_last_error(void);
+/* names of the known architectures, separated by commas */
+TM_API int tm_model_architectures(char* names, size_t capacity);
+TM_API int tm_model_describe(const tm_model* m, tm_model_info* info);
+TM_API int tm_model_new_cache(const tm_model* m, size_t max_entry_count, size_t chunk_size, tm_cache_manager** out);
+TM_API tm_model* tm_llama_as_model(tm_llama* m);
+/* New tokens of some sequences through all layers, on top of history_lengths[b] tokens of each.  All arrays are host
+ * memory and are copied; k_cache / v_cache hold the device addresses of a tm_cache_sequence.  `want` (ascending indexes
+ * into the packed tokens) asks for logits: logits_out is device memory, float [want_count][vocab].  residual_out (device,
+ * may be NULL, for tests) takes the residual stream behind every layer, float [layers][tokens][width].  Asynchronous on
+ * `stream`.  The tm_llama model computes no logits here (its scheduler takes them from the decoder step). */
+typedef struct tm_model_prefill_state {
+    int          batch_size;
+    const int*   input_ids;        /* packed sequence after sequence                */
+    const int*   cu_seqlens;       /* [batch + 1] prefix sums of the token counts   */
+    const int*   history_lengths;  /* [batch] tokens taken in before                */
+    void* const* k_cache;          /* [batch]                                       */
+    void* const* v_cache;          /* [batch]                                       */
+    int          want_count;
+    const int*   want;
+    float*       logits_out;
+    float*       residual_out;
+} tm_model_prefill_state;
+TM_API int tm_model_prefill(tm_model* m, const tm_model_prefill_state* st, void* stream);
+/* n_steps decoder steps of one token per sequence, as tm_llama_decode (same state; hidden_out belongs to tm_llama) */
+
+TM_API int tm_model_decode(tm_model* m, const struct tm_llama_decode_state* st, int n_steps, int use_graph, void* stream);
+TM_API unsigned long long tm_model_last_launches(const tm_model* m);
+TM_API int tm_model_check_status(tm_model* m, void* stream, unsigned* word);
+/* Replay of given tokens: `count` tokens of sequence `id` behind those it has taken in (several through tm_model_prefill, a
+ * single one through the captured tm_model_decode), logits of the places `want` (ascending) to host memory, float
+ * [want_count][vocab].  Synchronous.  tm_replay_end gives the sequence's slab back. */
+typedef struct tm_replay tm_replay;
+TM_API int tm_replay_create(tm_replay** out, tm_model* model, size_t max_sequences);
+TM_API int tm_replay_destroy(tm_replay* r);
+TM_API int tm_replay_step(tm_replay* r, uint64_t id, const int* tokens, int count, const int* want, int want_count, float* logits);
+TM_API int tm_replay_end(tm_replay* r, uint64_t id);
+/* A config-driven decoder with random weights (seeded, on the device), for measurements: `config_json` is the text of a
+ * config.json; a delta-rule mixer then names the rank of its decay projection itself ("rank", default 16). */
+TM_API int tm_decoder_create_random(tm_model** out, tm_handle* h, const char* config_json, const tm_model_options* opt,
+                                    unsigned long long seed);
+
+/* The decoder's mechanisms as operators.  Sequences: `batch` spans, host arrays; span b holds the rows
+ * [sum of n before it, + n[b]) of proj and out, at positions history[b], history[b] + 1, ...; slabs[b] is the device
+ * memory its cache or state lives in, at the byte offsets below.  decode != 0 runs the one-token kernels (every n is 1).
+ * Element type of proj, out, caches and w2: `dtype`. */
+typedef struct tm_mixer_call {
+    void*        proj;
+    int          proj_ld;
+    void*        out;
+    int          out_ld;
+    int          batch;
+    const int*   history;
+    const int*   n;
+    void* const* slabs;
+    int          dtype;
+    int          decode;
+} tm_mixer_call;
+/* Softmax attention of `heads` query heads over `kv_heads` key / value heads: the first rot_dims dimensions of q and k
+ * rotate (interleaved pairs, angle position * inv_freq[i]); position i sees the tokens j with 0 <= i - j < window (0: all)
+ * and, as one more key and value each, the mean of every block of `pool` tokens (0: none) that ends at or before
+ * i - window; score = softcap * tanh(q.k * scale / softcap) (softcap 0: no cap); head outputs are multiplied by
+ * sigmoid(gate logit).  Position p is cached in row p % ring of [kv head][ring][dim or vdim]. */
+typedef struct tm_window_attention_params {
+    int          heads, kv_heads, dim, vdim, rot_dims;
+    const float* inv_freq; /* device */
+    float        scale, softcap;
+    int          window, pool, ring, pool_rows;
+    size_t       k_off, v_off, pooled_k_off, pooled_v_off;
+    int          q_col, k_col, v_col, g_col;
+} tm_window_attention_params;
+TM_API int tm_window_attention(tm_handle* h, const tm_window_attention_params* a, const tm_mixer_call* c, void* stream);
+/* Generalised delta rule, fp32 state float [head][dim][dim] (zero at history 0):
+ *   w = exp(-decay_scale * sigmoid(w2 . w1 + w0)), a = sigmoid(a + a_bias), u = k / sqrt(k.k + unit_eps)
+ *   S <- diag(w) S - (a u)(u^T S) + k v^T,   o = S^T r;   out = o / rms(o) * norm * sigmoid(g) per head */
+typedef struct tm_delta_rule_params {
+    int          heads, dim, rank;
+    const void*  w2; /* device [heads * dim][w2_ld] */
+    int          w2_ld;
+    const float *w0, *a_bias, *norm; /* device [heads * dim] */
+    float        norm_eps, unit_eps, decay_scale;
+    size_t       state_off;
+    int          r_col, k_col, v_col, a_col, g_col, w1_col;
+} tm_delta_rule_params;
+TM_API int tm_delta_rule(tm_handle* h, const tm_delta_rule_params* d, const tm_mixer_call* c, void* stream);
+/* out[t][n] = sum_k x[t][k] * w[n][k]: bf16 on the tcgen05 tensor core (ld multiples of 8, 16-byte aligned; out in bf16, or
+ * in fp32 with out_f32), or fp32 throughout */
+TM_API int tm_gemm_dense(tm_handle* h, void* out, int out_ld, int out_f32, const void* x, int x_ld, const void* w, int w_ld, int tokens,
+                         int n_out, int k, int dtype, void* stream);
+
+/* ------------------------------------------------------------------------------------------
+ * Persistent-batch scheduler over tm_cache_*, tm_model_prefill, tm_model_decode, tm_sample_topk / tm_sample_topp and
  * tm_ban_bad_words: the part of
  * LlamaBatch<T> (src/turbomind/models/llama/LlamaBatch.cc: initialize :562-763, contextDecode :765-877, generate
  * :471-559, finish / finishRequest :930-970, 1056-1118) that decides who runs.  Requests wait in a queue; every
@@ -628,6 +747,8 @@ typedef struct tm_request {
     int                step;               /* input of the reference's requests, LlamaBatch.cc:587-596); 0: history kept     */
 } tm_request;
 enum { TM_REQUEST_QUEUED = 0, TM_REQUEST_RUNNING = 1, TM_REQUEST_FINISHED = 2, TM_REQUEST_FAILED = 3 };
+TM_API int tm_batch_create_model(tm_batch** out, tm_model* model, tm_cache_manager* cache, int max_batch_size, int session_len,
+                                 int start_id, int end_id, int max_context_token_num);
 TM_API int tm_batch_create(tm_batch** out, tm_llama* model, tm_cache_manager* cache, int max_batch_size, int session_len,
                            int start_id, int end_id, int max_context_token_num);
 TM_API int tm_batch_destroy(tm_batch* b);

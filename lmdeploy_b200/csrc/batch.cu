@@ -11,7 +11,7 @@
 // One scheduler is driven by one host thread; every call works on the stream it is given.
 #include "common.cuh"
 #include "handle.h"
-#include "llama.h"
+#include "model.h"
 #include "tm_b200.h"
 
 #include <algorithm>
@@ -54,7 +54,7 @@ __global__ void append_history_kernel(int* hist, const int* ids, const int* lens
 }  // namespace tmb
 
 struct tm_batch {
-    tm_llama*         model   = nullptr;
+    tm_model*         model   = nullptr;
     tm_cache_manager* cache   = nullptr;
     int               max_batch = 0, session_len = 0, vocab = 0, start_id = 0, end_id = 0, max_context_tokens = 0;
     int               device = 0;
@@ -76,11 +76,6 @@ struct tm_batch {
     int*                d_bad  = nullptr;  // [max batch][2][kMaxBadWords]: the live requests' banned tokens as word lists
     unsigned char*      d_skip = nullptr;  // [2][max batch]: rows the top-k draw leaves alone | rows the top-p draw leaves alone
     unsigned long long* d_seed = nullptr;
-    // prefill staging (grown on demand)
-    int*   d_pf_ids = nullptr;
-    size_t pf_capacity = 0;
-    int *  d_pf_cu = nullptr, *d_pf_hist = nullptr, *d_pf_ctx = nullptr;
-    void **d_pf_k = nullptr, **d_pf_v = nullptr;
     // pinned host
     int* h_ids = nullptr;
 
@@ -100,8 +95,7 @@ bool dev_alloc(T** p, size_t count)
 void batch_free(tm_batch* b)
 {
     void* ptrs[] = {b->d_k,    b->d_v,    b->d_len,  b->d_forced, b->d_out,    b->d_step,  b->d_ids,   b->d_hist, b->d_topk, b->d_hist_len,
-                    b->d_logits, b->d_topp, b->d_temp, b->d_rep,    b->d_rng,    b->d_seed,  b->d_pf_ids, b->d_pf_cu, b->d_pf_hist, b->d_pf_ctx,
-                    b->d_pf_k, b->d_pf_v, b->d_skip, b->d_bad};
+                    b->d_logits, b->d_topp, b->d_temp, b->d_rep,    b->d_rng,    b->d_seed,  b->d_skip, b->d_bad};
     for (void* p : ptrs) {
         if (p) cudaFree(p);
     }
@@ -111,11 +105,11 @@ void batch_free(tm_batch* b)
 
 }  // namespace
 
-extern "C" int tm_batch_create(tm_batch** out, tm_llama* model, tm_cache_manager* cache, int max_batch_size, int session_len,
-                               int start_id, int end_id, int max_context_token_num)
+extern "C" int tm_batch_create_model(tm_batch** out, tm_model* model, tm_cache_manager* cache, int max_batch_size, int session_len,
+                                     int start_id, int end_id, int max_context_token_num)
 {
     if (!out || !model || !cache || max_batch_size <= 0 || session_len <= 1) return TM_ERR_INVALID_ARG;
-    if (max_batch_size > model->cfg.max_batch_size || session_len > model->cfg.session_len) return TM_ERR_INVALID_ARG;
+    if (max_batch_size > model->max_batch_size || session_len > model->session_len) return TM_ERR_INVALID_ARG;
     *out        = nullptr;
     tm_batch* b = new (std::nothrow) tm_batch();
     if (!b) return TM_ERR_CUDA;
@@ -123,7 +117,7 @@ extern "C" int tm_batch_create(tm_batch** out, tm_llama* model, tm_cache_manager
     b->cache              = cache;
     b->max_batch          = max_batch_size;
     b->session_len        = session_len;
-    b->vocab              = model->cfg.vocab_size;
+    b->vocab              = model->vocab_size;
     b->start_id           = start_id;
     b->end_id             = end_id;
     b->max_context_tokens = max_context_token_num > 0 ? max_context_token_num : session_len;
@@ -134,8 +128,7 @@ extern "C" int tm_batch_create(tm_batch** out, tm_llama* model, tm_cache_manager
               && dev_alloc(&b->d_out, B) && dev_alloc(&b->d_step, 1) && dev_alloc(&b->d_ids, B)
               && dev_alloc(&b->d_hist, B * session_len) && dev_alloc(&b->d_topk, B) && dev_alloc(&b->d_hist_len, B)
               && dev_alloc(&b->d_logits, B * b->vocab) && dev_alloc(&b->d_topp, B) && dev_alloc(&b->d_temp, B) && dev_alloc(&b->d_rep, B)
-              && dev_alloc(&b->d_seed, B) && dev_alloc(&b->d_pf_cu, B + 1) && dev_alloc(&b->d_pf_hist, B) && dev_alloc(&b->d_pf_ctx, B)
-              && dev_alloc(&b->d_pf_k, B) && dev_alloc(&b->d_pf_v, B) && dev_alloc(&b->d_skip, 2 * B) && dev_alloc(&b->d_bad, B * 2 * kMaxBadWords);
+              && dev_alloc(&b->d_seed, B) && dev_alloc(&b->d_skip, 2 * B) && dev_alloc(&b->d_bad, B * 2 * kMaxBadWords);
     ok = ok && cudaMalloc(&b->d_rng, B * tm_sampling_rng_state_bytes()) == cudaSuccess;
     ok = ok && cudaMallocHost((void**)&b->h_ids, B * sizeof(int)) == cudaSuccess;
     ok = ok && cudaMemset(b->d_hist, 0, B * session_len * sizeof(int)) == cudaSuccess;
@@ -219,9 +212,8 @@ namespace {
 // except the last one, which goes through the decoder step (LlamaV2::contextDecode, LlamaV2.cc:204).
 int prefill_group(tm_batch* b, const std::vector<int>& group, const std::vector<int>& cached, cudaStream_t s)
 {
-    std::vector<int>   ids, cu{0}, hist, ctx;
+    std::vector<int>   ids, cu{0}, hist;
     std::vector<void*> kp, vp;
-    int                max_q = 0;
     for (size_t g = 0; g < group.size(); ++g) {
         const Slot& sl = b->slots[group[g]];
         const int   n  = (int)sl.tokens.size() - 1 - cached[g];
@@ -229,39 +221,18 @@ int prefill_group(tm_batch* b, const std::vector<int>& group, const std::vector<
         ids.insert(ids.end(), sl.tokens.begin() + cached[g], sl.tokens.end() - 1);
         cu.push_back((int)ids.size());
         hist.push_back(cached[g]);
-        ctx.push_back(cached[g] + n);
         kp.push_back(sl.seq.k_cache);
         vp.push_back(sl.seq.v_cache);
-        max_q = std::max(max_q, n);
     }
     if (ids.empty()) return TM_OK;
-    if (ids.size() > b->pf_capacity) {
-        if (b->d_pf_ids) cudaFree(b->d_pf_ids);
-        b->d_pf_ids    = nullptr;
-        b->pf_capacity = 0;
-        if (cudaMalloc((void**)&b->d_pf_ids, ids.size() * sizeof(int)) != cudaSuccess) return TM_ERR_CUDA;
-        b->pf_capacity = ids.size();
-    }
-    const size_t n = hist.size();
-    bool ok = cudaMemcpyAsync(b->d_pf_ids, ids.data(), ids.size() * sizeof(int), cudaMemcpyHostToDevice, s) == cudaSuccess
-              && cudaMemcpyAsync(b->d_pf_cu, cu.data(), cu.size() * sizeof(int), cudaMemcpyHostToDevice, s) == cudaSuccess
-              && cudaMemcpyAsync(b->d_pf_hist, hist.data(), n * sizeof(int), cudaMemcpyHostToDevice, s) == cudaSuccess
-              && cudaMemcpyAsync(b->d_pf_ctx, ctx.data(), n * sizeof(int), cudaMemcpyHostToDevice, s) == cudaSuccess
-              && cudaMemcpyAsync(b->d_pf_k, kp.data(), n * sizeof(void*), cudaMemcpyHostToDevice, s) == cudaSuccess
-              && cudaMemcpyAsync(b->d_pf_v, vp.data(), n * sizeof(void*), cudaMemcpyHostToDevice, s) == cudaSuccess;
-    if (!ok) return TM_ERR_CUDA;
-    tm_llama_prefill_state st{};
-    st.batch_size      = (int)n;
-    st.token_num       = (int)ids.size();
-    st.max_q_len       = max_q;
-    st.input_ids       = b->d_pf_ids;
-    st.cu_seqlens      = b->d_pf_cu;
-    st.history_lengths = b->d_pf_hist;
-    st.context_lengths = b->d_pf_ctx;
-    st.k_cache_ptrs    = b->d_pf_k;
-    st.v_cache_ptrs    = b->d_pf_v;
-    const int rc       = tm_llama_prefill(b->model, &st, s);
-    // the staging vectors above are pageable: their copies were staged before cudaMemcpyAsync returned
+    tm_model_prefill_state st{};
+    st.batch_size      = (int)hist.size();
+    st.input_ids       = ids.data();
+    st.cu_seqlens      = cu.data();
+    st.history_lengths = hist.data();
+    st.k_cache         = kp.data();
+    st.v_cache         = vp.data();
+    const int rc       = tm_model_prefill(b->model, &st, s);
     if (rc == TM_OK) b->prefill_tokens += ids.size();
     return rc;
 }
@@ -340,10 +311,13 @@ extern "C" int tm_batch_step(tm_batch* b, void* stream, int use_graph)
             // the session goes back to its first `step` tokens (LlamaBatch.cc:587-596; a step beyond the history is
             // ignored there with a warning, here silently); rows of the slab beyond them are overwritten as needed
             sl.tokens.resize(r.step);
-            cached = std::min(cached, r.step);
+            if (r.step < cached) cached = b->model->can_rewind() ? r.step : 0;
         }
         sl.tokens.insert(sl.tokens.end(), ids.begin(), ids.end());
         if (sl.tokens.empty()) sl.tokens.push_back(b->start_id);  // LlamaBatch.cc:599-604
+        // the last token goes through the decoder step: a state that has taken it in already, and cannot go back, is
+        // built again from the first token
+        if (cached >= (int)sl.tokens.size() && !b->model->can_rewind()) cached = 0;
         const int context_len = (int)sl.tokens.size();
         if (context_len >= b->session_len) {
             // no room for even one new token: refuse (the reference truncates request_output_len to nothing and warns)
@@ -452,7 +426,7 @@ extern "C" int tm_batch_step(tm_batch* b, void* stream, int use_graph)
     st.output_ids       = b->d_out;
     st.step             = b->d_step;
     st.logits_out       = b->d_logits;
-    if ((rc = tm_llama_decode(b->model, &st, 1, use_graph, s)) != TM_OK) return rc;
+    if ((rc = tm_model_decode(b->model, &st, 1, use_graph, s)) != TM_OK) return rc;
 
     // bad_words_list of the requests (DynamicDecodeLayer.cc:214-236): single tokens, as the reference's scheduler takes
     // them, banned through the word-list kernel (an item of one token is banned whatever came before it)

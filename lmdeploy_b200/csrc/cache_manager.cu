@@ -121,15 +121,10 @@ struct tm_cache_manager {
     }
 };
 
-extern "C" int tm_cache_manager_create(tm_cache_manager** out, size_t layer_num, size_t head_num, size_t size_per_head,
-                                       size_t max_seq_len, size_t elem_bits, size_t max_entry_count, size_t chunk_size, int device)
+static int create_manager(tm_cache_manager** out, size_t half_slab_bytes, size_t max_seq_len, size_t max_entry_count, size_t chunk_size, int device)
 {
-    if (!out || !layer_num || !head_num || !size_per_head || !max_seq_len || !elem_bits || elem_bits % 8 || !max_entry_count
-        || !chunk_size) {
-        return TM_ERR_INVALID_ARG;
-    }
     auto* m        = new tm_cache_manager;
-    m->cache_bytes = layer_num * head_num * max_seq_len * size_per_head * elem_bits / 8;
+    m->cache_bytes = half_slab_bytes;
     m->max_entries = max_entry_count, m->chunk_size = chunk_size, m->max_seq_len = max_seq_len, m->device = device;
     int prev = 0, rc = TM_OK;
     if (device >= 0) {
@@ -147,6 +142,24 @@ extern "C" int tm_cache_manager_create(tm_cache_manager** out, size_t layer_num,
     }
     *out = m;
     return TM_OK;
+}
+
+extern "C" int tm_cache_manager_create(tm_cache_manager** out, size_t layer_num, size_t head_num, size_t size_per_head,
+                                       size_t max_seq_len, size_t elem_bits, size_t max_entry_count, size_t chunk_size, int device)
+{
+    if (!out || !layer_num || !head_num || !size_per_head || !max_seq_len || !elem_bits || elem_bits % 8 || !max_entry_count
+        || !chunk_size) {
+        return TM_ERR_INVALID_ARG;
+    }
+    return create_manager(out, layer_num * head_num * max_seq_len * size_per_head * elem_bits / 8, max_seq_len, max_entry_count, chunk_size, device);
+}
+
+// Slabs of a model that lays them out itself: k_cache is the slab's start (v_cache its middle, of no meaning then)
+extern "C" int tm_cache_manager_create_slabs(tm_cache_manager** out, size_t slab_bytes, size_t max_seq_len, size_t max_entry_count,
+                                             size_t chunk_size, int device)
+{
+    if (!out || !slab_bytes || !max_seq_len || !max_entry_count || !chunk_size) return TM_ERR_INVALID_ARG;
+    return create_manager(out, (slab_bytes + 511) / 512 * 256, max_seq_len, max_entry_count, chunk_size, device);
 }
 
 extern "C" int tm_cache_manager_destroy(tm_cache_manager* m)

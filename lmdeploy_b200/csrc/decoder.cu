@@ -1,0 +1,628 @@
+// Config-driven decoder (decoder.h): set-up, weights, prefill passes and the decode step.
+#include "decoder.h"
+#include "common.cuh"
+#include "numeric.cuh"
+#include "safetensors.h"
+#include "step_kernels.h"
+
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+
+using namespace tmb;
+
+namespace tmb {
+namespace {
+
+constexpr int kDefaultPrefill = 4096;
+constexpr int kWantRows       = 256;  // rows of one lm-head product of a prefill
+
+int round_up(int x, int m)
+{
+    return (x + m - 1) / m * m;
+}
+size_t round_up_bytes(size_t x)
+{
+    return (x + 255) / 256 * 256;
+}
+
+// x row (from the embedding when ids are given), its copy in the element type and its sum of squares: one CTA per token
+template<typename E>
+__global__ void __launch_bounds__(256) rows_kernel(float* x, E* xb, float* ssq, const E* embed, const int* ids, float scale, int width, int x_ld,
+                                                   int vocab)
+{
+    __shared__ float red[8];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int t  = blockIdx.x;
+    float*    xr = x + (size_t)t * width;
+    E*        br = xb + (size_t)t * x_ld;
+    const E*  er = ids ? embed + (size_t)min(max(ids[t], 0), vocab - 1) * width : nullptr;
+    float     sq = 0.f;
+    for (int i = threadIdx.x; i < width; i += 256) {
+        const float v = er ? to_f32(er[i]) * scale : xr[i];
+        if (er) xr[i] = v;
+        br[i] = from_f32<E>(v);
+        sq += v * v;
+    }
+    sq = warp_sum(sq);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        float s = 0.f;
+        for (int i = 0; i < 8; ++i) s += red[i];
+        ssq[t] = s;
+    }
+}
+
+// rows `want[i]` of xb / ssq -> row i of the gathered copies
+template<typename E>
+__global__ void gather_rows_kernel(E* dst, float* dst_ssq, const E* xb, const float* ssq, const int* want, int x_ld)
+{
+    const int i = blockIdx.x, t = want[i];
+    for (int c = threadIdx.x; c < x_ld; c += blockDim.x) dst[(size_t)i * x_ld + c] = xb[(size_t)t * x_ld + c];
+    if (threadIdx.x == 0) dst_ssq[i] = ssq[t];
+}
+
+// one span and one input token per sequence of a decode step
+__global__ void step_spans_kernel(const tm_llama_decode_state st, const int* picked, int* ids, unsigned char* inactive, SeqSpan* spans, int vocab,
+                                  int session_len)
+{
+    const int b = blockIdx.x * blockDim.x + threadIdx.x;
+    if (b >= st.batch_size) return;
+    bool      off = false;
+    const int id  = step_input(st.step, st.start_step, st.forced_ids, picked, b, st.batch_size, st.max_steps, vocab, &off);
+    const int len = st.sequence_lengths[b];
+    ids[b]        = id;
+    inactive[b]   = off ? 1 : 0;
+    SeqSpan s;
+    s.slab    = static_cast<unsigned char*>(st.k_cache_ptrs[b]);
+    s.history = len;
+    s.n       = 1;
+    s.tok0    = b;
+    s.live    = !off && len < session_len ? 1 : 0;
+    spans[b]  = s;
+}
+
+__device__ __forceinline__ float hash_normal(unsigned long long seed, unsigned long long i)
+{
+    auto mix = [](unsigned long long z) {  // splitmix64 finaliser
+        z = (z ^ (z >> 30)) * 0xbf58476d1ce4e5b9ull;
+        z = (z ^ (z >> 27)) * 0x94d049bb133111ebull;
+        return z ^ (z >> 31);
+    };
+    const unsigned long long r = mix(seed + 0x9e3779b97f4a7c15ull * (i + 1));
+    const float u = ((unsigned)(r >> 40) + 1) * (1.f / 16777217.f), v = (unsigned)((r >> 8) & 0xffffff) * (1.f / 16777216.f);
+    return sqrtf(-2.f * logf(u)) * cospif(2.f * v);
+}
+template<typename E>
+__global__ void random_kernel(E* dst, long long rows, long long cols, long long row_stride, float mean, float std, unsigned long long seed)
+{
+    const long long n = rows * cols;
+    for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        dst[(i / cols) * row_stride + i % cols] = from_f32<E>(mean + std * hash_normal(seed, (unsigned long long)i));
+    }
+}
+
+float half_to_float(uint16_t h)
+{
+    const int   e = (h >> 10) & 31, m = h & 1023;
+    const float v = e == 0 ? std::ldexp((float)m, -24) : (e == 31 ? (m ? NAN : INFINITY) : std::ldexp((float)(m + 1024), e - 25));
+    return h & 0x8000 ? -v : v;
+}
+float element_as_float(const unsigned char* p, const std::string& dtype)
+{
+    if (dtype == "F32") {
+        float f;
+        std::memcpy(&f, p, 4);
+        return f;
+    }
+    uint16_t h;
+    std::memcpy(&h, p, 2);
+    if (dtype == "F16") return half_to_float(h);
+    const uint32_t w = (uint32_t)h << 16;
+    float          f;
+    std::memcpy(&f, &w, 4);
+    return f;
+}
+uint16_t float_to_bf16(float f)
+{
+    uint32_t w;
+    std::memcpy(&w, &f, 4);
+    if ((w & 0x7fffffffu) > 0x7f800000u) return 0x7fff;
+    return (uint16_t)((w + 0x7fffu + ((w >> 16) & 1)) >> 16);
+}
+
+}  // namespace
+}  // namespace tmb
+
+bool tm_decoder::alloc(void** p, size_t bytes)
+{
+    bytes = std::max<size_t>(bytes, 256);
+    if (cudaMalloc(p, bytes) != cudaSuccess) {
+        *p = nullptr;
+        cudaGetLastError();
+        return false;
+    }
+    owned.push_back(*p);
+    return cudaMemset(*p, 0, bytes) == cudaSuccess;
+}
+
+tm_decoder::~tm_decoder()
+{
+    graph.drop();
+    for (void* p : owned) cudaFree(p);
+}
+
+int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_options& opt)
+{
+    h              = handle;
+    cfg            = c;
+    f32            = opt.dtype == TM_DTYPE_F32;
+    vocab_size     = c.vocab;
+    max_batch_size = opt.max_batch_size;
+    session_len    = opt.session_len;
+    max_prefill    = std::min(opt.max_prefill_tokens > 0 ? opt.max_prefill_tokens : kDefaultPrefill, std::max(16, session_len * max_batch_size));
+    int prev = 0;
+    cudaGetDevice(&prev);
+    cudaSetDevice(h->device);
+    const size_t es = f32 ? 4 : 2;
+    const int    W = c.width, tokens = std::max(max_prefill, max_batch_size);
+    bool         ok = true;
+    x_ld            = round_up(W, 8);
+    size_t off      = 0;
+    int    delta_cols = 0;
+    auto   take = [&](size_t bytes) {
+        const size_t at = off;
+        off             = round_up_bytes(off + bytes);
+        return at;
+    };
+    auto target = [&](const std::string& name, int64_t rows, int64_t cols, void* dst, int64_t stride) -> WeightTarget& {
+        WeightTarget t;
+        t.name = name, t.rows = rows, t.cols = cols, t.dst = dst, t.row_stride = stride;
+        t.init_std = 1.f / std::sqrt((float)cols);
+        targets.push_back(t);
+        return targets.back();
+    };
+    auto vec = [&](const std::string& name, int64_t n, float** dst, float mean, float std) {
+        ok             = ok && alloc((void**)dst, n * 4);
+        WeightTarget& t = target(name, 1, n, *dst, n);
+        t.vector = true, t.f32 = true, t.init_mean = mean, t.init_std = std;
+    };
+    auto gain = [&](const std::string& name, float** dst) {
+        vec(name, 1, dst, 1.f, 0.f);
+        targets.back().scalar = true;
+    };
+    auto at = [&](void* base, int64_t row, int64_t ld, int64_t col = 0) { return static_cast<char*>(base) + (size_t)(row * ld + col) * es; };
+
+    layers.resize(c.layers.size());
+    for (size_t i = 0; i < layers.size() && ok; ++i) {
+        DecoderLayer&     L = layers[i];
+        const MixerSpec&  m = c.layers[i].mixer;
+        const std::string p = "l" + std::to_string(i) + ".", mp = p + "mix.";
+        L.spec              = c.layers[i];
+        const int ff        = L.spec.ff;
+        int       cols      = 0;
+        auto      segment   = [&](int n) {
+            const int at0 = cols;
+            cols += round_up(n, 8);
+            return at0;
+        };
+        struct Part {
+            const char* name;
+            int         rows, col;
+        };
+        std::vector<Part> parts;
+        if (m.type == MixerType::kAttention) {
+            WindowAttention& a = L.attention;
+            a.heads = m.heads, a.kv_heads = m.kv_heads, a.dim = m.dim, a.vdim = m.vdim, a.rot_dims = m.rot_dims;
+            a.scale = (float)m.scale, a.softcap = (float)m.softcap, a.window = m.window, a.pool = m.pool;
+            a.q_col = segment(m.heads * m.dim), a.k_col = segment(m.kv_heads * m.dim), a.v_col = segment(m.kv_heads * m.vdim);
+            a.g_col = segment(m.heads);
+            parts   = {{"q", m.heads * m.dim, a.q_col}, {"k", m.kv_heads * m.dim, a.k_col}, {"v", m.kv_heads * m.vdim, a.v_col}, {"g", m.heads, a.g_col}};
+            // the oldest query of a pass still sees its window, and the pass completes blocks that began before it
+            const long long keep = (long long)std::max(m.window, m.pool) + max_prefill;
+            a.ring               = round_up((int)std::min<long long>(m.window > 0 ? keep : session_len, session_len), 128);
+            a.pool_rows          = m.pool > 0 ? round_up(std::max(1, session_len / m.pool), 8) : 0;
+            a.k_off              = take((size_t)m.kv_heads * a.ring * m.dim * es);
+            a.v_off              = take((size_t)m.kv_heads * a.ring * m.vdim * es);
+            a.pk_off             = take((size_t)m.kv_heads * a.pool_rows * m.dim * es);
+            a.pv_off             = take((size_t)m.kv_heads * a.pool_rows * m.vdim * es);
+            std::vector<float> f(std::max(1, m.rot_dims / 2));
+            for (int k = 0; k < m.rot_dims / 2; ++k) f[k] = (float)(std::pow(m.rot_base, -2.0 * k / m.rot_dims) / m.rot_factor);
+            ok = ok && alloc((void**)&L.inv_freq, f.size() * 4) && cudaMemcpy(L.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice) == cudaSuccess;
+            a.inv_freq = L.inv_freq;
+        }
+        else {
+            DeltaRule& d = L.delta;
+            const int  n = m.heads * m.dim;
+            d.heads = m.heads, d.dim = m.dim, d.rank = m.rank, d.norm_eps = (float)c.norm_eps;
+            d.r_col = segment(n), d.k_col = segment(n), d.v_col = segment(n), d.a_col = segment(n), d.g_col = segment(n), d.w1_col = segment(m.rank);
+            parts = {{"r", n, d.r_col}, {"k", n, d.k_col}, {"v", n, d.v_col}, {"a", n, d.a_col}, {"g", n, d.g_col}, {"w1", m.rank, d.w1_col}};
+            L.tanh_lo = d.w1_col, L.tanh_hi = d.w1_col + m.rank;
+            d.w2_ld     = round_up(m.rank, 8);
+            d.state_off = take((size_t)m.heads * m.dim * m.dim * 4);
+            ok          = ok && alloc(&L.w2, (size_t)n * d.w2_ld * es);
+            target(mp + "w2", n, m.rank, L.w2, d.w2_ld);
+            vec(mp + "w0", n, &L.w0, 0.f, 1.f);
+            vec(mp + "a.b", n, &L.a_bias, 0.f, 1.f);
+            vec(mp + "norm", n, &L.norm, 1.f, 0.f);
+            d.w2 = L.w2, d.w0 = L.w0, d.a_bias = L.a_bias, d.norm = L.norm;
+            delta_cols = std::max(delta_cols, n);
+        }
+        L.mixer_cols = round_up(cols, kDenseTile);
+        L.in_rows    = L.mixer_cols + 2 * ff;
+        L.mix_pad    = round_up(m.out_width(), 8);
+        L.out_k      = L.mix_pad + ff;
+        ok = ok && alloc(&L.w_in, (size_t)L.in_rows * x_ld * es) && alloc(&L.w_out, (size_t)W * round_up(L.out_k, 8) * es);
+        if (!ok) break;
+        gain(p + "norm1", &L.gain);
+        for (const Part& q : parts) target(mp + q.name, q.rows, W, at(L.w_in, q.col, x_ld), x_ld);
+        target(mp + "o", W, m.out_width(), L.w_out, round_up(L.out_k, 8)).init_std *= 0.5f;
+        if (ff > 0) {
+            target(p + "mlp.gate", ff, W, at(L.w_in, L.mixer_cols, x_ld), 2 * x_ld);
+            target(p + "mlp.up", ff, W, at(L.w_in, L.mixer_cols + 1, x_ld), 2 * x_ld);
+            target(p + "mlp.down", W, ff, at(L.w_out, 0, 0, L.mix_pad), round_up(L.out_k, 8)).init_std *= 0.5f;
+        }
+        proj_ld = std::max(proj_ld, L.mixer_cols);
+        y_ld    = std::max(y_ld, round_up(L.out_k, 8));
+    }
+    slab = std::max<size_t>(off, 256);
+    ok   = ok && alloc(&embed, (size_t)c.vocab * W * es) && alloc(&head, (size_t)c.vocab * x_ld * es);
+    if (ok) {
+        target("embed", c.vocab, W, embed, W).init_std = 1.f;
+        target("head", c.vocab, W, head, x_ld);
+        gain("final.norm", &final_gain);
+    }
+    ssq_stride            = round_up(tokens, 8);
+    const size_t T        = (size_t)tokens, column_tiles = (size_t)(W + kDenseTile - 1) / kDenseTile;
+    const size_t logit_rows = (size_t)max_batch_size;
+    ok = ok && alloc((void**)&x, T * W * 4) && alloc((void**)&ssq, column_tiles * ssq_stride * 4) && alloc(&xb, T * x_ld * es)
+         && alloc(&proj, T * proj_ld * es) && alloc(&y, T * y_ld * es) && alloc((void**)&decay_pre, T * delta_cols * 4)
+         && alloc((void**)&delta_o, T * delta_cols * 4) && alloc((void**)&logits, logit_rows * c.vocab * 4)
+         && alloc(&want_xb, (size_t)kWantRows * x_ld * es) && alloc((void**)&want_ssq, (size_t)kWantRows * 4) && alloc((void**)&ids, T * 4)
+         && alloc((void**)&want, T * 4) && alloc((void**)&picked, T * 4) && alloc((void**)&inactive, T) && alloc((void**)&spans, T * sizeof(SeqSpan));
+    const cudaError_t e = cudaGetLastError();
+    cudaSetDevice(prev);
+    if (!ok) {
+        h->last_cuda_error = (int)e;
+        return TM_ERR_CUDA;
+    }
+    return TM_OK;
+}
+
+int tm_decoder::load(const std::string& path, std::string* why)
+{
+    SafeTensors st;
+    if (!st.open(path)) {
+        *why = "cannot read " + path;
+        return TM_ERR_IO;
+    }
+    int prev = 0;
+    cudaGetDevice(&prev);
+    cudaSetDevice(h->device);
+    int                        rc = TM_OK;
+    std::vector<unsigned char> raw, converted;
+    for (const WeightTarget& t : targets) {
+        const SafeTensor* s     = st.find(t.name);
+        bool              match = s && (s->dtype == "BF16" || s->dtype == "F32" || s->dtype == "F16");
+        if (match) {
+            if (t.scalar) {
+                match = s->count() == 1;
+            }
+            else if (t.vector) {
+                match = s->shape.size() == 1 && s->shape[0] == t.cols;
+            }
+            else {
+                match = s->shape.size() == 2 && s->shape[0] == t.rows && s->shape[1] == t.cols;
+            }
+        }
+        if (!match || !st.read(*s, raw)) {
+            *why = (s ? "tensor of another shape or type: " : "missing tensor: ") + t.name;
+            rc   = TM_ERR_IO;
+            break;
+        }
+        const size_t n = (size_t)(t.rows * t.cols), in = s->dtype == "F32" ? 4 : 2, es = t.f32 || f32 ? 4 : 2;
+        const void*  src = raw.data();
+        if (!(es == 4 && s->dtype == "F32") && !(es == 2 && s->dtype == "BF16")) {
+            converted.resize(n * es);
+            for (size_t i = 0; i < n; ++i) {
+                const float v = element_as_float(raw.data() + i * in, s->dtype);
+                if (es == 4) {
+                    std::memcpy(converted.data() + i * 4, &v, 4);
+                }
+                else {
+                    const uint16_t b = float_to_bf16(v);
+                    std::memcpy(converted.data() + i * 2, &b, 2);
+                }
+            }
+            src = converted.data();
+        }
+        if (cudaMemcpy2D(t.dst, (size_t)t.row_stride * es, src, (size_t)t.cols * es, (size_t)t.cols * es, (size_t)t.rows, cudaMemcpyHostToDevice)
+            != cudaSuccess) {
+            *why = "copy to the device failed: " + t.name;
+            rc   = TM_ERR_CUDA;
+            break;
+        }
+    }
+    cudaSetDevice(prev);
+    return rc;
+}
+
+int tm_decoder::random_weights(unsigned long long seed)
+{
+    int prev = 0;
+    cudaGetDevice(&prev);
+    cudaSetDevice(h->device);
+    unsigned long long k = seed * 1000003ull;
+    for (const WeightTarget& t : targets) {
+        k += 7919;
+        if (t.f32 || f32) {
+            random_kernel<float><<<1024, 256>>>(static_cast<float*>(t.dst), t.rows, t.cols, t.row_stride, t.init_mean, t.init_std, k);
+        }
+        else {
+            random_kernel<__nv_bfloat16><<<1024, 256>>>(static_cast<__nv_bfloat16*>(t.dst), t.rows, t.cols, t.row_stride, t.init_mean, t.init_std, k);
+        }
+    }
+    const cudaError_t e = cudaDeviceSynchronize();
+    cudaSetDevice(prev);
+    return e == cudaSuccess ? TM_OK : TM_ERR_CUDA;
+}
+
+int tm_decoder::new_cache(tm_cache_manager** out, size_t max_entry_count, size_t chunk_size) const
+{
+    return tm_cache_manager_create_slabs(out, slab, (size_t)session_len, max_entry_count, chunk_size, h->device);
+}
+
+// The tokens of one pass through the layers; spans, ids are on the device already
+struct tm_decoder::Pass {
+    int  batch = 0, tokens = 0, max_n = 0;
+    bool decode = false, fold = false, pdl = false;
+    bool need_output = true;        // whether anybody reads what the last layer leaves
+    // after every layer: residual rows out (prefill, optional)
+    float* const* residual_rows = nullptr;  // [batch] destination of each span's rows of layer 0
+    size_t        residual_layer_stride = 0;
+    const SeqSpan* host_spans = nullptr;
+};
+
+int tm_decoder::run_layers(const Pass& p, cudaStream_t s)
+{
+    const int  W   = cfg.width;
+    const bool pdl = p.pdl;
+    auto rows = [&](const int* token_ids) {
+        cudaError_t e;
+        if (f32) {
+            e = launch_kernel(rows_kernel<float>, dim3(p.tokens), dim3(256), 0, s, pdl, x, static_cast<float*>(xb), ssq, static_cast<const float*>(embed),
+                              token_ids, (float)cfg.embedding_scale, W, x_ld, cfg.vocab);
+        }
+        else {
+            using B = __nv_bfloat16;
+            e = launch_kernel(rows_kernel<B>, dim3(p.tokens), dim3(256), 0, s, pdl, x, static_cast<B*>(xb), ssq, static_cast<const B*>(embed), token_ids,
+                              (float)cfg.embedding_scale, W, x_ld, cfg.vocab);
+        }
+        ++h->launches;
+        return e == cudaSuccess ? TM_OK : TM_ERR_CUDA;
+    };
+    int rc = rows(ids);
+    int ssq_parts = 1;
+    for (size_t l = 0; l < layers.size() && rc == TM_OK; ++l) {
+        const DecoderLayer& L    = layers[l];
+        const bool          last = l + 1 == layers.size();
+        DenseGemm           g;
+        g.w = L.w_in, g.ldw = x_ld, g.x = xb, g.ldx = x_ld, g.tokens = p.tokens, g.n_out = L.in_rows, g.k = W;
+        g.ep.kind = DenseKind::kInput;
+        g.ep.ssq = ssq, g.ep.ssq_parts = ssq_parts, g.ep.ssq_stride = ssq_stride, g.ep.inv_width = 1.f / (float)W, g.ep.eps = (float)cfg.norm_eps;
+        g.ep.gain = L.gain;
+        g.ep.out = proj, g.ep.out_ld = proj_ld, g.ep.tanh_lo = L.tanh_lo, g.ep.tanh_hi = L.tanh_hi, g.ep.split = L.mixer_cols;
+        g.ep.act = static_cast<char*>(y) + (size_t)L.mix_pad * (f32 ? 4 : 2), g.ep.act_ld = y_ld;
+        if ((rc = dense_gemm(h, g, f32, s, pdl)) != TM_OK) break;
+
+        MixerCall c;
+        c.proj = proj, c.proj_ld = proj_ld, c.out = y, c.out_ld = y_ld, c.out_pad = L.mix_pad, c.spans = spans, c.batch = p.batch;
+        c.tokens = p.tokens, c.max_n = p.max_n, c.max_context = session_len, c.f32 = f32, c.pdl = pdl;
+        if (L.spec.mixer.type == MixerType::kAttention) {
+            rc = p.decode ? window_attention_decode(h, L.attention, c, s) : window_attention_prefill(h, L.attention, c, s);
+        }
+        else {
+            rc = p.decode ? delta_rule_decode(h, L.delta, c, s) : delta_rule_prefill(h, L.delta, c, decay_pre, delta_o, s);
+        }
+        if (rc != TM_OK || (last && !p.need_output)) break;
+
+        DenseGemm o;
+        o.w = L.w_out, o.ldw = round_up(L.out_k, 8), o.x = y, o.ldx = y_ld, o.tokens = p.tokens, o.n_out = W, o.k = L.out_k;
+        o.ep.kind = DenseKind::kResidual, o.ep.residual = x, o.ep.residual_ld = W;
+        if (p.fold) {
+            o.ep.cast = xb, o.ep.cast_ld = x_ld, o.ep.ssq_out = ssq, o.ep.ssq_out_stride = ssq_stride;
+            ssq_parts = (W + kDenseTile - 1) / kDenseTile;
+        }
+        if ((rc = dense_gemm(h, o, f32, s, pdl)) != TM_OK) break;
+        if (p.residual_rows) {
+            for (int b = 0; b < p.batch; ++b) {
+                if (cudaMemcpyAsync(p.residual_rows[b] + l * p.residual_layer_stride, x + (size_t)p.host_spans[b].tok0 * W,
+                                    (size_t)p.host_spans[b].n * W * 4, cudaMemcpyDeviceToDevice, s)
+                    != cudaSuccess) {
+                    return TM_ERR_CUDA;
+                }
+            }
+        }
+        if (!p.fold) rc = rows(nullptr);
+    }
+    return rc;
+}
+
+int tm_decoder::prefill(const tm_model_prefill_state& st, cudaStream_t s)
+{
+    const int B = st.batch_size, total = st.cu_seqlens[B];
+    if (total == 0) return TM_OK;
+    const size_t V = (size_t)cfg.vocab, W = (size_t)cfg.width;
+    std::vector<int> done(B, 0);
+    for (int left = total; left > 0;) {
+        // ---- one pass: the sequences in turn, each with as many of its tokens as still fit
+        std::vector<SeqSpan> sp;
+        std::vector<int>     tok, wanted, want_seq_begin;  // wanted: rows of this pass
+        std::vector<float*>  res_rows, logit_rows;         // destination per span
+        Pass                 p;
+        for (int b = 0; b < B && p.tokens < max_prefill; ++b) {
+            const int begin = st.cu_seqlens[b] + done[b], n = std::min(st.cu_seqlens[b + 1] - begin, max_prefill - p.tokens);
+            if (n <= 0) continue;
+            SeqSpan q;
+            q.slab = static_cast<unsigned char*>(st.k_cache[b]), q.history = st.history_lengths[b] + done[b], q.n = n, q.tok0 = p.tokens, q.live = 1;
+            tok.insert(tok.end(), st.input_ids + begin, st.input_ids + begin + n);
+            want_seq_begin.push_back((int)wanted.size());
+            const int* lo = std::lower_bound(st.want, st.want + st.want_count, begin);
+            const int* hi = std::lower_bound(st.want, st.want + st.want_count, begin + n);
+            logit_rows.push_back(st.logits_out + (size_t)(lo - st.want) * V);
+            for (; lo < hi; ++lo) wanted.push_back(*lo - begin + p.tokens);
+            if (st.residual_out) res_rows.push_back(st.residual_out + (size_t)begin * W);
+            sp.push_back(q);
+            p.tokens += n;
+            p.max_n = std::max(p.max_n, n);
+            done[b] += n;
+        }
+        want_seq_begin.push_back((int)wanted.size());
+        left -= p.tokens;
+        p.batch       = (int)sp.size();
+        p.need_output = !wanted.empty() || st.residual_out != nullptr;
+        p.host_spans  = sp.data();
+        if (st.residual_out) p.residual_rows = res_rows.data(), p.residual_layer_stride = (size_t)total * W;
+        if (cudaMemcpyAsync(spans, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess
+            || cudaMemcpyAsync(ids, tok.data(), tok.size() * 4, cudaMemcpyHostToDevice, s) != cudaSuccess
+            || (!wanted.empty() && cudaMemcpyAsync(want, wanted.data(), wanted.size() * 4, cudaMemcpyHostToDevice, s) != cudaSuccess)) {
+            return TM_ERR_CUDA;
+        }
+        int rc = run_layers(p, s);
+        // ---- logits of the wanted rows: per span, so that they land where the caller's order puts them
+        for (int b = 0; b < p.batch && rc == TM_OK; ++b) {
+            for (int w = want_seq_begin[b]; w < want_seq_begin[b + 1] && rc == TM_OK; w += kWantRows) {
+                const int n = std::min(kWantRows, want_seq_begin[b + 1] - w);
+                if (f32) {
+                    gather_rows_kernel<float><<<n, 128, 0, s>>>(static_cast<float*>(want_xb), want_ssq, static_cast<const float*>(xb), ssq, want + w, x_ld);
+                }
+                else {
+                    using E = __nv_bfloat16;
+                    gather_rows_kernel<E><<<n, 128, 0, s>>>(static_cast<E*>(want_xb), want_ssq, static_cast<const E*>(xb), ssq, want + w, x_ld);
+                }
+                ++h->launches;
+                DenseGemm g;
+                g.w = head, g.ldw = x_ld, g.x = want_xb, g.ldx = x_ld, g.tokens = n, g.n_out = cfg.vocab, g.k = cfg.width;
+                g.ep.kind = DenseKind::kF32, g.ep.out = logit_rows[b] + (size_t)(w - want_seq_begin[b]) * V, g.ep.out_ld = cfg.vocab;
+                g.ep.ssq = want_ssq, g.ep.ssq_parts = 1, g.ep.ssq_stride = kWantRows, g.ep.inv_width = 1.f / (float)W, g.ep.eps = (float)cfg.norm_eps;
+                g.ep.gain = final_gain;
+                rc        = dense_gemm(h, g, f32, s, false);
+            }
+        }
+        if (rc != TM_OK) return rc;
+    }
+    return TM_OK;
+}
+
+int tm_decoder::step(const tm_llama_decode_state& st, cudaStream_t s, unsigned long long* launches)
+{
+    const unsigned long long before = h->launches;
+    const int                B      = st.batch_size;
+    step_spans_kernel<<<(B + 127) / 128, 128, 0, s>>>(st, picked, ids, inactive, spans, cfg.vocab, session_len);
+    if (cudaPeekAtLastError() != cudaSuccess) return TM_ERR_CUDA;
+    Pass p;
+    p.batch = B, p.tokens = B, p.max_n = 1, p.decode = true, p.fold = !f32 && h->fold_norm, p.pdl = h->pdl != 0;
+    int rc = run_layers(p, s);
+    if (rc != TM_OK) return rc;
+    float*    out = st.logits_out ? st.logits_out : logits;
+    DenseGemm g;
+    g.w = head, g.ldw = x_ld, g.x = xb, g.ldx = x_ld, g.tokens = B, g.n_out = cfg.vocab, g.k = cfg.width;
+    g.ep.kind = DenseKind::kF32, g.ep.out = out, g.ep.out_ld = cfg.vocab;
+    g.ep.ssq = ssq, g.ep.ssq_parts = p.fold ? (cfg.width + kDenseTile - 1) / kDenseTile : 1, g.ep.ssq_stride = ssq_stride;
+    g.ep.inv_width = 1.f / (float)cfg.width, g.ep.eps = (float)cfg.norm_eps, g.ep.gain = final_gain;
+    if ((rc = dense_gemm(h, g, f32, s, p.pdl)) != TM_OK) return rc;
+    if (step_argmax(out, picked, st.output_ids, st.step, inactive, B, cfg.vocab, 1, st.max_steps, s) != cudaSuccess
+        || step_advance(st.step, st.sequence_lengths, inactive, B, s) != cudaSuccess) {
+        return TM_ERR_CUDA;
+    }
+    *launches = h->launches - before + 3;
+    return TM_OK;
+}
+
+int tm_decoder::decode(const tm_llama_decode_state& st, int n_steps, bool use_graph, cudaStream_t s)
+{
+    if (st.hidden_out) return TM_ERR_UNSUPPORTED;
+    return graph.run(h, st, n_steps, use_graph, s, &launches_of_last, [&](unsigned long long* n) { return step(st, s, n); });
+}
+
+// ---------------------------------------------------------------------------------------------------- mechanisms alone
+namespace {
+
+// spans of a call on the device, freed behind the work on the stream
+struct DeviceSpans {
+    SeqSpan*     d = nullptr;
+    cudaStream_t s;
+    MixerCall    c;
+    int          rc = TM_OK;
+
+    DeviceSpans(const tm_mixer_call& call, cudaStream_t stream): s(stream)
+    {
+        if (!call.proj || !call.out || call.batch <= 0 || !call.history || !call.n || !call.slabs
+            || (call.dtype != TM_DTYPE_BF16 && call.dtype != TM_DTYPE_F32)) {
+            rc = TM_ERR_INVALID_ARG;
+            return;
+        }
+        std::vector<SeqSpan> sp(call.batch);
+        c.max_n = 0;
+        for (int b = 0; b < call.batch; ++b) {
+            if (!call.slabs[b] || call.history[b] < 0 || call.n[b] < 0 || (call.decode && call.n[b] != 1)) rc = TM_ERR_INVALID_ARG;
+            sp[b].slab = static_cast<unsigned char*>(call.slabs[b]), sp[b].history = call.history[b], sp[b].n = call.n[b];
+            sp[b].tok0 = c.tokens, sp[b].live = 1;
+            c.tokens += call.n[b];
+            c.max_n       = std::max(c.max_n, call.n[b]);
+            c.max_context = std::max(c.max_context, call.history[b] + call.n[b]);
+        }
+        if (rc == TM_OK && c.tokens == 0) rc = TM_ERR_INVALID_ARG;
+        if (rc != TM_OK) return;
+        if (cudaMallocAsync((void**)&d, sp.size() * sizeof(SeqSpan), s) != cudaSuccess
+            || cudaMemcpyAsync(d, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess) {
+            rc = TM_ERR_CUDA;
+        }
+        c.proj = call.proj, c.proj_ld = call.proj_ld, c.out = call.out, c.out_ld = call.out_ld, c.spans = d, c.batch = call.batch;
+        c.f32 = call.dtype == TM_DTYPE_F32;
+    }
+    ~DeviceSpans()
+    {
+        if (d) cudaFreeAsync(d, s);
+    }
+};
+
+}  // namespace
+
+extern "C" int tm_window_attention(tm_handle* h, const tm_window_attention_params* q, const tm_mixer_call* call, void* stream)
+{
+    if (!h || !q || !call) return TM_ERR_INVALID_ARG;
+    DeviceSpans sp(*call, (cudaStream_t)stream);
+    if (sp.rc != TM_OK) return sp.rc;
+    WindowAttention a;
+    a.heads = q->heads, a.kv_heads = q->kv_heads, a.dim = q->dim, a.vdim = q->vdim, a.rot_dims = q->rot_dims, a.inv_freq = q->inv_freq;
+    a.scale = q->scale, a.softcap = q->softcap, a.window = q->window, a.pool = q->pool, a.ring = q->ring, a.pool_rows = q->pool_rows;
+    a.k_off = q->k_off, a.v_off = q->v_off, a.pk_off = q->pooled_k_off, a.pv_off = q->pooled_v_off;
+    a.q_col = q->q_col, a.k_col = q->k_col, a.v_col = q->v_col, a.g_col = q->g_col;
+    for (int b = 0; b < call->batch; ++b) {
+        // everything a query of the call may see has to be in the ring and in the pooled rows
+        const int end = call->history[b] + call->n[b], need = a.window > 0 ? std::min(end, std::max(a.window, a.pool) + call->n[b]) : end;
+        if (need > a.ring || (a.pool > 0 && end / a.pool > a.pool_rows)) return TM_ERR_INVALID_ARG;
+    }
+    return call->decode ? window_attention_decode(h, a, sp.c, sp.s) : window_attention_prefill(h, a, sp.c, sp.s);
+}
+
+extern "C" int tm_delta_rule(tm_handle* h, const tm_delta_rule_params* q, const tm_mixer_call* call, void* stream)
+{
+    if (!h || !q || !call || !q->w2 || !q->w0 || !q->a_bias || !q->norm) return TM_ERR_INVALID_ARG;
+    DeviceSpans sp(*call, (cudaStream_t)stream);
+    if (sp.rc != TM_OK) return sp.rc;
+    DeltaRule d;
+    d.heads = q->heads, d.dim = q->dim, d.rank = q->rank, d.w2 = q->w2, d.w2_ld = q->w2_ld, d.w0 = q->w0, d.a_bias = q->a_bias, d.norm = q->norm;
+    d.norm_eps = q->norm_eps, d.unit_eps = q->unit_eps, d.decay_scale = q->decay_scale, d.state_off = q->state_off;
+    d.r_col = q->r_col, d.k_col = q->k_col, d.v_col = q->v_col, d.a_col = q->a_col, d.g_col = q->g_col, d.w1_col = q->w1_col;
+    if (call->decode) return delta_rule_decode(h, d, sp.c, sp.s);
+    float*       scratch = nullptr;
+    const size_t n       = (size_t)sp.c.tokens * d.heads * d.dim;
+    if (cudaMallocAsync((void**)&scratch, 2 * n * sizeof(float), sp.s) != cudaSuccess) return TM_ERR_CUDA;
+    const int rc = delta_rule_prefill(h, d, sp.c, scratch, scratch + n, sp.s);
+    cudaFreeAsync(scratch, sp.s);
+    return rc;
+}

@@ -1,0 +1,117 @@
+// Config-driven decoder: a model whose layer list, mixers and sizes come from config.json.  Each layer is parallel,
+// x <- x + mixer(h) + ff(h) with h = norm(x), which makes it two GEMMs around a mixer:
+//   input GEMM    all projections of the mixer and the gated pair of the feed-forward, stacked in one weight; the norm is
+//                 one number per token (its gain is one number), so it scales the rows of the product
+//   mixer         window attention or delta rule (mixers.h), from and to the same buffers
+//   output GEMM   [mixer's output weight | feed-forward's down weight] over the concatenated inputs, added to the residual
+// Slab of a sequence: per attention layer the token rings of keys and values and the pooled rows, per recurrent layer the
+// fp32 state, each on a 256-byte boundary.
+#pragma once
+#include "gemm_dense.h"
+#include "json.h"
+#include "mixers.h"
+#include "model.h"
+
+#include <string>
+#include <vector>
+
+namespace tmb {
+
+enum class MixerType : int { kAttention, kGeneralDelta };
+
+struct MixerSpec {
+    MixerType type  = MixerType::kAttention;
+    int       heads = 0, dim = 0;
+    // attention
+    int    kv_heads = 0, vdim = 0;
+    int    rot_dims = 0;
+    double rot_base = 10000.0, rot_factor = 1.0;
+    double scale = 1.0, softcap = 0.0;
+    int    window = 0, pool = 0;
+    // general delta: rank of the decay's low-rank projection (given by the shape of its tensors)
+    int rank = 0;
+
+    int out_width() const { return heads * (type == MixerType::kAttention ? vdim : dim); }
+};
+
+struct LayerSpec {
+    MixerSpec mixer;
+    int       ff = 0;  // 0: no feed-forward
+};
+
+struct DecoderConfig {
+    std::string            architecture;
+    int                    vocab = 0, width = 0;
+    double                 norm_eps = 0, embedding_scale = 1.0;
+    std::vector<LayerSpec> layers;
+};
+
+// config.json of the architecture "Rumazen" -> DecoderConfig; false with a reason when something is missing or impossible
+bool read_rumazen_config(const Json& j, DecoderConfig* c, std::string* why);
+
+struct DecoderLayer {
+    LayerSpec       spec;
+    WindowAttention attention;
+    DeltaRule       delta;
+    int             mixer_cols = 0;  // projection columns, a multiple of kDenseTile
+    int             in_rows    = 0;  // mixer_cols + 2 ff, rounded up to kDenseTile
+    int             mix_pad    = 0;  // columns of the output GEMM's input that belong to the mixer
+    int             out_k      = 0;  // all columns of it
+    int             tanh_lo = 0, tanh_hi = 0;
+    void *          w_in = nullptr, *w_out = nullptr, *w2 = nullptr;  // element type
+    float *         gain = nullptr, *w0 = nullptr, *a_bias = nullptr, *norm = nullptr, *inv_freq = nullptr;
+};
+
+// Where a checkpoint tensor goes: rows x cols at `dst`, row r at dst + r * row_stride (elements)
+struct WeightTarget {
+    std::string name;
+    int64_t     rows = 0, cols = 0;
+    bool        scalar = false, vector = false;  // shape [] / [cols]
+    void*       dst = nullptr;
+    int64_t     row_stride = 0;
+    bool        f32 = false;      // kept in fp32 whatever the element type
+    float       init_std = 0.f, init_mean = 0.f;  // random initialisation
+};
+
+}  // namespace tmb
+
+struct tm_decoder final : tm_model {
+    tmb::DecoderConfig             cfg;
+    bool                           f32 = false;
+    int                            max_prefill = 0;  // tokens of one pass through the layers
+    std::vector<tmb::DecoderLayer> layers;
+    std::vector<tmb::WeightTarget> targets;
+    size_t                         slab = 0;
+    int                            x_ld = 0, proj_ld = 0, y_ld = 0;
+
+    std::vector<void*> owned;
+    void *             embed = nullptr, *head = nullptr;
+    float*             final_gain = nullptr;
+    // activations of one pass
+    float *       x = nullptr, *ssq = nullptr, *decay_pre = nullptr, *delta_o = nullptr, *logits = nullptr;
+    void *        xb = nullptr, *proj = nullptr, *y = nullptr, *want_xb = nullptr;
+    float*        want_ssq = nullptr;
+    int           ssq_stride = 0;
+    int *         ids = nullptr, *want = nullptr, *picked = nullptr;
+    unsigned char* inactive = nullptr;
+    tmb::SeqSpan* spans = nullptr;
+    tmb::StepGraph graph;
+    unsigned long long launches_of_last = 0;
+
+    ~tm_decoder() override;
+    int    init(tm_handle* handle, const tmb::DecoderConfig& c, const tm_model_options& opt);
+    int    load(const std::string& safetensors, std::string* why);
+    int    random_weights(unsigned long long seed);
+    int    prefill(const tm_model_prefill_state& st, cudaStream_t s) override;
+    int    decode(const tm_llama_decode_state& st, int n_steps, bool use_graph, cudaStream_t s) override;
+    int    new_cache(tm_cache_manager** out, size_t max_entry_count, size_t chunk_size) const override;
+    bool   can_rewind() const override { return false; }
+    size_t slab_bytes() const override { return slab; }
+    unsigned long long last_launches() const override { return launches_of_last; }
+
+private:
+    struct Pass;
+    int  run_layers(const Pass& p, cudaStream_t s);
+    int  step(const tm_llama_decode_state& st, cudaStream_t s, unsigned long long* launches);
+    bool alloc(void** p, size_t bytes);
+};

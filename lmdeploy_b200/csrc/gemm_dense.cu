@@ -1,0 +1,525 @@
+// Dense GEMM of the config-driven decoder (gemm_dense.h): bf16 on the tcgen05 tensor core, fp32 on the CUDA cores.
+//
+// dense_tc_kernel: 128 output columns (UMMA M) x up to 256 tokens (UMMA N) per tile, persistent, one CTA per SM.
+//   warp 0    one lane feeds a ring of stages with TMA: a [128 weight rows x 64 k] box and a [tokens x 64 k] box,
+//             128-byte swizzle (every CTA loads for itself); weight boxes start before the kernel ahead is complete
+//   warp 1    allocates TMEM (two accumulators, so that one tile's epilogue overlaps the next tile's products); one lane
+//             issues four K16 MMAs per stage and commits the stage back to the loader
+//   warps 2-5 epilogue: lane = output column, so that every token's 32 columns leave in one contiguous store
+// With fewer tiles than SMs (a decode step) the k range of every tile is cut in `splits` parts: each part publishes its
+// fp32 tile in scratch, the last one to arrive adds them up in part order (nobody waits, the sum does not depend on the
+// order of arrival) and runs the epilogue.
+// Every wait is bounded: a barrier that does not complete sets a status bit, the CTA drains its copies and leaves.
+#include "gemm_dense.h"
+#include "numeric.cuh"
+#include "tcgen05.cuh"
+#include "tm_b200.h"
+
+namespace tmb {
+namespace {
+
+constexpr int kKBlock    = 64;  // k per stage: 128 bytes per row, the swizzle span
+constexpr int kThreads   = 6 * 32;
+constexpr int kMaxStages = 12;
+constexpr int kMaxTokens = 256;  // tokens of one tile
+constexpr int kEpiBar    = 1;    // named barrier of the epilogue warps
+
+struct DenseShared {
+    uint64_t full[kMaxStages], empty[kMaxStages];
+    uint64_t acc_full[2], acc_empty[2];
+    uint32_t tmem_base;
+    int      dead;
+    int      last;
+    int      pad;
+    float    scale[kMaxTokens];
+    float    red[4][kMaxTokens];
+};
+
+struct DenseTcParams {
+    int           tokens, n_out, k_blocks;
+    int           token_tile, token_tiles, column_tiles, splits, units;
+    int           stages, tmem_columns;
+    float*        scratch;
+    int*          tickets;
+    unsigned*     status;
+    long long     max_wait;
+    DenseEpilogue ep;
+};
+
+// What happens to 16 consecutive tokens of one output column (lane = column); `live` = tokens of the 16 that exist
+__device__ __forceinline__ void epilogue16(const DenseEpilogue& ep, const float (&y)[16], int t0, int live, int n, int n_out, float (&sq)[16])
+{
+    using E        = __nv_bfloat16;
+    const bool col = n < n_out;
+    if (ep.kind == DenseKind::kResidual) {
+        float r[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) r[i] = i < live && col ? ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] : 0.f;
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            const bool on = i < live && col;
+            r[i]          = on ? r[i] + y[i] : 0.f;
+            sq[i]         = r[i] * r[i];
+            if (on) ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] = r[i];
+            if (on && ep.cast) static_cast<E*>(ep.cast)[(size_t)(t0 + i) * ep.cast_ld + n] = from_f32<E>(r[i]);
+        }
+        return;
+    }
+    if (ep.kind == DenseKind::kF32) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            if (i < live && col) static_cast<float*>(ep.out)[(size_t)(t0 + i) * ep.out_ld + n] = y[i];
+        }
+        return;
+    }
+    if (ep.kind == DenseKind::kInput && n >= ep.split) {
+        // even lanes hold gates, odd lanes the matching ups; of two tokens the even lane finishes one, the odd lane the other
+        const bool odd = n & 1;
+        E*         dst = static_cast<E*>(ep.act) + ((n - ep.split) >> 1);
+#pragma unroll
+        for (int i = 0; i < 16; i += 2) {
+            const float other = __shfl_xor_sync(0xffffffffu, odd ? y[i] : y[i + 1], 1);
+            const float gate = odd ? other : y[i], up = odd ? y[i + 1] : other;
+            const int   t = i + (odd ? 1 : 0);
+            if (t < live && col) dst[(size_t)(t0 + t) * ep.act_ld] = from_f32<E>(gelu_tanh_f32<true>(gate) * up);
+        }
+        return;
+    }
+    const bool th = ep.kind == DenseKind::kInput && n >= ep.tanh_lo && n < ep.tanh_hi;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+        if (i < live && col) static_cast<E*>(ep.out)[(size_t)(t0 + i) * ep.out_ld + n] = from_f32<E>(th ? tanhf(y[i]) : y[i]);
+    }
+}
+
+__global__ void __launch_bounds__(kThreads, 1)
+dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map)
+{
+    extern __shared__ unsigned char smem_dyn[];
+    const uint32_t raw  = smem_u32(smem_dyn);
+    const uint32_t base = (raw + 1023u) & ~1023u;  // operand tiles on 1024-byte boundaries (the swizzle is a function of the address)
+    const int      NT      = p.token_tile;
+    const uint32_t w_bytes = kDenseTile * 128;
+    const uint32_t stage_b = w_bytes + (uint32_t)NT * 128;
+    const int      ST      = p.stages;
+    DenseShared*   sh      = reinterpret_cast<DenseShared*>(smem_dyn + (base - raw) + (size_t)ST * stage_b);
+    const int      tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+
+    if (tid == 0) {
+        for (int s = 0; s < kMaxStages; ++s) {
+            mbar_init(&sh->full[s], 1);
+            mbar_init(&sh->empty[s], 1);
+        }
+        for (int a = 0; a < 2; ++a) {
+            mbar_init(&sh->acc_full[a], 1);
+            mbar_init(&sh->acc_empty[a], 4);
+        }
+        sh->dead = 0;
+        fence_mbar_init();
+    }
+    if (warp == 1) tmem_alloc(&sh->tmem_base, p.tmem_columns);
+    tcgen05_before_sync();
+    __syncthreads();
+    tcgen05_after_sync();
+    const uint32_t tmem = sh->tmem_base;
+
+    // unit u -> (column tile, token tile, part of the k range); token tiles vary fastest among tiles, so that the CTAs of
+    // a wave share weight tiles and activations in the L2
+    auto unit_of = [&](int u, int& ct, int& tt, int& kb0, int& kb1, int& part) {
+        const int tile = u / p.splits;
+        part           = u - tile * p.splits;
+        ct             = tile / p.token_tiles;
+        tt             = tile - ct * p.token_tiles;
+        kb0            = (int)((long long)part * p.k_blocks / p.splits);
+        kb1            = (int)((long long)(part + 1) * p.k_blocks / p.splits);
+    };
+
+    if (warp == 0) {
+        // ===================================================================================== loader
+        if (lane == 0) {
+            int  issued = 0;
+            bool ok = true, waited = false;
+            auto load_w = [&](int kb, int ct, int s) {
+                mbar_arrive_expect_tx(&sh->full[s], stage_b);
+                tma_load_2d(base + s * stage_b, &w_map, kb * kKBlock, ct * kDenseTile, &sh->full[s]);
+            };
+            auto load_x = [&](int kb, int tt, int s) { tma_load_2d(base + s * stage_b + w_bytes, &x_map, kb * kKBlock, tt * NT, &sh->full[s]); };
+            for (int u = blockIdx.x; u < p.units && ok; u += gridDim.x) {
+                int ct, tt, kb0, kb1, part;
+                unit_of(u, ct, tt, kb0, kb1, part);
+                int kb = kb0;
+                if (!waited) {
+                    // weights are written by no kernel: the first boxes go out before the kernel ahead is complete
+                    const int pre = min(ST, kb1 - kb0);
+                    for (int i = 0; i < pre; ++i) load_w(kb0 + i, ct, i);
+                    pdl_wait();
+                    pdl_launch_dependents();
+                    waited = true;
+                    for (int i = 0; i < pre; ++i) load_x(kb0 + i, tt, i);
+                    issued = pre;
+                    kb += pre;
+                }
+                for (; kb < kb1; ++kb, ++issued) {
+                    const int s = issued % ST;
+                    if (issued >= ST && !mbar_wait(&sh->empty[s], ((issued / ST) - 1) & 1, p.max_wait)) {
+                        atomicOr(p.status, kStatusGemmPipeWait);
+                        *(volatile int*)&sh->dead = 1;
+                        ok = false;
+                        break;
+                    }
+                    load_w(kb, ct, s);
+                    load_x(kb, tt, s);
+                }
+            }
+            if (!waited) {
+                pdl_wait();
+                pdl_launch_dependents();
+            }
+            if (!ok) {
+                // the CTA leaves early: not before its own copies have landed
+                for (int i = max(0, issued - ST); i < issued; ++i) mbar_wait(&sh->full[i % ST], (i / ST) & 1, p.max_wait);
+            }
+        }
+        else {
+            pdl_wait();
+            pdl_launch_dependents();
+        }
+    }
+    else if (warp == 1) {
+        // ===================================================================================== MMA issuer
+        pdl_wait();
+        pdl_launch_dependents();
+        if (lane == 0) {
+            const uint32_t idesc = umma_idesc_bf16(kDenseTile, NT);
+            int            it = 0, local = 0;
+            bool           ok = true;
+            for (int u = blockIdx.x; u < p.units && ok; u += gridDim.x, ++local) {
+                int ct, tt, kb0, kb1, part;
+                unit_of(u, ct, tt, kb0, kb1, part);
+                const int a = local & 1;
+                if (local >= 2 && !mbar_wait(&sh->acc_empty[a], ((local >> 1) - 1) & 1, p.max_wait)) ok = false;
+                tcgen05_after_sync();
+                for (int kb = kb0; kb < kb1 && ok; ++kb, ++it) {
+                    const int s = it % ST;
+                    if (!mbar_wait(&sh->full[s], (it / ST) & 1, p.max_wait)) {
+                        ok = false;
+                        break;
+                    }
+                    tcgen05_after_sync();
+                    const uint64_t da = umma_desc_k(base + s * stage_b), db = umma_desc_k(base + s * stage_b + w_bytes);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        umma_f16_ss(tmem + a * NT, da + (uint64_t)(2 * j), db + (uint64_t)(2 * j), idesc, (kb > kb0 || j) ? 1u : 0u);
+                    }
+                    umma_commit(&sh->empty[s]);
+                }
+                if (!ok) {
+                    atomicOr(p.status, kStatusGemmPipeWait);
+                    *(volatile int*)&sh->dead = 1;
+                }
+                umma_commit(&sh->acc_full[a]);  // arrives when everything issued so far is complete (also on the give-up path)
+            }
+        }
+    }
+    else {
+        // ===================================================================================== epilogue
+        pdl_wait();
+        pdl_launch_dependents();
+        const int q    = warp & 3;  // the TMEM lane quarter this warp may read
+        const int etid = tid - 64;
+        const int col  = q * 32 + lane;
+        int       local = 0, scaled_tile = -1;
+        bool      ok = true;
+        for (int u = blockIdx.x; u < p.units && ok; u += gridDim.x, ++local) {
+            int ct, tt, kb0, kb1, part;
+            unit_of(u, ct, tt, kb0, kb1, part);
+            const int a    = local & 1;
+            const int t0   = tt * NT;
+            const int rows = min(NT, p.tokens - t0);
+            const int n    = ct * kDenseTile + col;
+            if (p.ep.ssq && scaled_tile != tt) {
+                // 1 / rms of every token of the tile, once per token tile
+                named_bar_sync(kEpiBar, 128);
+                for (int t = etid; t < rows; t += 128) {
+                    float ss = 0.f;
+                    for (int i = 0; i < p.ep.ssq_parts; ++i) ss += p.ep.ssq[(size_t)i * p.ep.ssq_stride + t0 + t];
+                    sh->scale[t] = *p.ep.gain / sqrtf(ss * p.ep.inv_width + p.ep.eps);
+                }
+                named_bar_sync(kEpiBar, 128);
+                scaled_tile = tt;
+            }
+            int okw = 1;
+            if (lane == 0) okw = mbar_wait(&sh->acc_full[a], (local >> 1) & 1, p.max_wait) ? 1 : 0;
+            okw = __shfl_sync(0xffffffffu, okw, 0);
+            if (!okw || *(volatile int*)&sh->dead) {
+                if (lane == 0) {
+                    if (!okw) atomicOr(p.status, kStatusGemmTmemWait);
+                    *(volatile int*)&sh->dead = 1;
+                }
+            }
+            // all four warps take the same way out (the barriers below are theirs together)
+            named_bar_sync(kEpiBar, 128);
+            if (*(volatile int*)&sh->dead) {
+                ok = false;
+                break;
+            }
+            tcgen05_after_sync();
+            const uint32_t acc    = tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * NT);
+            bool           finish = true;
+            float*         slots  = nullptr;
+            if (p.splits > 1) {
+                slots       = p.scratch + (size_t)(u - part) * NT * kDenseTile;
+                float* mine = slots + (size_t)part * NT * kDenseTile;
+                for (int c0 = 0; c0 < rows; c0 += 16) {
+                    float v[16];
+                    tmem_load16(acc + c0, v);
+#pragma unroll
+                    for (int i = 0; i < 16; ++i) {
+                        if (c0 + i < rows) __stcg(mine + (size_t)(c0 + i) * kDenseTile + col, v[i]);
+                    }
+                }
+                __threadfence();
+                named_bar_sync(kEpiBar, 128);
+                if (etid == 0) {
+                    int*      ticket = p.tickets + (u - part) / p.splits;
+                    const int before = atomicAdd(ticket, 1);
+                    sh->last         = before == p.splits - 1;
+                    if (sh->last) *ticket = 0;
+                }
+                named_bar_sync(kEpiBar, 128);
+                finish = *(volatile int*)&sh->last != 0;
+                if (finish) __threadfence();
+            }
+            if (finish) {
+                const bool sums = p.ep.kind == DenseKind::kResidual && p.ep.ssq_out;
+                for (int c0 = 0; c0 < rows; c0 += 16) {
+                    float     v[16], sq[16];
+                    const int live = min(16, rows - c0);
+                    if (p.splits > 1) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) v[i] = 0.f;
+                        for (int s = 0; s < p.splits; ++s) {
+                            const float* src = slots + ((size_t)s * NT + c0) * kDenseTile + col;
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) {
+                                if (i < live) v[i] += __ldcg(src + (size_t)i * kDenseTile);
+                            }
+                        }
+                    }
+                    else {
+                        tmem_load16(acc + c0, v);
+                    }
+                    if (p.ep.ssq) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) v[i] *= i < live ? sh->scale[c0 + i] : 0.f;
+                    }
+                    epilogue16(p.ep, v, t0 + c0, live, n, p.n_out, sq);
+                    if (sums) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) {
+                            const float s = warp_sum(sq[i]);
+                            if (lane == i) sh->red[q][c0 + i] = s;
+                        }
+                    }
+                }
+                if (sums) {
+                    named_bar_sync(kEpiBar, 128);
+                    for (int t = etid; t < rows; t += 128) {
+                        p.ep.ssq_out[(size_t)ct * p.ep.ssq_out_stride + t0 + t] = (sh->red[0][t] + sh->red[1][t]) + (sh->red[2][t] + sh->red[3][t]);
+                    }
+                    named_bar_sync(kEpiBar, 128);
+                }
+            }
+            tcgen05_before_sync();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&sh->acc_empty[a]);
+        }
+    }
+
+    tcgen05_before_sync();
+    __syncthreads();
+    if (warp == 1) tmem_free(tmem, p.tmem_columns);
+}
+
+// ------------------------------------------------------------------------------------------------ fp32
+constexpr int kSimtTile = 64, kSimtK = 16;
+
+__global__ void __launch_bounds__(256) dense_f32_kernel(DenseGemm g)
+{
+    __shared__ float xs[kSimtK][kSimtTile + 4], ws[kSimtK][kSimtTile + 4];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int    t0 = blockIdx.y * kSimtTile, n0 = blockIdx.x * kSimtTile;
+    const int    tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const float* x = static_cast<const float*>(g.x);
+    const float* w = static_cast<const float*>(g.w);
+    float        acc[4][4] = {};
+    for (int k0 = 0; k0 < g.k; k0 += kSimtK) {
+        for (int i = threadIdx.x; i < kSimtTile * kSimtK; i += 256) {
+            const int r = i / kSimtK, kk = i % kSimtK, k = k0 + kk;
+            xs[kk][r] = t0 + r < g.tokens && k < g.k ? x[(size_t)(t0 + r) * g.ldx + k] : 0.f;
+            ws[kk][r] = n0 + r < g.n_out && k < g.k ? w[(size_t)(n0 + r) * g.ldw + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int kk = 0; kk < kSimtK; ++kk) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[i] = xs[kk][ty * 4 + i], b[i] = ws[kk][tx * 4 + i];
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    const DenseEpilogue& ep = g.ep;
+    for (int i = 0; i < 4; ++i) {
+        const int t = t0 + ty * 4 + i;
+        if (t >= g.tokens) continue;
+        float scale = 1.f;
+        if (ep.ssq) {
+            float ss = 0.f;
+            for (int p = 0; p < ep.ssq_parts; ++p) ss += ep.ssq[(size_t)p * ep.ssq_stride + t];
+            scale = *ep.gain / sqrtf(ss * ep.inv_width + ep.eps);
+        }
+        for (int j = 0; j < 4; ++j) {
+            const int n = n0 + tx * 4 + j;
+            if (n >= g.n_out) continue;
+            const float y = acc[i][j] * scale;
+            if (ep.kind == DenseKind::kResidual) {
+                ep.residual[(size_t)t * ep.residual_ld + n] += y;
+            }
+            else if (ep.kind == DenseKind::kInput && n >= ep.split) {
+                if ((j & 1) == 0) {
+                    const float up = n + 1 < g.n_out ? acc[i][j + 1] * scale : 0.f;
+                    static_cast<float*>(ep.act)[(size_t)t * ep.act_ld + ((n - ep.split) >> 1)] = gelu_tanh_f32<false>(y) * up;
+                }
+            }
+            else {
+                const bool th = ep.kind == DenseKind::kInput && n >= ep.tanh_lo && n < ep.tanh_hi;
+                static_cast<float*>(ep.out)[(size_t)t * ep.out_ld + n] = th ? tanhf(y) : y;
+            }
+        }
+    }
+}
+
+using EncodeTiled = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                 const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+EncodeTiled lookup_encode_tiled()
+{
+    void*                           fn = nullptr;
+    cudaDriverEntryPointQueryResult q{};
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) {
+        return nullptr;
+    }
+    return reinterpret_cast<EncodeTiled>(fn);
+}
+
+bool encode_rows(EncodeTiled encode, CUtensorMap* map, const void* ptr, int rows, int k, int ld, int box_rows)
+{
+    const cuuint64_t dims[2]    = {(cuuint64_t)k, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2]     = {(cuuint32_t)kKBlock, (cuuint32_t)box_rows};
+    const cuuint32_t estr[2]    = {1u, 1u};
+    return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE)
+           == CUDA_SUCCESS;
+}
+
+cudaError_t dense_prepare(int max_smem)
+{
+    return cudaFuncSetAttribute(dense_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+}
+const KernelPreparation g_prepare(dense_prepare);
+
+// parts of the k range per tile: as many as fill the SMs evenly, each of at least four k blocks
+int choose_splits(int tiles, int k_blocks, int sms, size_t tile_bytes, size_t scratch_bytes)
+{
+    if (tiles >= 4 * sms) return 1;
+    int    best      = 1;
+    double best_cost = 1e30;
+    for (int s = 1; s <= 16 && (s == 1 || k_blocks / s >= 4); ++s) {
+        if (s > 1 && (size_t)tiles * s * tile_bytes > scratch_bytes) break;
+        const int    waves = (tiles * s + sms - 1) / sms;
+        const double cost  = waves * ((double)((k_blocks + s - 1) / s) + 3.0) + (s > 1 ? 4.0 + 0.5 * s : 0.0);
+        if (cost < best_cost - 1e-9) best_cost = cost, best = s;
+    }
+    return best;
+}
+
+int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
+{
+    static const EncodeTiled encode = lookup_encode_tiled();
+    if (!encode) return TM_ERR_CUDA;
+    if (g.ldw % 8 || g.ldx % 8 || (reinterpret_cast<uintptr_t>(g.w) & 15) || (reinterpret_cast<uintptr_t>(g.x) & 15)) return TM_ERR_INVALID_ARG;
+    if (g.ep.kind == DenseKind::kInput && g.ep.split % kDenseTile) return TM_ERR_INVALID_ARG;
+    DenseTcParams p{};
+    p.tokens       = g.tokens;
+    p.n_out        = g.n_out;
+    p.k_blocks     = (g.k + kKBlock - 1) / kKBlock;
+    p.token_tile   = g.tokens >= kMaxTokens ? kMaxTokens : (g.tokens + 15) / 16 * 16;
+    p.token_tiles  = (g.tokens + p.token_tile - 1) / p.token_tile;
+    p.column_tiles = (g.n_out + kDenseTile - 1) / kDenseTile;
+    p.tmem_columns = 32;
+    while (p.tmem_columns < 2 * p.token_tile) p.tmem_columns *= 2;
+    const size_t stage_b = (size_t)kDenseTile * 128 + (size_t)p.token_tile * 128;
+    p.stages             = (int)(((size_t)h->max_smem - 1024 - sizeof(DenseShared)) / stage_b);
+    if (p.stages > kMaxStages) p.stages = kMaxStages;
+    if (p.stages < 2) return TM_ERR_UNSUPPORTED;
+    const int tiles = p.column_tiles * p.token_tiles;
+    p.splits        = choose_splits(tiles, p.k_blocks, h->sm_count, (size_t)p.token_tile * kDenseTile * 4, h->scratch_bytes);
+    if (tiles > (int)h->counter_ints) p.splits = 1;
+    p.units    = tiles * p.splits;
+    p.scratch  = static_cast<float*>(h->scratch);
+    p.tickets  = h->counters;
+    p.status   = h->status;
+    p.max_wait = h->gemm_wait_cycles > 0 ? h->gemm_wait_cycles : kMaxWaitCycles;
+    p.ep       = g.ep;
+    CUtensorMap w_map, x_map;
+    if (!encode_rows(encode, &w_map, g.w, g.n_out, g.k, g.ldw, kDenseTile)) return TM_ERR_CUDA;
+    if (!encode_rows(encode, &x_map, g.x, g.tokens, g.k, g.ldx, p.token_tile)) return TM_ERR_CUDA;
+    const size_t smem = 1024 + (size_t)p.stages * stage_b + sizeof(DenseShared);
+    const dim3   grid(p.units < h->sm_count ? p.units : h->sm_count);
+    const cudaError_t e = launch_kernel(dense_tc_kernel, grid, dim3(kThreads), smem, st, pdl, p, w_map, x_map);
+    if (e != cudaSuccess) {
+        h->last_cuda_error = (int)e;
+        return TM_ERR_CUDA;
+    }
+    ++h->launches;
+    return TM_OK;
+}
+
+}  // namespace
+
+int dense_gemm(tm_handle* h, const DenseGemm& g, bool f32, cudaStream_t st, bool pdl)
+{
+    if (!g.w || !g.x || g.tokens <= 0 || g.n_out <= 0 || g.k <= 0 || g.ldw < g.k || g.ldx < g.k) return TM_ERR_INVALID_ARG;
+    if (!f32) return dense_tc(h, g, st, pdl);
+    if (g.ep.kind == DenseKind::kResidual && (g.ep.cast || g.ep.ssq_out)) return TM_ERR_UNSUPPORTED;
+    const dim3 grid((g.n_out + kSimtTile - 1) / kSimtTile, (g.tokens + kSimtTile - 1) / kSimtTile);
+    const cudaError_t e = launch_kernel(dense_f32_kernel, grid, dim3(256), 0, st, pdl, g);
+    if (e != cudaSuccess) {
+        h->last_cuda_error = (int)e;
+        return TM_ERR_CUDA;
+    }
+    ++h->launches;
+    return TM_OK;
+}
+
+}  // namespace tmb
+
+using namespace tmb;
+
+extern "C" int tm_gemm_dense(tm_handle* h, void* out, int out_ld, int out_f32, const void* x, int x_ld, const void* w, int w_ld, int tokens,
+                             int n_out, int k, int dtype, void* stream)
+{
+    if (!h || !out || out_ld < n_out || (dtype != TM_DTYPE_BF16 && dtype != TM_DTYPE_F32)) return TM_ERR_INVALID_ARG;
+    if (tokens == 0) return TM_OK;
+    DenseGemm g;
+    g.w = w, g.x = x, g.ldw = w_ld, g.ldx = x_ld, g.tokens = tokens, g.n_out = n_out, g.k = k;
+    g.ep.kind = out_f32 ? DenseKind::kF32 : DenseKind::kStore;
+    g.ep.out = out, g.ep.out_ld = out_ld;
+    return dense_gemm(h, g, dtype == TM_DTYPE_F32, (cudaStream_t)stream, false);
+}

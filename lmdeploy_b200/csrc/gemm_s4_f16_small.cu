@@ -23,6 +23,7 @@
 // tile is 8 and which has no split-K across CTAs.  The weight seen by the MMA differs from the
 // reference's fp16_rn((q - z) s) only by that one rounding (the products are exact in fp32 here).
 #include "common.cuh"
+#include "handle.h"
 #include "gemm_s4_f16.h"
 #include "tm_b200.h"
 
@@ -771,6 +772,7 @@ cudaError_t gemm_small_prepare(int max_smem)
     if (e != cudaSuccess) return e;
     return cudaFuncSetAttribute(gemm_s4_f16_small_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
 }
+static const KernelPreparation g_prepare(gemm_small_prepare);
 
 cudaError_t gemm_small_launch(const GemmSmallPlan& pl, GemmSmallParams p, cudaStream_t st, bool pdl)
 {

@@ -24,6 +24,7 @@
 // Replaces the large-n end of GemmS4F16::Run (src/turbomind/kernels/gemm_s_f16/gemm_s4_f16.cu:
 // 208-234; mma.sync tiles of gemm_template.h:338-444).
 #include "common.cuh"
+#include "handle.h"
 #include "gemm_s4_f16.h"
 
 #include <cuda.h>  // CUtensorMap (types only: the encoder is looked up through the runtime)
@@ -849,6 +850,7 @@ cudaError_t gemm_tc_prepare(int max_smem)
 {
     return cudaFuncSetAttribute(gemm_s4_f16_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
 }
+static const KernelPreparation g_prepare(gemm_tc_prepare);
 
 cudaError_t gemm_tc_launch(const GemmTcPlan& pl, GemmTcParams p, cudaStream_t st, bool pdl)
 {

@@ -36,10 +36,13 @@ struct tm_handle {
 
 namespace tmb {
 // lm_head.cu: logits[tokens][ld] (fp32) = x[tokens][hidden] . w[vocab][hidden]^T, fp16 operands, tcgen05
-cudaError_t lm_head_prepare(int max_smem);
-cudaError_t sampling_prepare(int max_smem);  // sampling.cu
 int lm_head_launch(float* logits, int ld, const __half* x, const __half* w, int tokens, int vocab, int hidden, unsigned* status,
                    long long max_wait_cycles, int max_smem, cudaStream_t st, bool pdl, unsigned long long* launches);
+// A kernel file's per-device attributes (shared-memory limits and the like), set whenever a handle is created: one static
+// object of this type per file, so that a handle knows no kernel by name.
+struct KernelPreparation {
+    explicit KernelPreparation(cudaError_t (*fn)(int max_smem));
+};
 // Set by the decode driver around its launches (per host thread): the kernel launches made through
 // the C ABI on this thread carry the programmatic-dependent-launch attribute.  Off for direct callers,
 // who may put any kernel in front of ours.

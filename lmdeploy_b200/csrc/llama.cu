@@ -5,6 +5,7 @@
 // LlamaFfnLayer::forward (LlamaFfnLayer.cc:66-116), LlamaV2::embeddingLookup / postDecodeEmbedding
 // (LlamaV2.cc:184-201, 312-372) of lmdeploy v0.0.9.
 #include "llama.h"
+#include "step_kernels.h"
 
 #include <cstdlib>
 #include <cstring>
@@ -76,15 +77,9 @@ __global__ void prepare_step_kernel(const int* step, const int* start_step, cons
         rope_table[(size_t)rank * 64 + threadIdx.x] = make_float2(cs, sn);
     }
     if (threadIdx.x != 0) return;
-    const int  s   = *step;
-    const bool off = s >= max_steps || (start_step != nullptr && s < start_step[b]);
-    inactive[b]    = off ? 1 : 0;
-    int id         = picked[b];
-    if (!off && forced_ids != nullptr) {
-        const int f = forced_ids[(size_t)s * B + b];
-        if (f >= 0) id = f;
-    }
-    ids_in[b] = min(max(id, 0), vocab - 1);
+    bool off    = false;
+    ids_in[b]   = step_input(step, start_step, forced_ids, picked, b, B, max_steps, vocab, &off);
+    inactive[b] = off ? 1 : 0;
     order[rank] = b;
     MmhaSeqDesc d;
     d.k_cache = k_ptrs[b], d.v_cache = v_ptrs[b], d.length = mine, d.seq = b, d.finished = off ? 1 : 0, d.reserved = 0;
@@ -97,71 +92,6 @@ __global__ void embedding_lookup_kernel(__half* x, const __half* table, const in
     const uint4* src = reinterpret_cast<const uint4*>(table + (size_t)ids[blockIdx.x] * hidden);
     uint4*       dst = reinterpret_cast<uint4*>(x + (size_t)blockIdx.x * hidden);
     for (int i = threadIdx.x; i < hidden / 8; i += blockDim.x) dst[i] = src[i];
-}
-
-// greedy pick over logits laid out [tp][B][vocab / tp]; ties go to the lowest token id
-__global__ void argmax_kernel(const float* logits, int* picked, int* output_ids, const int* step,
-                              const unsigned char* inactive, int B, int local_vocab, int tp, int max_steps)
-{
-    __shared__ float s_val[1024];
-    __shared__ int   s_idx[1024];
-    const int b    = blockIdx.x;
-    float     best = -INFINITY;
-    int       idx  = 0x7fffffff;
-    auto take = [&](float x, int i) {
-        if (x > best || (x == best && i < idx)) {
-            best = x;
-            idx  = i;
-        }
-    };
-    for (int r = 0; r < tp; ++r) {
-        const float* row = logits + ((size_t)r * B + b) * local_vocab;
-        if ((local_vocab & 3) == 0 && (reinterpret_cast<uintptr_t>(row) & 15) == 0) {
-            // four logits per load, several loads in flight per thread
-            const float4* row4 = reinterpret_cast<const float4*>(row);
-            for (int v = threadIdx.x; v < local_vocab / 4; v += blockDim.x) {
-                const float4 x = row4[v];
-                const int    i = r * local_vocab + 4 * v;
-                take(x.x, i);
-                take(x.y, i + 1);
-                take(x.z, i + 2);
-                take(x.w, i + 3);
-            }
-        }
-        else {
-            for (int v = threadIdx.x; v < local_vocab; v += blockDim.x) take(row[v], r * local_vocab + v);
-        }
-    }
-    s_val[threadIdx.x] = best;
-    s_idx[threadIdx.x] = idx;
-    __syncthreads();
-    for (int off = blockDim.x / 2; off > 0; off >>= 1) {
-        if (threadIdx.x < off) {
-            const float x = s_val[threadIdx.x + off];
-            const int   i = s_idx[threadIdx.x + off];
-            if (x > s_val[threadIdx.x] || (x == s_val[threadIdx.x] && i < s_idx[threadIdx.x])) {
-                s_val[threadIdx.x] = x;
-                s_idx[threadIdx.x] = i;
-            }
-        }
-        __syncthreads();
-    }
-    if (threadIdx.x == 0) {
-        const int s = *step;
-        if (!inactive[b]) {
-            picked[b] = s_idx[0];
-        }
-        if (s < max_steps) {
-            output_ids[(size_t)s * B + b] = inactive[b] ? -1 : s_idx[0];
-        }
-    }
-}
-
-__global__ void advance_kernel(int* step, int* lengths, const unsigned char* inactive, int B)
-{
-    const int b = blockIdx.x * blockDim.x + threadIdx.x;
-    if (b < B && !inactive[b]) lengths[b] += 1;
-    if (b == 0) *step += 1;
 }
 
 // [tp][B][vocab/tp] -> [B][vocab]
@@ -402,9 +332,9 @@ int run_step(StepCtx& c)
         gather_logits_kernel<<<m.h->sm_count * 4, 256, 0, s>>>(st.logits_out, m.logits, B, m.local_vocab, tp);
         if (!c.ok_cuda()) return c.rc;
     }
-    argmax_kernel<<<B, 1024, 0, s>>>(m.logits, m.picked, st.output_ids, st.step, m.inactive, B, m.local_vocab, tp, st.max_steps);
+    step_argmax(m.logits, m.picked, st.output_ids, st.step, m.inactive, B, m.local_vocab, tp, st.max_steps, s);
     if (!c.ok_cuda()) return c.rc;
-    advance_kernel<<<(B + 127) / 128, 128, 0, s>>>(st.step, st.sequence_lengths, m.inactive, B);
+    step_advance(st.step, st.sequence_lengths, m.inactive, B, s);
     if (!c.ok_cuda()) return c.rc;
     c.launches += m.h->launches - l0;
     return c.rc;
@@ -436,6 +366,9 @@ extern "C" int tm_llama_create(tm_llama** out, tm_handle* h, tm_comm* comm, cons
     tm_llama* m = new (std::nothrow) tm_llama();
     if (!m) return TM_ERR_CUDA;
     m->h              = h;
+    m->vocab_size     = c.vocab_size;
+    m->max_batch_size = c.max_batch_size;
+    m->session_len    = c.session_len;
     m->comm           = comm;
     m->cfg            = c;
     m->hidden         = c.head_num * 128;
@@ -483,22 +416,47 @@ extern "C" int tm_llama_create(tm_llama** out, tm_handle* h, tm_comm* comm, cons
     return TM_OK;
 }
 
+tm_llama::~tm_llama()
+{
+    graph.drop();
+    if (cublas) cublasDestroy(cublas);
+    for (void* p : {(void*)x, (void*)hbuf, (void*)qkv, (void*)ctx, (void*)ffn, (void*)logits_local, (void*)logits, (void*)ids_in, (void*)picked,
+                    (void*)inactive, (void*)order, (void*)seq_desc, (void*)rope_table, (void*)ssq, cublas_ws}) {
+        if (p) cudaFree(p);
+    }
+    for (void* p : owned) cudaFree(p);
+    for (void* p : {(void*)prefill_buf.x, (void*)prefill_buf.h, (void*)prefill_buf.qkv, (void*)prefill_buf.q, (void*)prefill_buf.k,
+                    (void*)prefill_buf.v, (void*)prefill_buf.ctx, (void*)prefill_buf.ffn, (void*)prefill_buf.pad, (void*)prefill_buf.len,
+                    prefill_buf.staged}) {
+        if (p) cudaFree(p);
+    }
+}
+
+int tm_llama::decode(const tm_llama_decode_state& st, int n_steps, bool use_graph, cudaStream_t s)
+{
+    return tm_llama_decode(this, &st, n_steps, use_graph, s);
+}
+
+int tm_llama::new_cache(tm_cache_manager** out, size_t max_entry_count, size_t chunk_size) const
+{
+    return tm_cache_manager_create(out, cfg.num_layer, local_kv_heads, cfg.size_per_head, cfg.session_len, cfg.quant_policy & 4 ? 8 : 16,
+                                   max_entry_count, chunk_size, h->device);
+}
+
+size_t tm_llama::slab_bytes() const
+{
+    return (size_t)2 * cfg.num_layer * local_kv_heads * cfg.session_len * cfg.size_per_head * (cfg.quant_policy & 4 ? 1 : 2);
+}
+
 extern "C" int tm_llama_destroy(tm_llama* m)
 {
-    if (!m) return TM_OK;
-    if (m->graph_exec) cudaGraphExecDestroy(m->graph_exec);
-    if (m->cublas) cublasDestroy(m->cublas);
-    for (void* p : {(void*)m->x, (void*)m->hbuf, (void*)m->qkv, (void*)m->ctx, (void*)m->ffn, (void*)m->logits_local,
-                    (void*)m->logits, (void*)m->ids_in, (void*)m->picked, (void*)m->inactive, (void*)m->order, (void*)m->seq_desc, (void*)m->rope_table, (void*)m->ssq, m->cublas_ws}) {
-        if (p) cudaFree(p);
-    }
-    for (void* p : m->owned) cudaFree(p);
-    for (void* p : {(void*)m->prefill.x, (void*)m->prefill.h, (void*)m->prefill.qkv, (void*)m->prefill.q, (void*)m->prefill.k,
-                    (void*)m->prefill.v, (void*)m->prefill.ctx, (void*)m->prefill.ffn, (void*)m->prefill.pad, (void*)m->prefill.len}) {
-        if (p) cudaFree(p);
-    }
     delete m;
     return TM_OK;
+}
+
+extern "C" tm_model* tm_llama_as_model(tm_llama* m)
+{
+    return m;
 }
 
 extern "C" int tm_llama_set_layer(tm_llama* m, int layer, const tm_llama_layer_weights* w)
@@ -522,10 +480,7 @@ extern "C" int tm_llama_set_layer(tm_llama* m, int layer, const tm_llama_layer_w
     l.ffn_output.scales_and_zeros                = w->w2_scales_zeros;
     std::memcpy(l.past_kv_scale, w->past_kv_scale, sizeof(l.past_kv_scale));
     l.set = true;
-    if (m->graph_exec) {  // pointers are baked into the captured step
-        cudaGraphExecDestroy(m->graph_exec);
-        m->graph_exec = nullptr;
-    }
+    m->graph.drop();  // pointers are baked into the captured step
     return TM_OK;
 }
 
@@ -535,10 +490,7 @@ extern "C" int tm_llama_set_globals(tm_llama* m, const void* tok_embeddings, con
     m->tok_embeddings = tok_embeddings;
     m->output_norm    = output_norm;
     m->output_weight  = output_weight;
-    if (m->graph_exec) {
-        cudaGraphExecDestroy(m->graph_exec);
-        m->graph_exec = nullptr;
-    }
+    m->graph.drop();
     return TM_OK;
 }
 
@@ -550,7 +502,7 @@ extern "C" int tm_llama_check_status(tm_llama* m, void* stream, unsigned* word)
 
 extern "C" unsigned long long tm_llama_last_launches(const tm_llama* m)
 {
-    return m ? m->last_launches : 0ull;
+    return m ? m->launches_of_last : 0ull;
 }
 
 extern "C" int tm_llama_decode(tm_llama* m, const tm_llama_decode_state* st, int n_steps, int use_graph, void* stream)
@@ -562,45 +514,17 @@ extern "C" int tm_llama_decode(tm_llama* m, const tm_llama_decode_state* st, int
     for (const auto& l : m->layers) {
         if (!l.set) return TM_ERR_INVALID_ARG;
     }
-    cudaStream_t s   = (cudaStream_t)stream;
-    m->last_launches = 0;
-    if (!use_graph) {
-        for (int i = 0; i < n_steps; ++i) {
-            StepCtx c{m, st, s};
-            if (run_step(c) != TM_OK) return c.rc;
-            m->last_launches += c.launches;
-        }
-        return TM_OK;
-    }
-    if (!m->graph_exec || std::memcmp(&m->graph_key, st, sizeof(*st)) != 0) {
-        if (m->graph_exec) {
-            cudaGraphExecDestroy(m->graph_exec);
-            m->graph_exec = nullptr;
-        }
-        if (s == nullptr) return TM_ERR_INVALID_ARG;  // the legacy stream cannot be captured
-        cudaGraph_t g = nullptr;
-        if (cudaStreamBeginCapture(s, cudaStreamCaptureModeThreadLocal) != cudaSuccess) return TM_ERR_CUDA;
+    cudaStream_t s = (cudaStream_t)stream;
+    return m->graph.run(m->h, *st, n_steps, use_graph != 0, s, &m->launches_of_last, [&](unsigned long long* n) {
         StepCtx c{m, st, s};
         run_step(c);
-        const cudaError_t e = cudaStreamEndCapture(s, &g);
-        if (c.rc != TM_OK || e != cudaSuccess || !g) {
-            if (g) cudaGraphDestroy(g);
-            m->h->last_cuda_error = (int)e;
-            return c.rc != TM_OK ? c.rc : TM_ERR_CUDA;
-        }
-        const cudaError_t ei = cudaGraphInstantiate(&m->graph_exec, g, 0);
-        cudaGraphDestroy(g);
-        if (ei != cudaSuccess) {
-            m->graph_exec         = nullptr;
-            m->h->last_cuda_error = (int)ei;
-            return TM_ERR_CUDA;
-        }
-        m->graph_key         = *st;
-        m->launches_per_step = c.launches;
-    }
-    for (int i = 0; i < n_steps; ++i) {
-        if (cudaGraphLaunch(m->graph_exec, s) != cudaSuccess) return TM_ERR_CUDA;
-    }
-    m->last_launches = m->launches_per_step * (unsigned long long)n_steps;
-    return TM_OK;
+        *n = c.launches;
+        return c.rc;
+    });
+}
+
+extern "C" int tm_batch_create(tm_batch** out, tm_llama* model, tm_cache_manager* cache, int max_batch_size, int session_len, int start_id,
+                               int end_id, int max_context_token_num)
+{
+    return tm_batch_create_model(out, model, cache, max_batch_size, session_len, start_id, end_id, max_context_token_num);
 }

@@ -5,6 +5,7 @@
 
 #include "comm.h"
 #include "handle.h"
+#include "model.h"
 #include "tm_b200.h"
 
 #include <cublas_v2.h>
@@ -47,8 +48,7 @@ private:
 
 }  // namespace tmb
 
-struct tm_llama {
-    tm_handle*      h    = nullptr;
+struct tm_llama final : tm_model {
     tm_comm*        comm = nullptr;
     tm_llama_config cfg{};
     int             hidden = 0, local_heads = 0, local_kv_heads = 0, local_inter = 0, local_vocab = 0;
@@ -75,14 +75,20 @@ struct tm_llama {
         int *   pad = nullptr, *len = nullptr;
         size_t  x_bytes = 0, h_bytes = 0, qkv_bytes = 0, q_bytes = 0, k_bytes = 0, v_bytes = 0, ctx_bytes = 0, ffn_bytes = 0,
                pad_bytes = 0, len_bytes = 0;
-    } prefill;
+        void*  staged = nullptr;  // device copy of a tm_model_prefill_state's host arrays
+        size_t staged_bytes = 0;
+    } prefill_buf;
 
     cublasHandle_t cublas    = nullptr;
     void*          cublas_ws = nullptr;
 
-    // one captured step, keyed by the state it was captured for
-    cudaGraphExec_t       graph_exec = nullptr;
-    tm_llama_decode_state graph_key{};
-    unsigned long long    launches_per_step = 0;
-    unsigned long long    last_launches     = 0;
+    tmb::StepGraph     graph;
+    unsigned long long launches_of_last = 0;
+
+    ~tm_llama() override;
+    int    prefill(const tm_model_prefill_state& st, cudaStream_t s) override;
+    int    decode(const tm_llama_decode_state& st, int n_steps, bool use_graph, cudaStream_t s) override;
+    int    new_cache(tm_cache_manager** out, size_t max_entry_count, size_t chunk_size) const override;
+    size_t slab_bytes() const override;
+    unsigned long long last_launches() const override { return launches_of_last; }
 };

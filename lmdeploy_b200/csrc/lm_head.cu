@@ -254,6 +254,7 @@ cudaError_t lm_head_prepare(int max_smem)
 {
     return cudaFuncSetAttribute(lm_head_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
 }
+static const KernelPreparation g_prepare(lm_head_prepare);
 
 // logits[tokens][ld] = x[tokens][hidden] . w[vocab][hidden]^T; tokens <= 256 per launch (longer batches are cut)
 int lm_head_launch(float* logits, int ld, const __half* x, const __half* w, int tokens, int vocab, int hidden, unsigned* status,

@@ -276,3 +276,37 @@ extern "C" int tm_llama_read_config(const char* dir, tm_llama_config* cfg, tm_ll
     if (info) *info = x;
     return TM_OK;
 }
+
+// ---------------------------------------------------------------------------------------------
+// Architecture table entry: a TurboMind workspace (config.ini + weight files)
+namespace {
+
+bool workspace_claims(const std::string& dir)
+{
+    std::FILE* f = std::fopen((dir + "/config.ini").c_str(), "rb");
+    if (f) std::fclose(f);
+    return f != nullptr;
+}
+
+int workspace_open(tm_model** out, tm_handle* h, const std::string& dir, const tm_model_options& opt)
+{
+    if (opt.dtype == TM_DTYPE_F32) return TM_ERR_UNSUPPORTED;  // W4A16 with fp16 activations only
+    tm_llama_config cfg{};
+    int             rc = tm_llama_read_config(dir.c_str(), &cfg, nullptr);
+    if (rc != TM_OK) return rc;
+    if (cfg.tensor_para_size != 1) return TM_ERR_UNSUPPORTED;  // ranks are set up through tm_llama_create
+    cfg.max_batch_size = opt.max_batch_size;
+    cfg.session_len    = opt.session_len;
+    tm_llama* m        = nullptr;
+    if ((rc = tm_llama_create(&m, h, nullptr, &cfg)) != TM_OK) return rc;
+    if ((rc = tm_llama_load_workspace(m, dir.c_str())) != TM_OK) {
+        tm_llama_destroy(m);
+        return rc;
+    }
+    *out = m;
+    return TM_OK;
+}
+
+const tmb::ArchitectureRegistration g_workspace({"turbomind-workspace", workspace_claims, workspace_open});
+
+}  // namespace

@@ -1,0 +1,68 @@
+// Sequence mixers of the config-driven decoder: softmax attention over a sliding window with pooled blocks behind it, and
+// a recurrence with a generalised delta rule.  Every size and constant is a field; sequences are described by spans.
+#pragma once
+#include "handle.h"
+
+#include <cuda_runtime.h>
+
+namespace tmb {
+
+// The new tokens of one sequence in a launch: rows [tok0, tok0 + n) of the activations, positions history, history + 1, ...
+struct SeqSpan {
+    unsigned char* slab    = nullptr;  // what the sequence caches (layout: decoder.h)
+    int            history = 0;
+    int            n       = 0;
+    int            tok0    = 0;
+    int            live    = 0;        // 0: the sequence sits this step out and nothing of it is written
+};
+
+struct WindowAttention {
+    int          heads = 0, kv_heads = 0, dim = 0, vdim = 0;
+    int          rot_dims = 0;           // leading dimensions that rotate, pairs (2i, 2i + 1)
+    const float* inv_freq = nullptr;     // device [rot_dims / 2]
+    float        scale = 1.f, softcap = 0.f;  // softcap 0: none
+    // A position i sees the tokens j with 0 <= i - j < window (0: all), and the mean key / value of every block of `pool`
+    // tokens (0: none) that ends at or before i - window.
+    int          window = 0, pool = 0;
+    // Token rows live in a ring: position p in row p % ring.  A ring holds the window (and a block) of the oldest query
+    // of a launch and all tokens of the launch.  Pooled rows: one per block.
+    int          ring = 0, pool_rows = 0;
+    size_t       k_off = 0, v_off = 0, pk_off = 0, pv_off = 0;  // bytes in the slab; [kv head][row][dim or vdim]
+    int          q_col = 0, k_col = 0, v_col = 0, g_col = 0;    // columns of the projections; g: one gate logit per head
+};
+
+// proj [tokens][proj_ld] (q is rotated in place in prefill), out [tokens][out_ld]: columns [0, heads * vdim) get the gated
+// output, [heads * vdim, out_pad) zeros.  spans: device array.  max_n: the longest span; max_context: upper bound on
+// history + n.
+struct MixerCall {
+    void*          proj     = nullptr;
+    int            proj_ld  = 0;
+    void*          out      = nullptr;
+    int            out_ld   = 0, out_pad = 0;
+    const SeqSpan* spans    = nullptr;
+    int            batch    = 0, tokens = 0, max_n = 0, max_context = 0;
+    bool           f32      = false;
+    bool           pdl      = false;
+};
+int window_attention_prefill(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st);
+int window_attention_decode(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st);
+
+struct DeltaRule {
+    int          heads = 0, dim = 0;
+    int          rank     = 0;         // of the decay's low-rank projection
+    const void*  w2       = nullptr;   // [heads * dim][w2_ld], element type
+    int          w2_ld    = 0;
+    const float* w0       = nullptr;   // [heads * dim]
+    const float* a_bias   = nullptr;   // [heads * dim]
+    const float* norm     = nullptr;   // [heads * dim], weight behind the per-head norm
+    float        norm_eps = 0.f;
+    float        unit_eps = 1e-6f;     // u = k / sqrt(sum k^2 + unit_eps)
+    float        decay_scale = 0.60653065971263342f;  // decay = exp(-decay_scale * sigmoid(.)); here exp(-1/2)
+    size_t       state_off = 0;        // bytes in the slab: float [head][key dim][value dim]
+    int          r_col = 0, k_col = 0, v_col = 0, a_col = 0, g_col = 0, w1_col = 0;  // columns of the projections; w1 after tanh
+};
+// scratch of a prefill: decay pre-activations and outputs, fp32 [tokens][heads * dim] each
+int delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, float* decay_pre, float* o, cudaStream_t st);
+int delta_rule_decode(tm_handle* h, const DeltaRule& d, const MixerCall& c, cudaStream_t st);
+
+}  // namespace tmb

@@ -17,6 +17,7 @@
 // fused in.  Splits meet in scratch memory; the last CTA to arrive for a (sequence, KV head)
 // merges them in a fixed order (no CTA waits for another).
 #include "common.cuh"
+#include "handle.h"
 #include "mmha.h"
 
 #include <cfloat>
@@ -773,6 +774,7 @@ cudaError_t mmha_prepare()
     if (e == cudaSuccess) e = mmha_prepare_one<false, 1>();
     return e;
 }
+static const KernelPreparation g_prepare([](int) { return mmha_prepare(); });
 
 MmhaPlan mmha_plan(int B, int H, int Hkv, int max_len, int sm_count, int want_chunk, int want_warps)
 {

@@ -8,6 +8,8 @@
 #include "llama.h"
 #include "tm_b200.h"
 
+#include <vector>
+
 using namespace tmb;
 
 namespace {
@@ -72,7 +74,7 @@ extern "C" int tm_llama_prefill(tm_llama* m, const tm_llama_prefill_state* st, v
     cudaSetDevice(m->h->device);
 
     // ---- activations of this call (kept and reused; grown when a larger call comes)
-    tm_llama::PrefillBuffers& pb = m->prefill;
+    tm_llama::PrefillBuffers& pb = m->prefill_buf;
     const size_t qkv_cols = (size_t)(H + 2 * Hkv) * 128;
     bool ok = grow(m, (void**)&pb.x, &pb.x_bytes, T * hid * 2) && grow(m, (void**)&pb.h, &pb.h_bytes, T * hid * 2)
               && grow(m, (void**)&pb.qkv, &pb.qkv_bytes, T * qkv_cols * 2)
@@ -144,4 +146,43 @@ extern "C" int tm_llama_prefill(tm_llama* m, const tm_llama_prefill_state* st, v
     }
     cudaSetDevice(prev);
     return rc;
+}
+
+// The scheduler's side: host arrays, staged in one device buffer
+int tm_llama::prefill(const tm_model_prefill_state& st, cudaStream_t s)
+{
+    if (st.want_count > 0 || st.residual_out) return TM_ERR_UNSUPPORTED;  // tm_llama_prefill keeps no logits
+    const size_t B = (size_t)st.batch_size, T = (size_t)st.cu_seqlens[B];
+    if (T == 0) return TM_OK;
+    // ids | cu_seqlens | history | context, then the cache pointers
+    std::vector<int> ints(st.input_ids, st.input_ids + T);
+    ints.insert(ints.end(), st.cu_seqlens, st.cu_seqlens + B + 1);
+    ints.insert(ints.end(), st.history_lengths, st.history_lengths + B);
+    int max_q = 0;
+    for (size_t b = 0; b < B; ++b) {
+        const int n = st.cu_seqlens[b + 1] - st.cu_seqlens[b];
+        ints.push_back(st.history_lengths[b] + n);
+        max_q = n > max_q ? n : max_q;
+    }
+    const size_t ptr_at = (ints.size() * sizeof(int) + 15) / 16 * 16;
+    if (!grow(this, &prefill_buf.staged, &prefill_buf.staged_bytes, ptr_at + 2 * B * sizeof(void*))) return TM_ERR_CUDA;
+    char* d = static_cast<char*>(prefill_buf.staged);
+    // pageable sources: the copies are staged before cudaMemcpyAsync returns
+    if (cudaMemcpyAsync(d, ints.data(), ints.size() * sizeof(int), cudaMemcpyHostToDevice, s) != cudaSuccess
+        || cudaMemcpyAsync(d + ptr_at, st.k_cache, B * sizeof(void*), cudaMemcpyHostToDevice, s) != cudaSuccess
+        || cudaMemcpyAsync(d + ptr_at + B * sizeof(void*), st.v_cache, B * sizeof(void*), cudaMemcpyHostToDevice, s) != cudaSuccess) {
+        return TM_ERR_CUDA;
+    }
+    const int*             di = reinterpret_cast<const int*>(d);
+    tm_llama_prefill_state l{};
+    l.batch_size      = (int)B;
+    l.token_num       = (int)T;
+    l.max_q_len       = max_q;
+    l.input_ids       = di;
+    l.cu_seqlens      = di + T;
+    l.history_lengths = di + T + B + 1;
+    l.context_lengths = di + T + 2 * B + 1;
+    l.k_cache_ptrs    = reinterpret_cast<void**>(d + ptr_at);
+    l.v_cache_ptrs    = reinterpret_cast<void**>(d + ptr_at) + B;
+    return tm_llama_prefill(this, &l, s);
 }

@@ -378,6 +378,7 @@ cudaError_t sampling_prepare(int max_smem)
     if (e != cudaSuccess) return e;
     return cudaFuncSetAttribute(sample_topp_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem - 1024);
 }
+static const KernelPreparation g_prepare(sampling_prepare);
 
 }  // namespace tmb
 

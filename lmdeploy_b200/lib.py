@@ -9,7 +9,9 @@ import ctypes as C
 import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
-LIB_PATH = os.path.join(_HERE, "_lib", "libtm_b200.so")
+# TM_B200_LIBRARY names a library that holds a part of the framework (build.py, COMPONENTS): symbols it lacks stay unbound
+LIB_PATH = os.environ.get("TM_B200_LIBRARY") or os.path.join(_HERE, "_lib", "libtm_b200.so")
+PARTIAL = "TM_B200_LIBRARY" in os.environ
 
 TM_OK = 0
 TM_ERR_INVALID_ARG = -1
@@ -45,7 +47,8 @@ def _preload_bundled_nccl() -> None:
 
 
 def _load() -> C.CDLL:
-    _preload_bundled_nccl()
+    if not PARTIAL:
+        _preload_bundled_nccl()
     if not os.path.exists(LIB_PATH):
         raise ImportError(
             f"{LIB_PATH} is missing: build it with `python -m lmdeploy_b200.build` "
@@ -152,6 +155,50 @@ class TmLlamaPrefillState(C.Structure):
                 ("k_cache_ptrs", C.c_void_p), ("v_cache_ptrs", C.c_void_p), ("hidden_out", C.c_void_p)]
 
 
+TM_DTYPE_BF16, TM_DTYPE_F32 = 0, 1
+
+
+class TmModelOptions(C.Structure):
+    """ctypes mirror of ``tm_model_options``."""
+    _fields_ = [("dtype", C.c_int), ("max_batch_size", C.c_int), ("session_len", C.c_int), ("max_prefill_tokens", C.c_int)]
+
+
+class TmModelInfo(C.Structure):
+    """ctypes mirror of ``tm_model_info``."""
+    _fields_ = [("vocab_size", C.c_int), ("max_batch_size", C.c_int), ("session_len", C.c_int), ("can_rewind", C.c_int),
+                ("slab_bytes", C.c_size_t)]
+
+
+class TmModelPrefillState(C.Structure):
+    """ctypes mirror of ``tm_model_prefill_state`` (host arrays)."""
+    _fields_ = [("batch_size", C.c_int), ("input_ids", C.POINTER(C.c_int)), ("cu_seqlens", C.POINTER(C.c_int)),
+                ("history_lengths", C.POINTER(C.c_int)), ("k_cache", C.POINTER(C.c_void_p)), ("v_cache", C.POINTER(C.c_void_p)),
+                ("want_count", C.c_int), ("want", C.POINTER(C.c_int)), ("logits_out", C.c_void_p), ("residual_out", C.c_void_p)]
+
+
+class TmMixerCall(C.Structure):
+    """ctypes mirror of ``tm_mixer_call``."""
+    _fields_ = [("proj", C.c_void_p), ("proj_ld", C.c_int), ("out", C.c_void_p), ("out_ld", C.c_int), ("batch", C.c_int),
+                ("history", C.POINTER(C.c_int)), ("n", C.POINTER(C.c_int)), ("slabs", C.POINTER(C.c_void_p)), ("dtype", C.c_int),
+                ("decode", C.c_int)]
+
+
+class TmWindowAttentionParams(C.Structure):
+    """ctypes mirror of ``tm_window_attention_params``."""
+    _fields_ = [(n, C.c_int) for n in ("heads", "kv_heads", "dim", "vdim", "rot_dims")] + [("inv_freq", C.c_void_p)] \
+        + [("scale", C.c_float), ("softcap", C.c_float)] + [(n, C.c_int) for n in ("window", "pool", "ring", "pool_rows")] \
+        + [(n, C.c_size_t) for n in ("k_off", "v_off", "pooled_k_off", "pooled_v_off")] \
+        + [(n, C.c_int) for n in ("q_col", "k_col", "v_col", "g_col")]
+
+
+class TmDeltaRuleParams(C.Structure):
+    """ctypes mirror of ``tm_delta_rule_params``."""
+    _fields_ = [("heads", C.c_int), ("dim", C.c_int), ("rank", C.c_int), ("w2", C.c_void_p), ("w2_ld", C.c_int), ("w0", C.c_void_p),
+                ("a_bias", C.c_void_p), ("norm", C.c_void_p), ("norm_eps", C.c_float), ("unit_eps", C.c_float),
+                ("decay_scale", C.c_float), ("state_off", C.c_size_t)] \
+        + [(n, C.c_int) for n in ("r_col", "k_col", "v_col", "a_col", "g_col", "w1_col")]
+
+
 # name -> (restype, argtypes); must list every symbol declared in include/tm_b200.h
 SIGNATURES = {
     "tm_create": (_i, [C.POINTER(_vp), _i]),
@@ -171,6 +218,27 @@ SIGNATURES = {
     "tm_fuse_w1_w3_s4_k_m8": (_i, [_u32p, _u32p, _i, _i, _vp]),
     "tm_dequantize_s4": (_i, [_vp, _u32p, _sz, _vp]),
     "tm_batch_create": (_i, [C.POINTER(_vp), _vp, _vp, _i, _i, _i, _i, _i]),
+    "tm_batch_create_model": (_i, [C.POINTER(_vp), _vp, _vp, _i, _i, _i, _i, _i]),
+    "tm_cache_manager_create_slabs": (_i, [C.POINTER(_vp), _sz, _sz, _sz, _sz, _i]),
+    "tm_model_open": (_i, [C.POINTER(_vp), _vp, C.c_char_p, C.POINTER(TmModelOptions)]),
+    "tm_model_close": (_i, [_vp]),
+    "tm_model_last_error": (C.c_char_p, []),
+    "tm_model_architectures": (_i, [C.c_char_p, _sz]),
+    "tm_model_describe": (_i, [_vp, C.POINTER(TmModelInfo)]),
+    "tm_model_new_cache": (_i, [_vp, _sz, _sz, C.POINTER(_vp)]),
+    "tm_llama_as_model": (_vp, [_vp]),
+    "tm_model_prefill": (_i, [_vp, C.POINTER(TmModelPrefillState), _vp]),
+    "tm_model_decode": (_i, [_vp, C.POINTER(TmLlamaDecodeState), _i, _i, _vp]),
+    "tm_model_last_launches": (C.c_ulonglong, [_vp]),
+    "tm_model_check_status": (_i, [_vp, _vp, C.POINTER(C.c_uint)]),
+    "tm_replay_create": (_i, [C.POINTER(_vp), _vp, _sz]),
+    "tm_replay_destroy": (_i, [_vp]),
+    "tm_replay_step": (_i, [_vp, C.c_uint64, C.POINTER(C.c_int), _i, C.POINTER(C.c_int), _i, C.POINTER(C.c_float)]),
+    "tm_replay_end": (_i, [_vp, C.c_uint64]),
+    "tm_decoder_create_random": (_i, [C.POINTER(_vp), _vp, C.c_char_p, C.POINTER(TmModelOptions), C.c_ulonglong]),
+    "tm_window_attention": (_i, [_vp, C.POINTER(TmWindowAttentionParams), C.POINTER(TmMixerCall), _vp]),
+    "tm_delta_rule": (_i, [_vp, C.POINTER(TmDeltaRuleParams), C.POINTER(TmMixerCall), _vp]),
+    "tm_gemm_dense": (_i, [_vp, _vp, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _vp]),
     "tm_batch_destroy": (_i, [_vp]),
     "tm_batch_submit": (_i, [_vp, C.POINTER(TmRequest)]),
     "tm_batch_step": (_i, [_vp, _vp, _i]),
@@ -229,6 +297,8 @@ SIGNATURES = {
 
 def _bind():
     for name, (res, args) in SIGNATURES.items():
+        if PARTIAL and not hasattr(lib, name):
+            continue
         fn = getattr(lib, name)  # AttributeError if the library lacks a declared symbol
         fn.restype = res
         fn.argtypes = args
