@@ -595,7 +595,7 @@ TM_API int tm_llama_check_status(tm_llama* m, void* stream, unsigned* word);
 
 /* ------------------------------------------------------------------------------------------
  * Served models: one interface over the models of this library, which the scheduler, the command line
- * (lmdeploy_b200/serve.py) and the trace replay (bin/trace_run) use.  tm_model_open chooses by what the folder holds:
+ * (lmdeploy_b200/generate.py) and the trace replay (bin/trace_run) use.  tm_model_open chooses by what the folder holds:
  *   config.json with "architecture": "Rumazen" and model.safetensors   the config-driven decoder (window attention with
  *       pooled blocks, generalised delta rule, parallel layers); bf16, or everything in fp32
  *   config.ini and weight files                                        a TurboMind W4A16 workspace (tm_llama)

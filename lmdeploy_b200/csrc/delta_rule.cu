@@ -171,8 +171,8 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const DeltaKernelPara
 
 // One new token per sequence, one CTA per (head, sequence): decay projection, step, head norm and gate in one kernel.
 // The state passes through registers once: thread = (column, every RG-th row).
-constexpr int kStepThreads = 512;
-template<typename E, int ROWS>  // ROWS: state elements per thread
+// ROWS: state elements per thread, held in registers between the two products; 0: read again for the second (large heads).
+template<typename E, int ROWS, int kStepThreads>
 __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaKernelParams p)
 {
     __shared__ float u[kMaxDim], au[kMaxDim], w[kMaxDim], k[kMaxDim], r[kMaxDim], v[kMaxDim];
@@ -188,7 +188,7 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaKer
     const int    col = tid % dim, rg = tid / dim;
     const bool   on  = rg < groups;
     float*       state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * dim;
-    float        st[ROWS];
+    float        st[ROWS > 0 ? ROWS : 1];
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
         const int row = rg + i * groups;
@@ -229,6 +229,9 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaKer
         const int x = rg + i * groups;
         if (x < dim) z = fmaf(u[x], st[i], z);
     }
+    if (ROWS == 0 && on && s.history > 0) {
+        for (int x = rg; x < dim; x += groups) z = fmaf(u[x], state[(size_t)x * dim + col], z);
+    }
     red[tid] = on ? z : 0.f;
     __syncthreads();
     if (tid < dim) {
@@ -247,6 +250,14 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaKer
                 st[i] = fmaf(w[x], st[i], fmaf(k[x], v[col], -au[x] * z));
                 o     = fmaf(r[x], st[i], o);
                 state[(size_t)x * dim + col] = st[i];
+            }
+        }
+        if (ROWS == 0) {
+            for (int x = rg; x < dim; x += groups) {
+                const float old = s.history > 0 ? state[(size_t)x * dim + col] : 0.f;
+                const float now = fmaf(w[x], old, fmaf(k[x], v[col], -au[x] * z));
+                o               = fmaf(r[x], now, o);
+                state[(size_t)x * dim + col] = now;
             }
         }
     }
@@ -297,10 +308,10 @@ template<typename E>
 cudaError_t step_dispatch(const DeltaKernelParams& p, cudaStream_t st)
 {
     const dim3 grid(p.d.heads, p.c.batch);
-    const int  rows = (p.d.dim + kStepThreads / p.d.dim - 1) / (kStepThreads / p.d.dim);
-    if (rows <= 8) return launch_kernel(delta_step_kernel<E, 8>, grid, dim3(kStepThreads), 0, st, p.c.pdl, p);
-    if (rows <= 32) return launch_kernel(delta_step_kernel<E, 32>, grid, dim3(kStepThreads), 0, st, p.c.pdl, p);
-    return launch_kernel(delta_step_kernel<E, 128>, grid, dim3(kStepThreads), 0, st, p.c.pdl, p);
+    auto       rows = [&](int threads) { return (p.d.dim + threads / p.d.dim - 1) / (threads / p.d.dim); };
+    if (rows(512) <= 8) return launch_kernel(delta_step_kernel<E, 8, 512>, grid, dim3(512), 0, st, p.c.pdl, p);
+    if (rows(1024) <= 19) return launch_kernel(delta_step_kernel<E, 19, 1024>, grid, dim3(1024), 0, st, p.c.pdl, p);
+    return launch_kernel(delta_step_kernel<E, 0, 1024>, grid, dim3(1024), 0, st, p.c.pdl, p);
 }
 
 bool valid(const DeltaRule& d, const MixerCall& c)

@@ -224,12 +224,18 @@ int window_attention_prefill(tm_handle* h, const WindowAttention& a, const Mixer
     const WindowKernelParams p{a, c};
     int rc = c.f32 ? write_and_pool<float>(h, p, st) : write_and_pool<__nv_bfloat16>(h, p, st);
     if (rc != TM_OK) return rc;
+    if (window_attention_tc_supported(a, c)) return window_attention_tc(h, a, c, st);
     return c.f32 ? attend<float>(h, p, st) : attend<__nv_bfloat16>(h, p, st);
 }
 
 int window_attention_decode(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st)
 {
-    return window_attention_prefill(h, a, c, st);
+    if (!valid(a, c)) return TM_ERR_UNSUPPORTED;
+    if (window_attention_step_supported(a, c)) return window_attention_step(h, a, c, st);
+    const WindowKernelParams p{a, c};
+    const int rc = c.f32 ? write_and_pool<float>(h, p, st) : write_and_pool<__nv_bfloat16>(h, p, st);
+    if (rc != TM_OK) return rc;
+    return c.f32 ? attend<float>(h, p, st) : attend<__nv_bfloat16>(h, p, st);
 }
 
 }  // namespace tmb

@@ -30,5 +30,8 @@ struct WindowKernelParams {
 // tcgen05 prefill attention (window_attention_tc.cu): bf16, q rotated, keys / values / pooled rows in the slab
 bool window_attention_tc_supported(const WindowAttention& a, const MixerCall& c);
 int  window_attention_tc(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st);
+// one-token attention with the rotation, the cache append and the pooling fused in (window_attention_decode.cu): bf16
+bool window_attention_step_supported(const WindowAttention& a, const MixerCall& c);
+int  window_attention_step(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st);
 
 }  // namespace tmb

@@ -226,6 +226,11 @@ class LlamaModel:
         if rc != _l.TM_OK:
             raise _l.TmError(rc, f"tm_llama_check_status: device status word 0x{w.value:x}")
 
+    @property
+    def ptr(self):
+        """the model behind the served-model interface (tm_model)"""
+        return C.c_void_p(_l.lib.tm_llama_as_model(self._m))
+
     def last_launches(self) -> int:
         return int(_l.lib.tm_llama_last_launches(self._m))
 
@@ -296,18 +301,16 @@ class Batch:
 
     QUEUED, RUNNING, FINISHED, FAILED = 0, 1, 2, 3
 
-    def __init__(self, model: LlamaModel, max_batch_size: int, start_id: int = 1, end_id: int = 2, cache_max_entry_count: int = 0,
+    def __init__(self, model, max_batch_size: int, start_id: int = 1, end_id: int = 2, cache_max_entry_count: int = 0,
                  cache_chunk_size: int = 1, max_context_token_num: int = 0):
-        cfg = model.cfg
+        """``model``: anything with the served-model interface (``LlamaModel``, ``decoder.Model``)"""
         self.model = model
         self._cache = C.c_void_p()
         entries = cache_max_entry_count or max_batch_size
-        _l.check(_l.lib.tm_cache_manager_create(C.byref(self._cache), cfg.num_layer, cfg.kv_head_num // model.tp, cfg.size_per_head,
-                                                model.session_len, 8 if cfg.quant_policy & 4 else 16, entries, cache_chunk_size,
-                                                model.device), "tm_cache_manager_create")
+        _l.check(_l.lib.tm_model_new_cache(model.ptr, entries, cache_chunk_size, C.byref(self._cache)), "tm_model_new_cache")
         self._b = C.c_void_p()
-        _l.check(_l.lib.tm_batch_create(C.byref(self._b), model._m, self._cache, max_batch_size, model.session_len, start_id, end_id,
-                                        max_context_token_num), "tm_batch_create")
+        _l.check(_l.lib.tm_batch_create_model(C.byref(self._b), model.ptr, self._cache, max_batch_size, model.session_len, start_id, end_id,
+                                              max_context_token_num), "tm_batch_create_model")
 
     def submit(self, session_id: int, input_ids, request_output_len: int, start: bool = True, end: bool = True, top_k: int = 0,
                top_p: float = 0.0, temperature: float = 0.0, repetition_penalty: float = 0.0, random_seed: int = 0,
