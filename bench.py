@@ -712,6 +712,266 @@ def run_prefill_model_workload(args, rank, world, device):
     }
 
 
+def rumazen_config(layers=8):
+    """layers of the size of a 7B-class model: one window-attention layer in four, the others with the delta rule"""
+    attn = dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, softcap=30.0, mask=dict(size=2048, pool=16),
+                rot=dict(dims=128, base=500000.0, scaling=dict(factor=8.0)))
+    delta = dict(heads=64, dim=64, rank=96)
+    return dict(architecture="Rumazen", vocab=32000, width=4096, norm=dict(eps=1e-6), embedding=dict(scale=1.0),
+                layers=[dict(type="general_delta" if i % 4 else "attention", mixer=delta if i % 4 else attn,
+                             mlp=dict(kind="dense", ff=11008)) for i in range(layers)])
+
+
+def device_ms(fn, stream, steps, warmup, flush=None):
+    """mean device time of fn on `stream` (CUDA events around every call, L2 flushed between the calls when asked)"""
+    for _ in range(warmup):
+        fn()
+    torch.cuda.synchronize()
+    total = 0.0
+    for _ in range(steps):
+        if flush is not None:
+            flush.zero_()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(stream)
+        fn()
+        e1.record(stream)
+        torch.cuda.synchronize()
+        total += e0.elapsed_time(e1)
+    return total / steps
+
+
+def rumazen_kernels(device, stream, args, peaks, flush):
+    """The kernels of the Rumazen layers one at a time, each with the like kernel of the W4A16 LLaMA beside it at equal
+    size: achieved share of the measured peak (HBM for decode, bf16 GEMM for prefill contractions)."""
+    import ctypes as C
+    from lmdeploy_b200 import lib as l
+    from lmdeploy_b200 import turbomind as tm
+    from lmdeploy_b200 import awq
+    h = l.default_handle(device)
+    st = C.c_void_p(stream.cuda_stream)
+    W, FF, H, G, D = 4096, 11008, 32, 8, 128
+    K, Wm = args.steps, args.warmup
+    bf, rows = torch.bfloat16, []
+    g = torch.Generator(device=device).manual_seed(1)
+
+    def add(name, ms, flops=0.0, nbytes=0.0, like=False):
+        tf, gb = flops / ms * 1e-9, nbytes / ms * 1e-6
+        bound = "tensor" if flops / (peaks["bf16_tflops"] * 1e12) > nbytes / (peaks["hbm_gbs"] * 1e9) else "hbm"
+        frac = tf / peaks["bf16_tflops"] if bound == "tensor" else gb / peaks["hbm_gbs"]
+        rows.append(dict(kernel=name, like_kernel_of_llama=like, us=round(ms * 1e3, 2), bound=bound, tflops=round(tf, 1), gbs=round(gb, 1),
+                         frac=round(frac, 3)))
+
+    # ---- dense GEMMs: gate/up-sized input projection and down-sized output projection
+    for n, k in ((2 * FF, W), (W, FF)):
+        w = torch.randn(n, k, device=device, generator=g).to(bf)
+        lin = awq.random_linear(n, k, g)
+        op = tm.LlamaLinear(device)
+        for t in (1, 16, 64, 4096):
+            x, out = torch.randn(t, k, device=device, generator=g).to(bf), torch.empty(t, n, dtype=bf, device=device)
+            ms = device_ms(lambda: l.check(l.lib.tm_gemm_dense(h.ptr, out.data_ptr(), n, 0, x.data_ptr(), k, w.data_ptr(), k, t, n, k, 0, st), "gemm"),
+                           stream, K, Wm, flush)
+            add(f"dense_tc_kernel {n}x{k}, {t} tokens", ms, 2.0 * t * n * k, 2.0 * (n * k + t * k + t * n))
+            xh, oh = x.half(), torch.empty(t, n, dtype=torch.float16, device=device)
+            ms = device_ms(lambda: op.forward(oh, xh, t, lin), stream, K, Wm, flush)
+            add(f"gemm_s4_f16 {n}x{k}, {t} tokens", ms, 2.0 * t * n * k, n * k / 2 + n * k / 128 * 4 + 2.0 * (t * k + t * n), True)
+        del w, lin
+
+    # ---- window attention
+    def call(proj, ld, out, out_ld, hist, n, slabs, decode):
+        c = l.TmMixerCall()
+        keep = (proj, out, slabs)
+        c.proj, c.proj_ld, c.out, c.out_ld, c.batch = proj.data_ptr(), ld, out.data_ptr(), out_ld, len(n)
+        c.history, c.n = (C.c_int * len(n))(*hist), (C.c_int * len(n))(*n)
+        c.slabs = (C.c_void_p * len(n))(*[s.data_ptr() for s in slabs])
+        c.dtype, c.decode = l.TM_DTYPE_BF16, int(decode)
+        return c, keep
+
+    def window(size, pool, softcap, context, portion):
+        p = l.TmWindowAttentionParams()
+        freq = (500000.0 ** (-2.0 * torch.arange(D // 2, dtype=torch.float64) / D)).float().to(device)
+        p.heads, p.kv_heads, p.dim, p.vdim, p.rot_dims, p.inv_freq = H, G, D, D, D, freq.data_ptr()
+        p.scale, p.softcap, p.window, p.pool = D ** -0.5, softcap, size, pool
+        p.ring = -(-(min(context, max(size, pool) + portion) if size else context) // 128) * 128
+        p.pool_rows = context // pool + 8 if pool else 0
+        p.k_off, p.v_off = 0, G * p.ring * D * 2
+        p.pooled_k_off = 2 * p.v_off
+        p.pooled_v_off = p.pooled_k_off + G * p.pool_rows * D * 2
+        p.q_col, p.k_col, p.v_col, p.g_col = 0, H * D, (H + G) * D, (H + 2 * G) * D
+        return p, freq, p.pooled_v_off + G * p.pool_rows * D * 2 + 256
+
+    ld = (H + 2 * G) * D + 128
+    for what, size, pool, softcap in (("window 2048, blocks of 16, softcap", 2048, 16, 30.0), ("all keys, no softcap", 0, 0, 0.0)):
+        S, B = 2048, 8
+        p, freq, nbytes = window(size, pool, softcap, S, S)
+        slabs = [torch.zeros(nbytes, dtype=torch.uint8, device=device) for _ in range(B)]
+        proj = torch.randn(B * S, ld, device=device, generator=g).to(bf)
+        out = torch.empty(B * S, H * D, dtype=bf, device=device)
+        c, keep = call(proj, ld, out, H * D, [0] * B, [S] * B, slabs, False)
+        ms = device_ms(lambda: l.check(l.lib.tm_window_attention(h.ptr, C.byref(p), C.byref(c), st), "attention"), stream, K, Wm)
+        add(f"window attention prefill (write + pool + attention), {B} x {S} tokens, {what}", ms, 4.0 * D * H * B * S * (S + 1) / 2)
+        if size:
+            S2 = 16384
+            p, freq, nbytes = window(size, pool, softcap, S2, S2)
+            slabs = [torch.zeros(nbytes, dtype=torch.uint8, device=device)]
+            c, keep = call(proj, ld, out, H * D, [0], [S2], slabs, False)
+            pairs = sum(min(i + 1, size) + max(0, (i - size + 1) // pool) for i in range(S2))
+            ms = device_ms(lambda: l.check(l.lib.tm_window_attention(h.ptr, C.byref(p), C.byref(c), st), "attention"), stream, K, Wm)
+            add(f"window attention prefill (write + pool + attention), 1 x {S2} tokens, {what}", ms, 4.0 * D * H * pairs)
+        del slabs, proj, out, keep
+        for B, ctx in ((1, 4096), (64, 4096)):
+            p, freq, nbytes = window(size, pool, softcap, ctx + 8, 1)
+            slabs = [torch.zeros(nbytes, dtype=torch.uint8, device=device) for _ in range(B)]
+            proj, out = torch.randn(B, ld, device=device, generator=g).to(bf), torch.empty(B, H * D, dtype=bf, device=device)
+            c, keep = call(proj, ld, out, H * D, [ctx] * B, [1] * B, slabs, True)
+            keys = min(ctx, size) + (ctx - size + 1) // pool if size else ctx
+            ms = device_ms(lambda: l.check(l.lib.tm_window_attention(h.ptr, C.byref(p), C.byref(c), st), "attention"), stream, K, Wm, flush)
+            add(f"window_step_kernel, batch {B} at {ctx} tokens, {what}", ms, 0.0, B * G * keys * D * 4.0)
+            del slabs, keep
+    # the LLaMA's attention kernels on the same keys: 8 x 2048 tokens of prefill, 4096 cached tokens in decode, fp16 cache
+    S, B = 2048, 8
+    q = torch.randn(B, H, S, D, device=device, generator=g).half()
+    kc, vc = (torch.zeros(B, G * S * D, dtype=torch.float16, device=device) for _ in range(2))
+    kp, vp = (torch.tensor([t[b].data_ptr() for b in range(B)], dtype=torch.int64, device=device) for t in (kc, vc))
+    cu = torch.arange(0, (B + 1) * S, S, dtype=torch.int32, device=device)
+    lens = torch.full((B,), S, dtype=torch.int32, device=device)
+    out = torch.empty(B * S, H * D, dtype=torch.float16, device=device)
+    ms = device_ms(lambda: tm.fusedMultiHeadAttention(out, q, kp, vp, 0, cu, lens, B, S, S, H, G, D, 0, None), stream, K, Wm)
+    add(f"context_attention_tc_kernel, {B} x {S} tokens", ms, 4.0 * D * H * B * S * (S + 1) / 2, 0.0, True)
+    del q, kc, vc, out
+    for B, ctx in ((1, 4096), (64, 4096)):
+        kc, vc = (torch.zeros(B, G * (ctx + 64) * D, dtype=torch.float16, device=device) for _ in range(2))
+        kp, vp = (torch.tensor([t[b].data_ptr() for b in range(B)], dtype=torch.int64, device=device) for t in (kc, vc))
+        qkv, out = torch.randn(B, (H + 2 * G) * D, device=device, generator=g).half(), torch.empty(B, H * D, dtype=torch.float16, device=device)
+        ln = torch.full((B,), ctx, dtype=torch.int32, device=device)
+        a = l.TmMmhaParams()
+        a.out, a.q, a.k, a.v = out.data_ptr(), qkv.data_ptr(), qkv.data_ptr() + H * D * 2, qkv.data_ptr() + (H + G) * D * 2
+        a.stride, a.batch_size, a.memory_max_len, a.num_heads, a.num_kv_heads = (H + 2 * G) * D, B, ctx + 64, H, G
+        a.hidden_size_per_head, a.rotary_embedding_dim, a.timestep, a.inv_sqrt_dh = D, D, ctx, D ** -0.5
+        a.length_per_sample, a.k_cache_per_sample, a.v_cache_per_sample = ln.data_ptr(), kp.data_ptr(), vp.data_ptr()
+        a.rotary_embedding_base = 10000.0
+        ms = device_ms(lambda: l.check(l.lib.tm_mmha_decode(h.ptr, C.byref(a), st), "mmha"), stream, K, Wm, flush)
+        add(f"mmha_decode_kernel (fp16 cache), batch {B} at {ctx} tokens", ms, 0.0, B * G * ctx * D * 4.0, True)
+
+    # ---- delta rule (no like kernel in the LLaMA; bytes: projections, outputs, decay pre-activations, state)
+    HD, dim, rank = 64, 64, 96
+    n = HD * dim
+    w2 = torch.randn(n, rank, device=device, generator=g).to(bf)
+    vecs = torch.randn(3, n, device=device, generator=g)
+    p = l.TmDeltaRuleParams()
+    p.heads, p.dim, p.rank, p.w2, p.w2_ld = HD, dim, rank, w2.data_ptr(), rank
+    p.w0, p.a_bias, p.norm = (vecs[i].data_ptr() for i in range(3))
+    p.norm_eps, p.unit_eps, p.decay_scale = 1e-6, 1e-6, float(np.exp(-0.5))
+    p.r_col, p.k_col, p.v_col, p.a_col, p.g_col, p.w1_col = 0, n, 2 * n, 3 * n, 4 * n, 5 * n
+    ld = 5 * n + rank
+    for B, t, decode in ((1, 4096, False), (4, 1024, False), (8, 2048, False), (1, 1, True), (16, 1, True), (64, 1, True)):
+        proj, out = torch.randn(B * t, ld, device=device, generator=g).to(bf), torch.empty(B * t, n, dtype=bf, device=device)
+        slabs = [torch.zeros(n * dim * 4, dtype=torch.uint8, device=device) for _ in range(B)]
+        c, keep = call(proj, ld, out, n, [8 if decode else 0] * B, [t] * B, slabs, decode)
+        ms = device_ms(lambda: l.check(l.lib.tm_delta_rule(h.ptr, C.byref(p), C.byref(c), st), "delta"), stream, K, Wm, flush if decode else None)
+        nbytes = B * (t * (ld * 2.0 + n * 2.0) + n * dim * 8.0) + n * rank * 2.0
+        add(f"delta_step_kernel, batch {B}" if decode else f"delta rule prefill (decay GEMM + scan + finish), {B} x {t} tokens", ms, 0.0, nbytes)
+    return rows
+
+
+def run_rumazen_workload(args, rank, world, device):
+    """Prefill and decode throughput of a random-weight Rumazen model with layers of a 7B-class size (8 layers, bf16), beside
+    the W4A16 LLaMA of the same width, depth, feed-forward and attention heads, and the kernels of both one at a time.
+    value = tokens/s of a decode step at batch 64 behind 4096 tokens each."""
+    from lmdeploy_b200 import decoder, llama
+    torch.cuda.set_device(device)
+    K, Wm, L = min(args.steps, 32), args.warmup, 8
+    cfg, peaks = rumazen_config(L), measured_peaks()
+    stream = torch.cuda.Stream(device)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)   # larger than L2
+    rng = np.random.default_rng(5 + rank)
+    sampler = ClockSampler(device)
+    res, launches = {"rumazen": {}, "llama_w4a16": {}}, 0
+    ctx = 4096
+    with torch.cuda.stream(stream):
+        sampler.start()
+        model = decoder.Model.random(cfg, "bfloat16", 64, ctx + 512, 4096, device)
+        slabs = torch.zeros(64, -(-model.slab_bytes // 256) * 256, dtype=torch.uint8, device=device)
+        addr = [slabs[b].data_ptr() for b in range(64)]
+        prompts = [list(map(int, rng.integers(0, cfg["vocab"], 4096))) for _ in range(1)]
+        for B, t in ((1, 1024), (1, 4096), (4, 1024)):
+            ms = device_ms(lambda: model.prefill([prompts[0][:t]] * B, [0] * B, addr[:B]), stream, max(3, K // 4), Wm)
+            res["rumazen"][f"prefill {B} x {t}"] = dict(ms=round(ms, 3), tokens_per_s=round(B * t / ms * 1e3, 1))
+        for B in (1, 16, 64):
+            st = model.new_state(addr[:B], [ctx] * B, 400)
+            model.decode(st, Wm, True, stream.cuda_stream)
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            barrier(world)
+            e0.record(stream)
+            model.decode(st, K, True, stream.cuda_stream)
+            e1.record(stream)
+            torch.cuda.synchronize()
+            ms = max_over_ranks(e0.elapsed_time(e1), world) / K
+            launches += model.last_launches()
+            res["rumazen"][f"decode batch {B} at {ctx}"] = dict(ms=round(ms, 4), tokens_per_s=round(B / ms * 1e3, 1), launches=model.last_launches() // K)
+        headline_ms = ms
+        # end to end: the step's input tokens from pinned host memory, the drawn tokens back, every step
+        st = model.new_state(addr, [ctx] * 64, 400, np.full((400, 64), 0, np.int32))
+        host_in, host_out = torch.randint(0, cfg["vocab"], (64,), dtype=torch.int32).pin_memory(), torch.empty(64, dtype=torch.int32).pin_memory()
+
+        def e2e_step(i):
+            st.forced_ids[i].copy_(host_in, non_blocking=True)
+            model.decode(st, 1, True, stream.cuda_stream)
+            host_out.copy_(st.output_ids[i], non_blocking=True)
+            stream.synchronize()
+
+        for i in range(Wm):
+            e2e_step(i)
+        t0 = time.time()
+        for i in range(Wm, Wm + K):
+            e2e_step(i)
+        e2e = 64 * K / (time.time() - t0)
+        model.check_status()
+        model.close()
+        del slabs, st
+        lcfg = llama.LlamaConfig(32, 8, 11008, L, quant_policy=0, name="llama 8 layers")
+        lm = llama.LlamaModel(lcfg, 64, ctx + 512, device, None)
+        lm.random_init(seed=0)
+        for B, t in ((1, 1024), (1, 4096), (4, 1024)):
+            ls = lm.new_state(B, 1, np.zeros(B, np.int32), None)
+
+            def run():
+                ls.lengths.zero_()
+                lm.prefill(ls, [prompts[0][:t]] * B)
+            ms = device_ms(run, stream, max(3, K // 4), Wm)
+            res["llama_w4a16"][f"prefill {B} x {t}"] = dict(ms=round(ms, 3), tokens_per_s=round(B * t / ms * 1e3, 1))
+            del ls
+        for B in (1, 16, 64):
+            ls = lm.new_state(B, 400)
+            ls.lengths.fill_(ctx)
+            lm.decode(ls, Wm, True)
+            torch.cuda.synchronize()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(stream)
+            lm.decode(ls, K, True)
+            e1.record(stream)
+            torch.cuda.synchronize()
+            ms = e0.elapsed_time(e1) / K
+            res["llama_w4a16"][f"decode batch {B} at {ctx}"] = dict(ms=round(ms, 4), tokens_per_s=round(B / ms * 1e3, 1), launches=lm.last_launches() // K)
+            del ls
+        lm.close()
+        del lm
+        torch.cuda.empty_cache()
+        kernels = rumazen_kernels(device, stream, argparse.Namespace(steps=max(5, K // 2), warmup=Wm), peaks, flush)
+        clocks = sampler.stop()
+    return {
+        "metric": "decode tokens/s Rumazen, 8 layers of a 7B-class size", "value": round(64 * world / headline_ms * 1e3, 1), "unit": "tokens/s",
+        "n_gpus": world, "steps": K, "warmup": Wm, "ms_per_step": round(headline_ms, 4), "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "rumazen", "model": "8 layers, width 4096, ff 11008, vocab 32000; 2 window attention (32 / 8 heads of 128, window "
+                   "2048, blocks of 16), 6 delta rule (64 heads of 64, rank 96)", "global_batch": 64 * world, "seq_len": ctx,
+                   "l2": "decode: weights and caches of a step larger than L2; single kernels: L2 flushed between launches (decode), inputs larger "
+                   "than L2 (prefill)", "parallelism": "replicas only" if world > 1 else "single GPU"},
+        "throughput": res, "per_kernel": kernels, "clocks": clocks, "gpu_launches": int(launches),
+        "e2e": {"value": round(e2e * world, 1), "unit": "tokens/s", "h2d_bytes_per_step": 64 * 4, "d2h_bytes_per_step": 64 * 4},
+    }
+
+
 DECODE_WORKLOADS = {
     # name: (config attr, batch, prompt_lo, prompt_hi, new_tokens)
     "decode7b": ("LLAMA2_7B", 64, 128, 1024, 256),
@@ -1163,7 +1423,7 @@ def main():
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--workload", default="decode",
-                    help="decode (7B at 1 GPU, 70B tensor-parallel at N > 1) | decode7b | decode70b | gemm | mmha | prefill | prefill7b")
+                    help="decode (7B at 1 GPU, 70B tensor-parallel at N > 1) | decode7b | decode70b | gemm | mmha | prefill | prefill7b | rumazen")
     ap.add_argument("--batch-override", type=int, default=0, help="smaller batch for smoke runs")
     ap.add_argument("--max-prompt", type=int, default=0, help="cap on the prompt length for smoke runs")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
@@ -1185,6 +1445,10 @@ def main():
         if rank == 0:   # the reference's prefill needs its engine and its flash-attention build (CUTLASS): neither is built
             print(json.dumps({"impl": "reference", "unavailable": "whole-model prefill of the reference needs its engine and "
                               "CUTLASS flash attention; use --workload prefill for its kernels"}), flush=True)
+        return
+    if args.impl == "reference" and args.workload == "rumazen":
+        if rank == 0:
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no such model"}), flush=True)
         return
     if args.impl == "reference" and args.workload not in ("gemm", "mmha", "prefill"):
         # whole-model workloads: the reference's CPU path (the engine around its kernels is out of scope)
@@ -1210,6 +1474,8 @@ def main():
         out = run_prefill_workload(args, rank, world, local)
     elif args.workload == "prefill7b":
         out = run_prefill_model_workload(args, rank, world, local)
+    elif args.workload == "rumazen":
+        out = run_rumazen_workload(args, rank, world, local)
     else:
         raise SystemExit(f"unknown workload {args.workload}")
     if rank == 0:
