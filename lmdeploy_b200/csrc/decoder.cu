@@ -171,7 +171,7 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
     bool         ok = true;
     x_ld            = round_up(W, 8);
     size_t off      = 0;
-    int    delta_cols = 0;
+    size_t delta_floats = 0;  // of a prefill, per token
     auto   take = [&](size_t bytes) {
         const size_t at = off;
         off             = round_up_bytes(off + bytes);
@@ -248,7 +248,7 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
             vec(mp + "a.b", n, &L.a_bias, 0.f, 1.f);
             vec(mp + "norm", n, &L.norm, 1.f, 0.f);
             d.w2 = L.w2, d.w0 = L.w0, d.a_bias = L.a_bias, d.norm = L.norm;
-            delta_cols = std::max(delta_cols, n);
+            delta_floats = std::max(delta_floats, delta_rule_scratch_floats(d));
         }
         L.mixer_cols = round_up(cols, kDenseTile);
         L.in_rows    = L.mixer_cols + 2 * ff;
@@ -278,8 +278,7 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
     const size_t T        = (size_t)tokens, column_tiles = (size_t)(W + kDenseTile - 1) / kDenseTile;
     const size_t logit_rows = (size_t)max_batch_size;
     ok = ok && alloc((void**)&x, T * W * 4) && alloc((void**)&ssq, column_tiles * ssq_stride * 4) && alloc(&xb, T * x_ld * es)
-         && alloc(&proj, T * proj_ld * es) && alloc(&y, T * y_ld * es) && alloc((void**)&decay_pre, T * delta_cols * 4)
-         && alloc((void**)&delta_o, T * delta_cols * 4) && alloc((void**)&logits, logit_rows * c.vocab * 4)
+         && alloc(&proj, T * proj_ld * es) && alloc(&y, T * y_ld * es) && alloc((void**)&delta_scratch, (size_t)max_prefill * delta_floats * 4) && alloc((void**)&logits, logit_rows * c.vocab * 4)
          && alloc(&want_xb, (size_t)kWantRows * x_ld * es) && alloc((void**)&want_ssq, (size_t)kWantRows * 4) && alloc((void**)&ids, T * 4)
          && alloc((void**)&want, T * 4) && alloc((void**)&picked, T * 4) && alloc((void**)&inactive, T) && alloc((void**)&spans, T * sizeof(SeqSpan));
     const cudaError_t e = cudaGetLastError();
@@ -424,7 +423,7 @@ int tm_decoder::run_layers(const Pass& p, cudaStream_t s)
             rc = p.decode ? window_attention_decode(h, L.attention, c, s) : window_attention_prefill(h, L.attention, c, s);
         }
         else {
-            rc = p.decode ? delta_rule_decode(h, L.delta, c, s) : delta_rule_prefill(h, L.delta, c, decay_pre, delta_o, s);
+            rc = p.decode ? delta_rule_decode(h, L.delta, c, s) : delta_rule_prefill(h, L.delta, c, delta_scratch, s);
         }
         if (rc != TM_OK || (last && !p.need_output)) break;
 
@@ -550,14 +549,13 @@ int tm_decoder::decode(const tm_llama_decode_state& st, int n_steps, bool use_gr
 // ---------------------------------------------------------------------------------------------------- mechanisms alone
 namespace {
 
-// spans of a call on the device, freed behind the work on the stream
+// Spans of a call on the device, and `extra` bytes of scratch behind them, in the handle's operator buffer
 struct DeviceSpans {
-    SeqSpan*     d = nullptr;
-    cudaStream_t s;
-    MixerCall    c;
-    int          rc = TM_OK;
+    MixerCall c;
+    void*     scratch = nullptr;
+    int       rc      = TM_OK;
 
-    DeviceSpans(const tm_mixer_call& call, cudaStream_t stream): s(stream)
+    DeviceSpans(tm_handle* h, const tm_mixer_call& call, size_t extra_per_token, cudaStream_t s)
     {
         if (!call.proj || !call.out || call.batch <= 0 || !call.history || !call.n || !call.slabs
             || (call.dtype != TM_DTYPE_BF16 && call.dtype != TM_DTYPE_F32)) {
@@ -565,7 +563,6 @@ struct DeviceSpans {
             return;
         }
         std::vector<SeqSpan> sp(call.batch);
-        c.max_n = 0;
         for (int b = 0; b < call.batch; ++b) {
             if (!call.slabs[b] || call.history[b] < 0 || call.n[b] < 0 || (call.decode && call.n[b] != 1)) rc = TM_ERR_INVALID_ARG;
             sp[b].slab = static_cast<unsigned char*>(call.slabs[b]), sp[b].history = call.history[b], sp[b].n = call.n[b];
@@ -576,16 +573,21 @@ struct DeviceSpans {
         }
         if (rc == TM_OK && c.tokens == 0) rc = TM_ERR_INVALID_ARG;
         if (rc != TM_OK) return;
-        if (cudaMallocAsync((void**)&d, sp.size() * sizeof(SeqSpan), s) != cudaSuccess
-            || cudaMemcpyAsync(d, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess) {
-            rc = TM_ERR_CUDA;
+        const size_t spans_bytes = round_up_bytes(sp.size() * sizeof(SeqSpan)), need = spans_bytes + extra_per_token * c.tokens;
+        if (need > h->op_buffer_bytes) {
+            if (h->op_buffer) cudaFree(h->op_buffer);  // waits for the work that uses it
+            h->op_buffer = nullptr, h->op_buffer_bytes = 0;
+            if (cudaMalloc(&h->op_buffer, need) != cudaSuccess) {
+                rc = TM_ERR_CUDA;
+                return;
+            }
+            h->op_buffer_bytes = need;
         }
+        SeqSpan* d = static_cast<SeqSpan*>(h->op_buffer);
+        scratch    = static_cast<char*>(h->op_buffer) + spans_bytes;
+        if (cudaMemcpyAsync(d, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess) rc = TM_ERR_CUDA;
         c.proj = call.proj, c.proj_ld = call.proj_ld, c.out = call.out, c.out_ld = call.out_ld, c.spans = d, c.batch = call.batch;
         c.f32 = call.dtype == TM_DTYPE_F32;
-    }
-    ~DeviceSpans()
-    {
-        if (d) cudaFreeAsync(d, s);
     }
 };
 
@@ -594,7 +596,8 @@ struct DeviceSpans {
 extern "C" int tm_window_attention(tm_handle* h, const tm_window_attention_params* q, const tm_mixer_call* call, void* stream)
 {
     if (!h || !q || !call) return TM_ERR_INVALID_ARG;
-    DeviceSpans sp(*call, (cudaStream_t)stream);
+    const cudaStream_t s = (cudaStream_t)stream;
+    DeviceSpans        sp(h, *call, 0, s);
     if (sp.rc != TM_OK) return sp.rc;
     WindowAttention a;
     a.heads = q->heads, a.kv_heads = q->kv_heads, a.dim = q->dim, a.vdim = q->vdim, a.rot_dims = q->rot_dims, a.inv_freq = q->inv_freq;
@@ -606,23 +609,18 @@ extern "C" int tm_window_attention(tm_handle* h, const tm_window_attention_param
         const int end = call->history[b] + call->n[b], need = a.window > 0 ? std::min(end, std::max(a.window, a.pool) + call->n[b]) : end;
         if (need > a.ring || (a.pool > 0 && end / a.pool > a.pool_rows)) return TM_ERR_INVALID_ARG;
     }
-    return call->decode ? window_attention_decode(h, a, sp.c, sp.s) : window_attention_prefill(h, a, sp.c, sp.s);
+    return call->decode ? window_attention_decode(h, a, sp.c, s) : window_attention_prefill(h, a, sp.c, s);
 }
 
 extern "C" int tm_delta_rule(tm_handle* h, const tm_delta_rule_params* q, const tm_mixer_call* call, void* stream)
 {
     if (!h || !q || !call || !q->w2 || !q->w0 || !q->a_bias || !q->norm) return TM_ERR_INVALID_ARG;
-    DeviceSpans sp(*call, (cudaStream_t)stream);
-    if (sp.rc != TM_OK) return sp.rc;
-    DeltaRule d;
+    const cudaStream_t s = (cudaStream_t)stream;
+    DeltaRule          d;
     d.heads = q->heads, d.dim = q->dim, d.rank = q->rank, d.w2 = q->w2, d.w2_ld = q->w2_ld, d.w0 = q->w0, d.a_bias = q->a_bias, d.norm = q->norm;
     d.norm_eps = q->norm_eps, d.unit_eps = q->unit_eps, d.decay_scale = q->decay_scale, d.state_off = q->state_off;
     d.r_col = q->r_col, d.k_col = q->k_col, d.v_col = q->v_col, d.a_col = q->a_col, d.g_col = q->g_col, d.w1_col = q->w1_col;
-    if (call->decode) return delta_rule_decode(h, d, sp.c, sp.s);
-    float*       scratch = nullptr;
-    const size_t n       = (size_t)sp.c.tokens * d.heads * d.dim;
-    if (cudaMallocAsync((void**)&scratch, 2 * n * sizeof(float), sp.s) != cudaSuccess) return TM_ERR_CUDA;
-    const int rc = delta_rule_prefill(h, d, sp.c, scratch, scratch + n, sp.s);
-    cudaFreeAsync(scratch, sp.s);
-    return rc;
+    DeviceSpans sp(h, *call, call->decode ? 0 : delta_rule_scratch_floats(d) * sizeof(float), s);
+    if (sp.rc != TM_OK) return sp.rc;
+    return call->decode ? delta_rule_decode(h, d, sp.c, s) : delta_rule_prefill(h, d, sp.c, static_cast<float*>(sp.scratch), s);
 }

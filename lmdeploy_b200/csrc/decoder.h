@@ -88,7 +88,7 @@ struct tm_decoder final : tm_model {
     void *             embed = nullptr, *head = nullptr;
     float*             final_gain = nullptr;
     // activations of one pass
-    float *       x = nullptr, *ssq = nullptr, *decay_pre = nullptr, *delta_o = nullptr, *logits = nullptr;
+    float *       x = nullptr, *ssq = nullptr, *delta_scratch = nullptr, *logits = nullptr;
     void *        xb = nullptr, *proj = nullptr, *y = nullptr, *want_xb = nullptr;
     float*        want_ssq = nullptr;
     int           ssq_stride = 0;

@@ -12,137 +12,207 @@
 namespace tmb {
 namespace {
 
-constexpr int kMaxDim    = 256;
-constexpr int kChunk     = 16;   // tokens staged in shared memory at a time
-constexpr int kPrepWarps = 4;    // warps that stage the next chunk while the others walk through this one
+constexpr int kMaxDim = 256;
 
 struct DeltaKernelParams {
     DeltaRule    d;
     MixerCall    c;
-    const float* decay_pre;
-    float*       o;
-    int          column_parts;
+    const float* decay_pre;  // [tokens][heads * dim]
+    float*       records;    // [head][token][record]
+    float*       o;          // [tokens][heads * dim], over decay_pre, which nobody needs by then
+    unsigned*    status;
+    long long    max_wait;
 };
 
-// DP: head size rounded up to 16, 32, ..., 256.  A group of DP / 8 lanes owns a column of S, eight rows per lane in
-// registers.
+// DP: head size rounded up to 16, 32, ..., 256.
+// What the scan reads of a (head, token), made by delta_gates_kernel:
+//   u (first token of a pair) or u * w of the token before (second)  |  b = a u  |  w  |  k  |  r  |  v  |  beta, kappa
+// Tokens go in pairs, counted from the start of the span.  With z = u^T S read before the token's own update, the second
+// token's z follows from the state before the FIRST one:
+//   z1 = (u1 * w0)^T S - (u1 . b0) z0 + (u1 . k0) v0 = ... - beta z0 + kappa v0
+// so that both products with the state are in flight together.
 template<int DP>
 struct ScanShape {
-    static constexpr int kLanes    = DP / 8;
-    static constexpr int kThreads  = 256;                 // scanning threads
-    static constexpr int kColumns  = kThreads / kLanes;   // columns of one CTA
-    static constexpr int kSmem     = 2 * kChunk * (5 * DP + kColumns) * 4;
+    static constexpr int kLanes   = DP / 8;              // lanes that own a column of S, eight rows each in registers
+    static constexpr int kThreads = 256;
+    static constexpr int kColumns = kThreads / kLanes;   // columns of one CTA
+    static constexpr int kRecord  = 6 * DP + 4;          // floats
+    static constexpr int kChunk   = DP <= 64 ? 16 : (DP == 128 ? 8 : 4);  // tokens of a stage
+    static constexpr int kStages  = 3;
+    static constexpr int kSmem    = kStages * kChunk * kRecord * 4;
 };
 
+// one warp per (pair of tokens, head)
 template<typename E, int DP>
-__global__ void __launch_bounds__(ScanShape<DP>::kThreads + kPrepWarps * 32) delta_scan_kernel(const DeltaKernelParams p)
+__global__ void __launch_bounds__(128) delta_gates_kernel(const DeltaKernelParams p)
+{
+    using S           = ScanShape<DP>;
+    constexpr int kPer = (DP + 31) / 32;
+    pdl_wait();
+    pdl_launch_dependents();
+    const DeltaRule& d = p.d;
+    const SeqSpan    s = p.c.spans[blockIdx.z];
+    const int        h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31, dim = d.dim;
+    const int        t0 = 2 * (int)blockIdx.x;
+    if (!s.live || t0 >= s.n || h >= d.heads) return;
+    const int n = h * dim;
+    float     w0[kPer], b0[kPer], k0[kPer];
+#pragma unroll
+    for (int t = 0; t < 2; ++t) {
+        if (t0 + t >= s.n) return;
+        const size_t tok = (size_t)s.tok0 + t0 + t;
+        const E*     row = static_cast<const E*>(p.c.proj) + tok * p.c.proj_ld;
+        const float* pre = p.decay_pre + tok * d.heads * dim + n;
+        float        k[kPer], a[kPer], z[kPer], r[kPer], v[kPer], ksq = 0.f;
+#pragma unroll
+        for (int e = 0; e < kPer; ++e) {
+            const int  c  = lane + 32 * e;
+            const bool on = c < dim;
+            k[e] = on ? to_f32(row[d.k_col + n + c]) : 0.f;
+            a[e] = on ? to_f32(row[d.a_col + n + c]) + d.a_bias[n + c] : 0.f;
+            z[e] = on ? pre[c] + d.w0[n + c] : 0.f;
+            r[e] = on ? to_f32(row[d.r_col + n + c]) : 0.f;
+            v[e] = on ? to_f32(row[d.v_col + n + c]) : 0.f;
+            ksq += k[e] * k[e];
+        }
+        const float inv   = 1.f / sqrtf(warp_sum(ksq) + d.unit_eps);
+        float       beta = 0.f, kappa = 0.f;
+        float*      rec = p.records + ((size_t)h * p.c.tokens + tok) * S::kRecord;
+#pragma unroll
+        for (int e = 0; e < kPer; ++e) {
+            const int   c = lane + 32 * e;
+            const float u = k[e] * inv, b = sigmoid_f32(a[e]) * u, w = expf(-d.decay_scale * sigmoid_f32(z[e]));
+            float       first = u;
+            if (t == 1) {
+                beta += u * b0[e];
+                kappa += u * k0[e];
+                first = u * w0[e];
+            }
+            if (c < DP) rec[c] = first, rec[DP + c] = b, rec[2 * DP + c] = w, rec[3 * DP + c] = k[e], rec[4 * DP + c] = r[e], rec[5 * DP + c] = v[e];
+            w0[e] = w, b0[e] = b, k0[e] = k[e];
+        }
+        if (t == 1) {
+            beta  = warp_sum(beta);
+            kappa = warp_sum(kappa);
+        }
+        if (lane == 0) *reinterpret_cast<float4*>(rec + 6 * DP) = make_float4(beta, kappa, 0.f, 0.f);
+    }
+}
+
+// The sequential part.  CTA = (block of value columns, head, sequence); the records of a head are contiguous, so one bulk
+// copy brings a chunk of tokens into a stage.
+template<int DP>
+__global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(const DeltaKernelParams p)
 {
     using S = ScanShape<DP>;
-    extern __shared__ __align__(16) float sm[];  // [2][kChunk][5][DP] u, a u, w, k, r; then [2][kChunk][columns] v
-    float* const sm_v = sm + 2 * kChunk * 5 * DP;
+    extern __shared__ __align__(128) float sm[];
+    __shared__ uint64_t full[S::kStages];
+    const int tid = threadIdx.x;
+    if (tid == 0) {
+        for (int i = 0; i < S::kStages; ++i) mbar_init(&full[i], 1);
+        fence_mbar_init();
+    }
+    __syncthreads();
     pdl_wait();
     pdl_launch_dependents();
     const DeltaRule& d = p.d;
     const SeqSpan    s = p.c.spans[blockIdx.z];
     if (!s.live || s.n <= 0) return;
-    const int  h = blockIdx.y, dim = d.dim, c0 = blockIdx.x * S::kColumns;
-    const int  tid = threadIdx.x;
-    const bool scan = tid < S::kThreads;
-    const E*   proj = static_cast<const E*>(p.c.proj) + (size_t)s.tok0 * p.c.proj_ld;
-
-    // the keys' side of one chunk: a warp per token
-    auto stage = [&](int chunk, int buf) {
-        const int warp = (tid - S::kThreads) >> 5, lane = tid & 31;
-        for (int t = warp; t < kChunk; t += kPrepWarps) {
-            const int tok = chunk * kChunk + t;
-            if (tok >= s.n) break;
-            const E*     row = proj + (size_t)tok * p.c.proj_ld;
-            const float* pre = p.decay_pre + (size_t)(s.tok0 + tok) * d.heads * dim + h * dim;
-            float*       dst = sm + (size_t)(buf * kChunk + t) * 5 * DP;
-            float        k[DP / 32 + 1], ksq = 0.f;
-#pragma unroll
-            for (int e = 0; e < (DP + 31) / 32; ++e) {
-                const int c = lane + 32 * e;
-                k[e]        = c < dim ? to_f32(row[d.k_col + h * dim + c]) : 0.f;
-                ksq += k[e] * k[e];
-            }
-            const float inv = 1.f / sqrtf(warp_sum(ksq) + d.unit_eps);
-#pragma unroll
-            for (int e = 0; e < (DP + 31) / 32; ++e) {
-                const int c = lane + 32 * e;
-                if (c >= DP) continue;
-                float u = 0.f, au = 0.f, w = 0.f, r = 0.f;
-                if (c < dim) {
-                    u  = k[e] * inv;
-                    au = sigmoid_f32(to_f32(row[d.a_col + h * dim + c]) + d.a_bias[h * dim + c]) * u;
-                    w  = expf(-d.decay_scale * sigmoid_f32(pre[c] + d.w0[h * dim + c]));
-                    r  = to_f32(row[d.r_col + h * dim + c]);
-                }
-                dst[c] = u, dst[DP + c] = au, dst[2 * DP + c] = w, dst[3 * DP + c] = k[e], dst[4 * DP + c] = r;
-            }
-            float* vd = sm_v + (size_t)(buf * kChunk + t) * S::kColumns;
-            for (int j = lane; j < S::kColumns; j += 32) vd[j] = c0 + j < dim ? to_f32(row[d.v_col + h * dim + c0 + j]) : 0.f;
-        }
+    const int    h = blockIdx.y, dim = d.dim, c0 = blockIdx.x * S::kColumns;
+    const float* src    = p.records + ((size_t)h * p.c.tokens + s.tok0) * S::kRecord;
+    const int    chunks = (s.n + S::kChunk - 1) / S::kChunk;
+    auto fetch = [&](int ch) {
+        const int      stage = ch % S::kStages;
+        const uint32_t bytes = (uint32_t)min(S::kChunk, s.n - ch * S::kChunk) * S::kRecord * 4;
+        mbar_arrive_expect_tx(&full[stage], bytes);
+        asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                         smem_u32(sm + (size_t)stage * S::kChunk * S::kRecord)),
+                     "l"(src + (size_t)ch * S::kChunk * S::kRecord), "r"(bytes), "r"(smem_u32(&full[stage]))
+                     : "memory");
     };
-
+    if (tid == 0) {
+        for (int ch = 0; ch < min(S::kStages, chunks); ++ch) fetch(ch);
+    }
     // lane's rows of its column: 4 at 4 * part and 4 at DP / 2 + 4 * part (conflict-free 16-byte reads)
-    const int part = tid % S::kLanes, lc = tid / S::kLanes, col = c0 + lc;
+    const int part = tid % S::kLanes, col = c0 + tid / S::kLanes, v_at = min(col, DP - 1);
     float*    state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * dim;
     float     st[8];
     auto      row_of = [&](int i) { return (i < 4 ? 0 : DP / 2) + 4 * part + (i & 3); };
-    if (scan) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int r = row_of(i);
-            st[i]       = s.history > 0 && r < dim && col < dim ? state[(size_t)r * dim + col] : 0.f;
-        }
+    for (int i = 0; i < 8; ++i) {
+        const int r = row_of(i);
+        st[i]       = s.history > 0 && r < dim && col < dim ? state[(size_t)r * dim + col] : 0.f;
     }
-    else {
-        stage(0, 0);
-    }
-    __syncthreads();
-    const int chunks = (s.n + kChunk - 1) / kChunk;
-    for (int ch = 0; ch < chunks; ++ch) {
-        const int buf = ch & 1;
-        if (scan) {
-            const int nt = min(kChunk, s.n - ch * kChunk);
-            for (int t = 0; t < nt; ++t) {
-                const float* src = sm + (size_t)(buf * kChunk + t) * 5 * DP + 4 * part;
-                auto vec = [&](int which, float (&x)[8]) {
-                    const float4 lo = *reinterpret_cast<const float4*>(src + which * DP);
-                    const float4 hi = *reinterpret_cast<const float4*>(src + which * DP + DP / 2);
-                    x[0] = lo.x, x[1] = lo.y, x[2] = lo.z, x[3] = lo.w, x[4] = hi.x, x[5] = hi.y, x[6] = hi.z, x[7] = hi.w;
-                };
-                float u[8], au[8], w[8], k[8], r[8];
-                vec(0, u), vec(1, au), vec(2, w), vec(3, k), vec(4, r);
-                const float v = sm_v[(size_t)(buf * kChunk + t) * S::kColumns + lc];
-                float       z = 0.f;
+    float* o_out = p.o + (size_t)s.tok0 * d.heads * dim + h * dim + col;
+    bool   ok    = true;
+    int    ch    = 0;
+    for (; ch < chunks; ++ch) {
+        ok           = mbar_wait(&full[ch % S::kStages], (ch / S::kStages) & 1, p.max_wait);
+        const int nt = min(S::kChunk, s.n - ch * S::kChunk);
+        for (int t = 0; t < nt; t += 2) {
+            const float* rec = sm + (size_t)((ch % S::kStages) * S::kChunk + t) * S::kRecord;
+            auto vec = [&](const float* r, int which, float (&x)[8]) {
+                const float4 lo = *reinterpret_cast<const float4*>(r + which * DP + 4 * part);
+                const float4 hi = *reinterpret_cast<const float4*>(r + which * DP + DP / 2 + 4 * part);
+                x[0] = lo.x, x[1] = lo.y, x[2] = lo.z, x[3] = lo.w, x[4] = hi.x, x[5] = hi.y, x[6] = hi.z, x[7] = hi.w;
+            };
+            auto dot = [&](const float (&x)[8]) {
+                float a = x[0] * st[0], b = x[1] * st[1];
 #pragma unroll
-                for (int i = 0; i < 8; ++i) z = fmaf(u[i], st[i], z);
+                for (int i = 2; i < 8; i += 2) a = fmaf(x[i], st[i], a), b = fmaf(x[i + 1], st[i + 1], b);
+                return a + b;
+            };
+            auto update = [&](const float* r, float z, float v) {
+                float b[8], w[8], k[8];
+                vec(r, 1, b), vec(r, 2, w), vec(r, 3, k);
 #pragma unroll
-                for (int m = S::kLanes / 2; m >= 1; m >>= 1) z += __shfl_xor_sync(0xffffffffu, z, m);
-                float o = 0.f;
+                for (int i = 0; i < 8; ++i) st[i] = fmaf(w[i], st[i], fmaf(k[i], v, -b[i] * z));
+            };
+            // two sums over the lanes of the column at the price of one: even lanes end up with the first, odd lanes with
+            // the second
+            auto reduce2 = [&](float a, float b) {
+                const bool odd = part & 1;
+                float      x   = odd ? b : a;
+                x += __shfl_xor_sync(0xffffffffu, odd ? a : b, 1);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    st[i] = fmaf(w[i], st[i], fmaf(k[i], v, -au[i] * z));
-                    o     = fmaf(r[i], st[i], o);
-                }
-#pragma unroll
-                for (int m = S::kLanes / 2; m >= 1; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
-                if (part == 0 && col < dim) p.o[(size_t)(s.tok0 + ch * kChunk + t) * d.heads * dim + h * dim + col] = o;
+                for (int m = 2; m < S::kLanes; m *= 2) x += __shfl_xor_sync(0xffffffffu, x, m);
+                return x;
+            };
+            const bool   two  = t + 1 < nt;
+            const float* rec1 = two ? rec + S::kRecord : rec;
+            float        u0[8], u1[8], r0[8], r1[8];
+            vec(rec, 0, u0), vec(rec1, 0, u1);
+            const float v0 = rec[5 * DP + v_at], v1 = rec1[5 * DP + v_at];
+            const float mine = reduce2(dot(u0), dot(u1)), other = __shfl_xor_sync(0xffffffffu, mine, 1);
+            const float z0 = part & 1 ? other : mine, y1 = part & 1 ? mine : other;
+            update(rec, z0, v0);
+            vec(rec, 4, r0);
+            const float o0 = dot(r0);
+            float       o1 = 0.f;
+            if (two) {
+                update(rec1, y1 - rec1[6 * DP] * z0 + rec1[6 * DP + 1] * v0, v1);
+                vec(rec1, 4, r1);
+                o1 = dot(r1);
             }
+            const float o = reduce2(o0, o1);
+            if (part < 2 && (part == 0 || two) && col < dim) o_out[(size_t)(ch * S::kChunk + t + part) * d.heads * dim] = o;
         }
-        else if (ch + 1 < chunks) {
-            stage(ch + 1, buf ^ 1);
-        }
-        __syncthreads();
+        // everybody is through with the stage; one outcome for the whole CTA
+        if (!__syncthreads_and(ok)) break;
+        if (tid == 0 && ch + S::kStages < chunks) fetch(ch + S::kStages);
     }
-    if (scan) {
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int r = row_of(i);
-            if (r < dim && col < dim) state[(size_t)r * dim + col] = st[i];
+    if (ch < chunks) {
+        if (tid == 0) {
+            atomicOr(p.status, kStatusGemmPipeWait);
+            // not before the copies in flight have landed
+            for (int c = ch; c < min(ch + S::kStages, chunks); ++c) mbar_wait(&full[c % S::kStages], (c / S::kStages) & 1, p.max_wait);
         }
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int r = row_of(i);
+        if (r < dim && col < dim) state[(size_t)r * dim + col] = st[i];
     }
 }
 
@@ -153,20 +223,27 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const DeltaKernelPara
     pdl_wait();
     pdl_launch_dependents();
     const DeltaRule& d    = p.d;
-    const int        lane = threadIdx.x & 31, t = blockIdx.x;
+    const int        lane = threadIdx.x & 31, t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5);
     const E*         row  = static_cast<const E*>(p.c.proj) + (size_t)t * p.c.proj_ld;
     E*               out  = static_cast<E*>(p.c.out) + (size_t)t * p.c.out_ld;
-    for (int h = threadIdx.x >> 5; h < d.heads; h += 8) {
-        const float* o  = p.o + ((size_t)t * d.heads + h) * d.dim;
-        float        sq = 0.f;
-        for (int c = lane; c < d.dim; c += 32) sq += o[c] * o[c];
-        const float inv = 1.f / sqrtf(warp_sum(sq) / (float)d.dim + d.norm_eps);
-        for (int c = lane; c < d.dim; c += 32) {
-            const int n = h * d.dim + c;
-            out[n]      = from_f32<E>(o[c] * inv * d.norm[n] * sigmoid_f32(to_f32(row[d.g_col + n])));
-        }
+    if (blockIdx.y == 0) {
+        for (int n = d.heads * d.dim + threadIdx.x; n < p.c.out_pad; n += 256) out[n] = from_f32<E>(0.f);
     }
-    for (int n = d.heads * d.dim + threadIdx.x; n < p.c.out_pad; n += 256) out[n] = from_f32<E>(0.f);
+    if (h >= d.heads) return;
+    const float* o = p.o + ((size_t)t * d.heads + h) * d.dim;
+    float        x[kMaxDim / 32], sq = 0.f;
+#pragma unroll
+    for (int e = 0; e < kMaxDim / 32; ++e) {
+        const int c = lane + 32 * e;
+        x[e]        = c < d.dim ? o[c] : 0.f;
+        sq += x[e] * x[e];
+    }
+    const float inv = 1.f / sqrtf(warp_sum(sq) / (float)d.dim + d.norm_eps);
+#pragma unroll
+    for (int e = 0; e < kMaxDim / 32; ++e) {
+        const int c = lane + 32 * e, n = h * d.dim + c;
+        if (c < d.dim) out[n] = from_f32<E>(x[e] * inv * d.norm[n] * sigmoid_f32(to_f32(row[d.g_col + n])));
+    }
 }
 
 // One new token per sequence, one CTA per (head, sequence): decay projection, step, head norm and gate in one kernel.
@@ -285,23 +362,34 @@ __global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaKer
 }
 
 template<typename E, int DP>
-cudaError_t scan_launch(DeltaKernelParams p, cudaStream_t st)
+cudaError_t scan_launch(const DeltaKernelParams& p, cudaStream_t st)
 {
-    using S = ScanShape<DP>;
-    cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<E, DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kSmem);
+    using S       = ScanShape<DP>;
+    cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, S::kSmem);
+    if (e != cudaSuccess) return e;
+    e = launch_kernel(delta_gates_kernel<E, DP>, dim3((p.c.max_n + 1) / 2, (p.d.heads + 3) / 4, p.c.batch), dim3(128), 0, st, p.c.pdl, p);
     if (e != cudaSuccess) return e;
     const dim3 grid((p.d.dim + S::kColumns - 1) / S::kColumns, p.d.heads, p.c.batch);
-    return launch_kernel(delta_scan_kernel<E, DP>, grid, dim3(S::kThreads + kPrepWarps * 32), S::kSmem, st, p.c.pdl, p);
+    return launch_kernel(delta_scan_kernel<DP>, grid, dim3(S::kThreads), S::kSmem, st, p.c.pdl, p);
+}
+
+int padded_dim(int dim)
+{
+    int dp = 16;
+    while (dp < dim) dp *= 2;
+    return dp;
 }
 
 template<typename E>
 cudaError_t scan_dispatch(const DeltaKernelParams& p, cudaStream_t st)
 {
-    if (p.d.dim <= 16) return scan_launch<E, 16>(p, st);
-    if (p.d.dim <= 32) return scan_launch<E, 32>(p, st);
-    if (p.d.dim <= 64) return scan_launch<E, 64>(p, st);
-    if (p.d.dim <= 128) return scan_launch<E, 128>(p, st);
-    return scan_launch<E, 256>(p, st);
+    switch (padded_dim(p.d.dim)) {
+        case 16: return scan_launch<E, 16>(p, st);
+        case 32: return scan_launch<E, 32>(p, st);
+        case 64: return scan_launch<E, 64>(p, st);
+        case 128: return scan_launch<E, 128>(p, st);
+        default: return scan_launch<E, 256>(p, st);
+    }
 }
 
 template<typename E>
@@ -321,35 +409,43 @@ bool valid(const DeltaRule& d, const MixerCall& c)
 
 }  // namespace
 
-int delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, float* decay_pre, float* o, cudaStream_t st)
+// decay pre-activations, later the outputs, to a multiple of four floats; behind them the records
+size_t delta_rule_scratch_floats(const DeltaRule& d)
 {
-    if (!valid(d, c) || !decay_pre || !o) return TM_ERR_UNSUPPORTED;
+    return (size_t)(d.heads * d.dim + 3) / 4 * 4 + (size_t)d.heads * (6 * padded_dim(d.dim) + 4);
+}
+
+int delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, float* scratch, cudaStream_t st)
+{
+    if (!valid(d, c) || !scratch) return TM_ERR_UNSUPPORTED;
     const size_t esz = c.f32 ? 4 : 2;
     DenseGemm    g;
     g.w = d.w2, g.ldw = d.w2_ld;
     g.x = static_cast<const char*>(c.proj) + d.w1_col * esz, g.ldx = c.proj_ld;
     g.tokens = c.tokens, g.n_out = d.heads * d.dim, g.k = d.rank;
-    g.ep.kind = DenseKind::kF32, g.ep.out = decay_pre, g.ep.out_ld = d.heads * d.dim;
+    g.ep.kind = DenseKind::kF32, g.ep.out = scratch, g.ep.out_ld = d.heads * d.dim;
     const int rc = dense_gemm(h, g, c.f32, st, c.pdl);
     if (rc != TM_OK) return rc;
-    const DeltaKernelParams p{d, c, decay_pre, o, 0};
+    float* const            records = scratch + (size_t)c.tokens * ((d.heads * d.dim + 3) / 4 * 4);
+    const DeltaKernelParams p{d, c, scratch, records, scratch, h->status, kMaxWaitCycles};
     cudaError_t             e = c.f32 ? scan_dispatch<float>(p, st) : scan_dispatch<__nv_bfloat16>(p, st);
     if (e == cudaSuccess) {
-        e = c.f32 ? launch_kernel(delta_finish_kernel<float>, dim3(c.tokens), dim3(256), 0, st, c.pdl, p) :
-                    launch_kernel(delta_finish_kernel<__nv_bfloat16>, dim3(c.tokens), dim3(256), 0, st, c.pdl, p);
+        const dim3 grid(c.tokens, (d.heads + 7) / 8);
+        e = c.f32 ? launch_kernel(delta_finish_kernel<float>, grid, dim3(256), 0, st, c.pdl, p) :
+                    launch_kernel(delta_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, c.pdl, p);
     }
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;
         return TM_ERR_CUDA;
     }
-    h->launches += 2;
+    h->launches += 3;
     return TM_OK;
 }
 
 int delta_rule_decode(tm_handle* h, const DeltaRule& d, const MixerCall& c, cudaStream_t st)
 {
     if (!valid(d, c)) return TM_ERR_UNSUPPORTED;
-    const DeltaKernelParams p{d, c, nullptr, nullptr, 0};
+    const DeltaKernelParams p{d, c, nullptr, nullptr, nullptr, h->status, kMaxWaitCycles};
     const cudaError_t       e = c.f32 ? step_dispatch<float>(p, st) : step_dispatch<__nv_bfloat16>(p, st);
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;

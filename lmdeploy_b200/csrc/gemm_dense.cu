@@ -6,14 +6,17 @@
 //   warp 1    allocates TMEM (two accumulators, so that one tile's epilogue overlaps the next tile's products); one lane
 //             issues four K16 MMAs per stage and commits the stage back to the loader
 //   warps 2-5 epilogue: lane = output column, so that every token's 32 columns leave in one contiguous store
-// With fewer tiles than SMs (a decode step) the k range of every tile is cut in `splits` parts: each part publishes its
-// fp32 tile in scratch, the last one to arrive adds them up in part order (nobody waits, the sum does not depend on the
-// order of arrival) and runs the epilogue.
+// Work split: whole tiles in full waves of one per CTA; the k blocks of the tiles that are left (all of them in a decode
+// step) are cut evenly over the CTAs, so that every SM streams the same number of bytes (stream-K).  A tile with several
+// CTAs: each publishes its fp32 part in scratch, the last one to arrive adds the parts up in CTA order (nobody waits, the
+// sum does not depend on the order of arrival) and runs the epilogue.
 // Every wait is bounded: a barrier that does not complete sets a status bit, the CTA drains its copies and leaves.
 #include "gemm_dense.h"
 #include "numeric.cuh"
 #include "tcgen05.cuh"
 #include "tm_b200.h"
+
+#include <algorithm>
 
 namespace tmb {
 namespace {
@@ -30,14 +33,16 @@ struct DenseShared {
     uint32_t tmem_base;
     int      dead;
     int      last;
-    int      pad;
+    int      stop;
     float    scale[kMaxTokens];
     float    red[4][kMaxTokens];
 };
 
 struct DenseTcParams {
     int           tokens, n_out, k_blocks;
-    int           token_tile, token_tiles, column_tiles, splits, units;
+    int           token_tile, token_tiles, tiles;
+    int           whole_waves;   // tiles a CTA takes as a whole: blockIdx, blockIdx + grid, ...
+    int           cut_ctas;      // CTAs that share the k blocks of the tiles behind them; at most two tiles each
     int           stages, tmem_columns;
     float*        scratch;
     int*          tickets;
@@ -123,15 +128,28 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
     tcgen05_after_sync();
     const uint32_t tmem = sh->tmem_base;
 
-    // unit u -> (column tile, token tile, part of the k range); token tiles vary fastest among tiles, so that the CTAs of
-    // a wave share weight tiles and activations in the L2
-    auto unit_of = [&](int u, int& ct, int& tt, int& kb0, int& kb1, int& part) {
-        const int tile = u / p.splits;
-        part           = u - tile * p.splits;
-        ct             = tile / p.token_tiles;
-        tt             = tile - ct * p.token_tiles;
-        kb0            = (int)((long long)part * p.k_blocks / p.splits);
-        kb1            = (int)((long long)(part + 1) * p.k_blocks / p.splits);
+    // segment i of this CTA -> tile and k blocks; false behind the last.  Token tiles vary fastest among tiles, so that
+    // the CTAs of a wave share weight tiles and activations in the L2.
+    const int       first_cut = p.whole_waves * (int)gridDim.x;
+    const long long cut_total = (long long)(p.tiles - first_cut) * p.k_blocks;
+    auto            cut       = [&](int c) { return (long long)c * cut_total / p.cut_ctas; };
+    auto            segment   = [&](int i, int& tile, int& kb0, int& kb1) {
+        if (i < p.whole_waves) {
+            tile = i * (int)gridDim.x + (int)blockIdx.x, kb0 = 0, kb1 = p.k_blocks;
+            return true;
+        }
+        if ((int)blockIdx.x >= p.cut_ctas || cut_total == 0) return false;
+        long long       begin = cut(blockIdx.x);
+        const long long end   = cut(blockIdx.x + 1);
+        for (int n = p.whole_waves; begin < end; ++n) {
+            const long long t = begin / p.k_blocks, stop = min(end, (t + 1) * p.k_blocks);
+            if (n == i) {
+                tile = first_cut + (int)t, kb0 = (int)(begin - t * p.k_blocks), kb1 = (int)(stop - t * p.k_blocks);
+                return true;
+            }
+            begin = stop;
+        }
+        return false;
     };
 
     if (warp == 0) {
@@ -144,10 +162,10 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                 tma_load_2d(base + s * stage_b, &w_map, kb * kKBlock, ct * kDenseTile, &sh->full[s]);
             };
             auto load_x = [&](int kb, int tt, int s) { tma_load_2d(base + s * stage_b + w_bytes, &x_map, kb * kKBlock, tt * NT, &sh->full[s]); };
-            for (int u = blockIdx.x; u < p.units && ok; u += gridDim.x) {
-                int ct, tt, kb0, kb1, part;
-                unit_of(u, ct, tt, kb0, kb1, part);
-                int kb = kb0;
+            int tile, kb0, kb1;
+            for (int seg = 0; ok && segment(seg, tile, kb0, kb1); ++seg) {
+                const int ct = tile / p.token_tiles, tt = tile - ct * p.token_tiles;
+                int       kb = kb0;
                 if (!waited) {
                     // weights are written by no kernel: the first boxes go out before the kernel ahead is complete
                     const int pre = min(ST, kb1 - kb0);
@@ -193,9 +211,8 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
             const uint32_t idesc = umma_idesc_bf16(kDenseTile, NT);
             int            it = 0, local = 0;
             bool           ok = true;
-            for (int u = blockIdx.x; u < p.units && ok; u += gridDim.x, ++local) {
-                int ct, tt, kb0, kb1, part;
-                unit_of(u, ct, tt, kb0, kb1, part);
+            int            tile, kb0, kb1;
+            for (; ok && segment(local, tile, kb0, kb1); ++local) {
                 const int a = local & 1;
                 if (local >= 2 && !mbar_wait(&sh->acc_empty[a], ((local >> 1) - 1) & 1, p.max_wait)) ok = false;
                 tcgen05_after_sync();
@@ -230,9 +247,9 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
         const int col  = q * 32 + lane;
         int       local = 0, scaled_tile = -1;
         bool      ok = true;
-        for (int u = blockIdx.x; u < p.units && ok; u += gridDim.x, ++local) {
-            int ct, tt, kb0, kb1, part;
-            unit_of(u, ct, tt, kb0, kb1, part);
+        int       tile, kb0, kb1;
+        for (; ok && segment(local, tile, kb0, kb1); ++local) {
+            const int ct = tile / p.token_tiles, tt = tile - ct * p.token_tiles;
             const int a    = local & 1;
             const int t0   = tt * NT;
             const int rows = min(NT, p.tokens - t0);
@@ -251,25 +268,35 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
             int okw = 1;
             if (lane == 0) okw = mbar_wait(&sh->acc_full[a], (local >> 1) & 1, p.max_wait) ? 1 : 0;
             okw = __shfl_sync(0xffffffffu, okw, 0);
-            if (!okw || *(volatile int*)&sh->dead) {
-                if (lane == 0) {
-                    if (!okw) atomicOr(p.status, kStatusGemmTmemWait);
-                    *(volatile int*)&sh->dead = 1;
-                }
+            if (!okw && lane == 0) {
+                atomicOr(p.status, kStatusGemmTmemWait);
+                *(volatile int*)&sh->dead = 1;
             }
-            // all four warps take the same way out (the barriers below are theirs together)
+            // one thread decides for all four warps, which share the barriers below
             named_bar_sync(kEpiBar, 128);
-            if (*(volatile int*)&sh->dead) {
+            if (etid == 0) sh->stop = *(volatile int*)&sh->dead;
+            named_bar_sync(kEpiBar, 128);
+            if (*(volatile int*)&sh->stop) {
                 ok = false;
                 break;
             }
             tcgen05_after_sync();
             const uint32_t acc    = tmem + ((uint32_t)(q * 32) << 16) + (uint32_t)(a * NT);
             bool           finish = true;
-            float*         slots  = nullptr;
-            if (p.splits > 1) {
-                slots       = p.scratch + (size_t)(u - part) * NT * kDenseTile;
-                float* mine = slots + (size_t)part * NT * kDenseTile;
+            int            parts = 1, part0 = 0;  // CTAs that share this tile: part0, part0 + 1, ...
+            const size_t   slot_floats = (size_t)NT * kDenseTile;
+            // slot of a CTA's part of the tile: two per CTA, the second for the tile its range ends in
+            auto slot_of = [&](int c) { return p.scratch + (size_t)(2 * c + (cut(c) / p.k_blocks == tile - first_cut ? 0 : 1)) * slot_floats; };
+            if (kb1 - kb0 < p.k_blocks) {
+                const long long lo = (long long)(tile - first_cut) * p.k_blocks, hi = lo + p.k_blocks - 1;
+                part0 = (int)(lo * p.cut_ctas / cut_total);
+                while (cut(part0 + 1) <= lo) ++part0;
+                while (cut(part0) > lo) --part0;
+                int last = (int)(hi * p.cut_ctas / cut_total);
+                while (cut(last + 1) <= hi) ++last;
+                while (cut(last) > hi) --last;
+                parts       = last - part0 + 1;
+                float* mine = slot_of(blockIdx.x);
                 for (int c0 = 0; c0 < rows; c0 += 16) {
                     float v[16];
                     tmem_load16(acc + c0, v);
@@ -281,9 +308,9 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                 __threadfence();
                 named_bar_sync(kEpiBar, 128);
                 if (etid == 0) {
-                    int*      ticket = p.tickets + (u - part) / p.splits;
+                    int*      ticket = p.tickets + (tile - first_cut);
                     const int before = atomicAdd(ticket, 1);
-                    sh->last         = before == p.splits - 1;
+                    sh->last         = before == parts - 1;
                     if (sh->last) *ticket = 0;
                 }
                 named_bar_sync(kEpiBar, 128);
@@ -295,11 +322,11 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                 for (int c0 = 0; c0 < rows; c0 += 16) {
                     float     v[16], sq[16];
                     const int live = min(16, rows - c0);
-                    if (p.splits > 1) {
+                    if (parts > 1) {
 #pragma unroll
                         for (int i = 0; i < 16; ++i) v[i] = 0.f;
-                        for (int s = 0; s < p.splits; ++s) {
-                            const float* src = slots + ((size_t)s * NT + c0) * kDenseTile + col;
+                        for (int c = part0; c < part0 + parts; ++c) {
+                            const float* src = slot_of(c) + (size_t)c0 * kDenseTile + col;
 #pragma unroll
                             for (int i = 0; i < 16; ++i) {
                                 if (i < live) v[i] += __ldcg(src + (size_t)i * kDenseTile);
@@ -434,21 +461,6 @@ cudaError_t dense_prepare(int max_smem)
 }
 const KernelPreparation g_prepare(dense_prepare);
 
-// parts of the k range per tile: as many as fill the SMs evenly, each of at least four k blocks
-int choose_splits(int tiles, int k_blocks, int sms, size_t tile_bytes, size_t scratch_bytes)
-{
-    if (tiles >= 4 * sms) return 1;
-    int    best      = 1;
-    double best_cost = 1e30;
-    for (int s = 1; s <= 16 && (s == 1 || k_blocks / s >= 4); ++s) {
-        if (s > 1 && (size_t)tiles * s * tile_bytes > scratch_bytes) break;
-        const int    waves = (tiles * s + sms - 1) / sms;
-        const double cost  = waves * ((double)((k_blocks + s - 1) / s) + 3.0) + (s > 1 ? 4.0 + 0.5 * s : 0.0);
-        if (cost < best_cost - 1e-9) best_cost = cost, best = s;
-    }
-    return best;
-}
-
 int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
 {
     static const EncodeTiled encode = lookup_encode_tiled();
@@ -461,17 +473,20 @@ int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
     p.k_blocks     = (g.k + kKBlock - 1) / kKBlock;
     p.token_tile   = g.tokens >= kMaxTokens ? kMaxTokens : (g.tokens + 15) / 16 * 16;
     p.token_tiles  = (g.tokens + p.token_tile - 1) / p.token_tile;
-    p.column_tiles = (g.n_out + kDenseTile - 1) / kDenseTile;
+    p.tiles        = (g.n_out + kDenseTile - 1) / kDenseTile * p.token_tiles;
     p.tmem_columns = 32;
     while (p.tmem_columns < 2 * p.token_tile) p.tmem_columns *= 2;
     const size_t stage_b = (size_t)kDenseTile * 128 + (size_t)p.token_tile * 128;
     p.stages             = (int)(((size_t)h->max_smem - 1024 - sizeof(DenseShared)) / stage_b);
     if (p.stages > kMaxStages) p.stages = kMaxStages;
     if (p.stages < 2) return TM_ERR_UNSUPPORTED;
-    const int tiles = p.column_tiles * p.token_tiles;
-    p.splits        = choose_splits(tiles, p.k_blocks, h->sm_count, (size_t)p.token_tile * kDenseTile * 4, h->scratch_bytes);
-    if (tiles > (int)h->counter_ints) p.splits = 1;
-    p.units    = tiles * p.splits;
+    // whole tiles in full waves, the rest cut; each CTA of the cut part gets at least four k blocks
+    const int sms = h->sm_count;
+    p.whole_waves = p.tiles / sms;
+    int rest      = p.tiles - p.whole_waves * sms;
+    p.cut_ctas    = (int)std::min<long long>(sms, std::max<long long>(1, (long long)rest * p.k_blocks / 4));
+    if (p.cut_ctas < rest || (size_t)2 * p.cut_ctas * p.token_tile * kDenseTile * 4 > h->scratch_bytes) p.cut_ctas = std::max(1, rest);
+    const int grid_ctas = p.whole_waves > 0 ? sms : std::max(1, p.cut_ctas);
     p.scratch  = static_cast<float*>(h->scratch);
     p.tickets  = h->counters;
     p.status   = h->status;
@@ -481,7 +496,7 @@ int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
     if (!encode_rows(encode, &w_map, g.w, g.n_out, g.k, g.ldw, kDenseTile)) return TM_ERR_CUDA;
     if (!encode_rows(encode, &x_map, g.x, g.tokens, g.k, g.ldx, p.token_tile)) return TM_ERR_CUDA;
     const size_t smem = 1024 + (size_t)p.stages * stage_b + sizeof(DenseShared);
-    const dim3   grid(p.units < h->sm_count ? p.units : h->sm_count);
+    const dim3   grid(grid_ctas);
     const cudaError_t e = launch_kernel(dense_tc_kernel, grid, dim3(kThreads), smem, st, pdl, p, w_map, x_map);
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;

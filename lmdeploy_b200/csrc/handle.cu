@@ -132,6 +132,7 @@ extern "C" int tm_destroy(tm_handle* h)
     if (h->attn_scratch) cudaFree(h->attn_scratch);
     if (h->attn_counters) cudaFree(h->attn_counters);
     if (h->status) cudaFree(h->status);
+    if (h->op_buffer) cudaFree(h->op_buffer);
     cudaSetDevice(prev);
     delete h;
     return TM_OK;

@@ -18,6 +18,8 @@ struct tm_handle {
     size_t             attn_scratch_bytes = 0;
     int*               attn_counters   = nullptr;
     size_t             attn_counter_ints = 0;
+    void*              op_buffer       = nullptr;  // device copies and scratch of single operator calls, grown on demand
+    size_t             op_buffer_bytes = 0;
     unsigned*          status          = nullptr;  // device status word (bounded waits)
     int                last_cuda_error = 0;
     unsigned long long launches        = 0;

@@ -61,8 +61,9 @@ struct DeltaRule {
     size_t       state_off = 0;        // bytes in the slab: float [head][key dim][value dim]
     int          r_col = 0, k_col = 0, v_col = 0, a_col = 0, g_col = 0, w1_col = 0;  // columns of the projections; w1 after tanh
 };
-// scratch of a prefill: decay pre-activations and outputs, fp32 [tokens][heads * dim] each
-int delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, float* decay_pre, float* o, cudaStream_t st);
+// scratch of a prefill, fp32: so many floats per token
+size_t delta_rule_scratch_floats(const DeltaRule& d);
+int    delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, float* scratch, cudaStream_t st);
 int delta_rule_decode(tm_handle* h, const DeltaRule& d, const MixerCall& c, cudaStream_t st);
 
 }  // namespace tmb

@@ -51,6 +51,45 @@ __global__ void __launch_bounds__(128) window_write_kernel(const WindowKernelPar
     }
 }
 
+// The same for bf16 heads of a multiple of 8 dimensions: 16 bytes per access
+__global__ void __launch_bounds__(256) window_write8_kernel(const WindowKernelParams p)
+{
+    using E = __nv_bfloat16;
+    __shared__ float cs[kMaxHeadDim / 2], sn[kMaxHeadDim / 2];
+    pdl_wait();
+    pdl_launch_dependents();
+    const WindowAttention& a = p.a;
+    const SeqSpan          s = p.c.spans[blockIdx.y];
+    if ((int)blockIdx.x >= s.n || !s.live) return;
+    const int pos = s.history + blockIdx.x;
+    E*        row = static_cast<E*>(p.c.proj) + (size_t)(s.tok0 + blockIdx.x) * p.c.proj_ld;
+    for (int i = threadIdx.x; i < a.rot_dims / 2; i += blockDim.x) sincosf((float)pos * a.inv_freq[i], &sn[i], &cs[i]);
+    __syncthreads();
+    const int slot = pos % a.ring, per = a.dim / 8, per_v = a.vdim / 8;
+    const int n_qk = (a.heads + a.kv_heads) * per, total = n_qk + a.kv_heads * per_v;
+    for (int w = threadIdx.x; w < total; w += blockDim.x) {
+        if (w >= n_qk) {
+            const int x = w - n_qk, g = x / per_v, d = (x - g * per_v) * 8;
+            *reinterpret_cast<uint4*>(slab_rows<E>(s.slab, a.v_off) + ((size_t)g * a.ring + slot) * a.vdim + d) =
+                *reinterpret_cast<const uint4*>(row + a.v_col + g * a.vdim + d);
+            continue;
+        }
+        const int  hh = w / per, d = (w - hh * per) * 8;
+        const bool is_q = hh < a.heads;
+        if (is_q && d >= a.rot_dims) continue;  // stays where it is
+        E*    src = row + (is_q ? a.q_col + hh * a.dim : a.k_col + (hh - a.heads) * a.dim) + d;
+        E*    dst = is_q ? src : slab_rows<E>(s.slab, a.k_off) + ((size_t)(hh - a.heads) * a.ring + slot) * a.dim + d;
+        uint4 v   = *reinterpret_cast<const uint4*>(src);
+        auto  turn = [&](uint32_t x, int i) {
+            if (2 * i >= a.rot_dims) return x;
+            const float u = bf16_lo(x), y = bf16_hi(x), c = cs[i], z = sn[i];
+            return pack_bf16(u * c - y * z, y * c + u * z);
+        };
+        v.x = turn(v.x, d / 2), v.y = turn(v.y, d / 2 + 1), v.z = turn(v.z, d / 2 + 2), v.w = turn(v.w, d / 2 + 3);
+        *reinterpret_cast<uint4*>(dst) = v;
+    }
+}
+
 // One CTA per (block that this launch completes, kv head, sequence): the mean of its keys and of its values as cached.
 template<typename E>
 __global__ void __launch_bounds__(128) window_pool_kernel(const WindowKernelParams p)
@@ -194,7 +233,11 @@ bool valid(const WindowAttention& a, const MixerCall& c)
 template<typename E>
 int write_and_pool(tm_handle* h, const WindowKernelParams& p, cudaStream_t st)
 {
-    if (launch_kernel(window_write_kernel<E>, dim3(p.c.max_n, p.c.batch), dim3(128), 0, st, p.c.pdl, p) != cudaSuccess) return TM_ERR_CUDA;
+    const bool wide = sizeof(E) == 2 && p.a.dim % 8 == 0 && p.a.vdim % 8 == 0 && p.c.proj_ld % 8 == 0 && p.a.q_col % 8 == 0 && p.a.k_col % 8 == 0
+                      && p.a.v_col % 8 == 0;
+    const cudaError_t e = wide ? launch_kernel(window_write8_kernel, dim3(p.c.max_n, p.c.batch), dim3(256), 0, st, p.c.pdl, p) :
+                                 launch_kernel(window_write_kernel<E>, dim3(p.c.max_n, p.c.batch), dim3(128), 0, st, p.c.pdl, p);
+    if (e != cudaSuccess) return TM_ERR_CUDA;
     ++h->launches;
     if (p.a.pool > 0) {
         const dim3 grid((p.c.max_n + p.a.pool - 1) / p.a.pool, p.a.kv_heads, p.c.batch);
