@@ -730,7 +730,7 @@ def device_ms(fn, stream, steps, warmup, flush=None):
     total = 0.0
     for _ in range(steps):
         if flush is not None:
-            flush.zero_()
+            flush.sum()               # reads more than L2 holds (a write would leave lines whose write-back the kernel pays for)
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         e0.record(stream)
         fn()
@@ -882,7 +882,7 @@ def run_rumazen_workload(args, rank, world, device):
     K, Wm, L = min(args.steps, 32), args.warmup, 8
     cfg, peaks = rumazen_config(L), measured_peaks()
     stream = torch.cuda.Stream(device)
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=device)   # larger than L2
+    flush = torch.zeros(64 << 20, dtype=torch.int32, device=device)   # 256 MB, larger than L2
     rng = np.random.default_rng(5 + rank)
     sampler = ClockSampler(device)
     res, launches = {"rumazen": {}, "llama_w4a16": {}}, 0

@@ -690,7 +690,7 @@ typedef struct tm_window_attention_params {
     int          q_col, k_col, v_col, g_col;
 } tm_window_attention_params;
 TM_API int tm_window_attention(tm_handle* h, const tm_window_attention_params* a, const tm_mixer_call* c, void* stream);
-/* Generalised delta rule, fp32 state float [head][dim][dim] (zero at history 0):
+/* Generalised delta rule, fp32 state float [head][value dim][key dim] (zero at history 0):
  *   w = exp(-decay_scale * sigmoid(w2 . w1 + w0)), a = sigmoid(a + a_bias), u = k / sqrt(k.k + unit_eps)
  *   S <- diag(w) S - (a u)(u^T S) + k v^T,   o = S^T r;   out = o / rms(o) * norm * sigmoid(g) per head */
 typedef struct tm_delta_rule_params {

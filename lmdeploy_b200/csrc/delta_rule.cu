@@ -3,6 +3,7 @@
 //     S <- diag(w) S - (a u) (u^T S) + k v^T          o = S^T r
 // (both terms read the old S), all of it in fp32.  The columns of S (value channels) never meet, which is what the
 // prefill kernel splits over lanes, warps and CTAs; the keys' side (u, a u, w, k, r) is shared by all columns of a head.
+// A column is contiguous in memory.
 #include "common.cuh"
 #include "gemm_dense.h"
 #include "mixers.h"
@@ -141,7 +142,7 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int r = row_of(i);
-        st[i]       = s.history > 0 && r < dim && col < dim ? state[(size_t)r * dim + col] : 0.f;
+        st[i]       = s.history > 0 && r < dim && col < dim ? state[(size_t)col * dim + r] : 0.f;
     }
     float* o_out = p.o + (size_t)s.tok0 * d.heads * dim + h * dim + col;
     bool   ok    = true;
@@ -212,7 +213,7 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int r = row_of(i);
-        if (r < dim && col < dim) state[(size_t)r * dim + col] = st[i];
+        if (r < dim && col < dim) state[(size_t)col * dim + r] = st[i];
     }
 }
 
@@ -247,117 +248,162 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const DeltaKernelPara
 }
 
 // One new token per sequence, one CTA per (head, sequence): decay projection, step, head norm and gate in one kernel.
-// The state passes through registers once: thread = (column, every RG-th row).
-// ROWS: state elements per thread, held in registers between the two products; 0: read again for the second (large heads).
-template<typename E, int ROWS, int kStepThreads>
-__global__ void __launch_bounds__(kStepThreads) delta_step_kernel(const DeltaKernelParams p)
+// Lanes share a column of S as in the scan; the state passes through registers once, and its reads are under way before
+// anything else is known.
+template<int DP>
+struct StepShape {
+    static constexpr int  kThreads = 256, kLanes = DP / 8, kColumns = kThreads / kLanes;
+    static constexpr int  kPasses = (DP + kColumns - 1) / kColumns;  // columns per thread
+    static constexpr bool kHeld   = kPasses <= 8;                    // all of them in registers from the start
+    static constexpr int  kPer    = kThreads / DP;                   // threads that share a channel's decay projection
+};
+
+template<typename E, int DP>
+__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaKernelParams p)
 {
-    __shared__ float u[kMaxDim], au[kMaxDim], w[kMaxDim], k[kMaxDim], r[kMaxDim], v[kMaxDim];
-    __shared__ float red[kStepThreads], zs[kMaxDim], warp_red[kStepThreads / 32];
-    const DeltaRule& d   = p.d;
-    const int        h   = blockIdx.x, dim = d.dim;
+    using S = StepShape<DP>;
+    constexpr int kVec = 16 / sizeof(E);
+    __shared__ __align__(16) float u[DP], b[DP], w[DP], k[DP], r[DP];
+    __shared__ float v[DP], y[DP], red[8];
+    const DeltaRule& d    = p.d;
+    const int        h    = blockIdx.x, dim = d.dim, n = h * dim;
     const int        tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const SeqSpan    s    = p.c.spans[blockIdx.y];
+    const int        part = tid % S::kLanes, lc = tid / S::kLanes;
+    float*           state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * dim;
+    const bool       quad = dim % 4 == 0, old = s.live && s.history > 0;
+    float            st[S::kHeld ? S::kPasses : 1][8];
+    auto load = [&](int pass, float (&x)[8]) {
+        const int col = pass * S::kColumns + lc;
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+            const int    r0  = q * (DP / 2) + 4 * part;
+            const float* src = state + (size_t)col * dim + r0;
+            if (old && col < dim && quad && r0 < dim) {
+                const float4 f = *reinterpret_cast<const float4*>(src);
+                x[4 * q] = f.x, x[4 * q + 1] = f.y, x[4 * q + 2] = f.z, x[4 * q + 3] = f.w;
+            }
+            else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) x[4 * q + e] = old && col < dim && r0 + e < dim ? src[e] : 0.f;
+            }
+        }
+    };
+    // written by this layer's kernel of an earlier step: nothing of this step touches it before
+    if (S::kHeld) {
+#pragma unroll
+        for (int i = 0; i < S::kPasses; ++i) load(i, st[i]);
+    }
+    // constants of this thread's channel
+    const int  c  = tid / S::kPer, sub = tid % S::kPer;
+    const bool on = c < dim;
+    uint4      w2[4];
+    const E*   w2_row = static_cast<const E*>(d.w2) + (size_t)(n + (on ? c : 0)) * d.w2_ld;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int m = (sub + i * S::kPer) * kVec;
+        w2[i]       = m < d.rank ? *reinterpret_cast<const uint4*>(w2_row + m) : make_uint4(0, 0, 0, 0);
+    }
+    const float w0 = on ? d.w0[n + c] : 0.f, ab = on ? d.a_bias[n + c] : 0.f, nw = tid < dim ? d.norm[n + tid] : 0.f;
     pdl_wait();
     pdl_launch_dependents();
-    const SeqSpan s = p.c.spans[blockIdx.y];
     if (!s.live) return;
-    const int    groups = kStepThreads / dim;  // row groups; dim <= 256 leaves at least two
-    const int    col = tid % dim, rg = tid / dim;
-    const bool   on  = rg < groups;
-    float*       state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * dim;
-    float        st[ROWS > 0 ? ROWS : 1];
+    const E*    row = static_cast<const E*>(p.c.proj) + (size_t)s.tok0 * p.c.proj_ld;
+    const float kc = on ? to_f32(row[d.k_col + n + c]) : 0.f, rc = on ? to_f32(row[d.r_col + n + c]) : 0.f;
+    const float vc = on ? to_f32(row[d.v_col + n + c]) : 0.f, ac = on ? to_f32(row[d.a_col + n + c]) : 0.f;
+    const float gate = tid < dim ? to_f32(row[d.g_col + n + tid]) : 0.f;
+    // ---- decay pre-activation: w2 . tanh(w1 h)
+    float x = 0.f;
+    for (int i = 0;; ++i) {
+        const int m = (sub + i * S::kPer) * kVec;
+        if (m >= d.rank) break;
+        const uint4 a = i == 0 ? w2[0] : i == 1 ? w2[1] : i == 2 ? w2[2] : i == 3 ? w2[3] : *reinterpret_cast<const uint4*>(w2_row + m);
+        const E*    wa = reinterpret_cast<const E*>(&a);
 #pragma unroll
-    for (int i = 0; i < ROWS; ++i) {
-        const int row = rg + i * groups;
-        st[i]         = on && row < dim && s.history > 0 ? state[(size_t)row * dim + col] : 0.f;
+        for (int e = 0; e < kVec; ++e) {
+            if (m + e < d.rank) x = fmaf(to_f32(wa[e]), to_f32(row[d.w1_col + m + e]), x);
+        }
     }
-    const E* row = static_cast<const E*>(p.c.proj) + (size_t)s.tok0 * p.c.proj_ld;
-    float    ksq = 0.f;
-    for (int c = tid; c < dim; c += kStepThreads) {
-        k[c] = to_f32(row[d.k_col + h * dim + c]);
-        v[c] = to_f32(row[d.v_col + h * dim + c]);
-        r[c] = to_f32(row[d.r_col + h * dim + c]);
-        ksq += k[c] * k[c];
+    // the threads of a channel are neighbours; up to 16 of them
+#pragma unroll
+    for (int m = 1; m < S::kPer; m *= 2) x += __shfl_xor_sync(0xffffffffu, x, m);
+    const float ksq = warp_sum(sub == 0 ? kc * kc : 0.f);
+    if (lane == 0) red[warp] = ksq;
+    __syncthreads();
+    if (sub == 0 && c < DP) {
+        float total = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) total += red[i];
+        const float uc = kc / sqrtf(total + d.unit_eps);
+        u[c] = uc, b[c] = sigmoid_f32(ac + ab) * uc, w[c] = on ? expf(-d.decay_scale * sigmoid_f32(x + w0)) : 0.f;
+        k[c] = kc, r[c] = rc, v[c] = vc;
     }
-    ksq = warp_sum(ksq);
-    if (lane == 0) warp_red[warp] = ksq;
-    // decay: w2 . tanh(w1 h), a warp per channel
-    const E* w1 = row + d.w1_col;
-    for (int c = warp; c < dim; c += kStepThreads / 32) {
-        const E* w2 = static_cast<const E*>(d.w2) + (size_t)(h * dim + c) * d.w2_ld;
-        float    x  = 0.f;
-        for (int m = lane; m < d.rank; m += 32) x = fmaf(to_f32(w2[m]), to_f32(w1[m]), x);
-        x = warp_sum(x);
-        if (lane == 0) w[c] = expf(-d.decay_scale * sigmoid_f32(x + d.w0[h * dim + c]));
+    __syncthreads();
+    // ---- the step
+    auto vec = [&](const float* a, float (&f)[8]) {
+        const float4 lo = *reinterpret_cast<const float4*>(a + 4 * part), hi = *reinterpret_cast<const float4*>(a + DP / 2 + 4 * part);
+        f[0] = lo.x, f[1] = lo.y, f[2] = lo.z, f[3] = lo.w, f[4] = hi.x, f[5] = hi.y, f[6] = hi.z, f[7] = hi.w;
+    };
+    float uu[8], bb[8], ww[8], kk[8], rr[8];
+    vec(u, uu), vec(b, bb), vec(w, ww), vec(k, kk), vec(r, rr);
+    float sq = 0.f;
+#pragma unroll
+    for (int pass = 0; pass < S::kPasses; ++pass) {
+        float now[8];
+        if (S::kHeld) {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) now[i] = st[S::kHeld ? pass : 0][i];
+        }
+        else {
+            load(pass, now);
+        }
+        const int   col = pass * S::kColumns + lc;
+        const float vj  = col < DP ? v[min(col, DP - 1)] : 0.f;
+        float       z = 0.f, o = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) z = fmaf(uu[i], now[i], z);
+#pragma unroll
+        for (int m = S::kLanes / 2; m >= 1; m >>= 1) z += __shfl_xor_sync(0xffffffffu, z, m);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            now[i] = fmaf(ww[i], now[i], fmaf(kk[i], vj, -bb[i] * z));
+            o      = fmaf(rr[i], now[i], o);
+        }
+#pragma unroll
+        for (int m = S::kLanes / 2; m >= 1; m >>= 1) o += __shfl_xor_sync(0xffffffffu, o, m);
+        if (col < dim) {
+#pragma unroll
+            for (int q = 0; q < 2; ++q) {
+                const int r0  = q * (DP / 2) + 4 * part;
+                float*    dst = state + (size_t)col * dim + r0;
+                if (quad && r0 < dim) {
+                    *reinterpret_cast<float4*>(dst) = make_float4(now[4 * q], now[4 * q + 1], now[4 * q + 2], now[4 * q + 3]);
+                }
+                else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        if (r0 + e < dim) dst[e] = now[4 * q + e];
+                    }
+                }
+            }
+            if (part == 0) {
+                y[col] = o;
+                sq += o * o;
+            }
+        }
     }
+    sq = warp_sum(sq);
+    __syncthreads();  // the first use of red is over for everybody
+    if (lane == 0) red[warp] = sq;
     __syncthreads();
     float total = 0.f;
 #pragma unroll
-    for (int i = 0; i < kStepThreads / 32; ++i) total += warp_red[i];
-    const float inv = 1.f / sqrtf(total + d.unit_eps);
-    for (int c = tid; c < dim; c += kStepThreads) {
-        u[c]  = k[c] * inv;
-        au[c] = sigmoid_f32(to_f32(row[d.a_col + h * dim + c]) + d.a_bias[h * dim + c]) * u[c];
-    }
-    __syncthreads();
-    float z = 0.f;
-#pragma unroll
-    for (int i = 0; i < ROWS; ++i) {
-        const int x = rg + i * groups;
-        if (x < dim) z = fmaf(u[x], st[i], z);
-    }
-    if (ROWS == 0 && on && s.history > 0) {
-        for (int x = rg; x < dim; x += groups) z = fmaf(u[x], state[(size_t)x * dim + col], z);
-    }
-    red[tid] = on ? z : 0.f;
-    __syncthreads();
-    if (tid < dim) {
-        float x = 0.f;
-        for (int g = 0; g < groups; ++g) x += red[g * dim + tid];
-        zs[tid] = x;
-    }
-    __syncthreads();
-    float o = 0.f;
-    if (on) {
-        z = zs[col];
-#pragma unroll
-        for (int i = 0; i < ROWS; ++i) {
-            const int x = rg + i * groups;
-            if (x < dim) {
-                st[i] = fmaf(w[x], st[i], fmaf(k[x], v[col], -au[x] * z));
-                o     = fmaf(r[x], st[i], o);
-                state[(size_t)x * dim + col] = st[i];
-            }
-        }
-        if (ROWS == 0) {
-            for (int x = rg; x < dim; x += groups) {
-                const float old = s.history > 0 ? state[(size_t)x * dim + col] : 0.f;
-                const float now = fmaf(w[x], old, fmaf(k[x], v[col], -au[x] * z));
-                o               = fmaf(r[x], now, o);
-                state[(size_t)x * dim + col] = now;
-            }
-        }
-    }
-    red[tid] = on ? o : 0.f;
-    __syncthreads();
-    float y = 0.f;
-    if (tid < dim) {
-        for (int g = 0; g < groups; ++g) y += red[g * dim + tid];
-    }
-    const float sq = warp_sum(y * y);
-    if (lane == 0) warp_red[warp] = sq;
-    __syncthreads();
-    total = 0.f;
-#pragma unroll
-    for (int i = 0; i < kStepThreads / 32; ++i) total += warp_red[i];
-    const float rms = 1.f / sqrtf(total / (float)dim + d.norm_eps);
+    for (int i = 0; i < 8; ++i) total += red[i];
+    const float inv = 1.f / sqrtf(total / (float)dim + d.norm_eps);
     E*          out = static_cast<E*>(p.c.out) + (size_t)s.tok0 * p.c.out_ld;
-    if (tid < dim) {
-        const int n = h * dim + tid;
-        out[n]      = from_f32<E>(y * rms * d.norm[n] * sigmoid_f32(to_f32(row[d.g_col + n])));
-    }
+    if (tid < dim) out[n + tid] = from_f32<E>(y[tid] * inv * nw * sigmoid_f32(gate));
     if (h == d.heads - 1) {
-        for (int n = d.heads * dim + tid; n < p.c.out_pad; n += kStepThreads) out[n] = from_f32<E>(0.f);
+        for (int i = d.heads * dim + tid; i < p.c.out_pad; i += S::kThreads) out[i] = from_f32<E>(0.f);
     }
 }
 
@@ -395,11 +441,14 @@ cudaError_t scan_dispatch(const DeltaKernelParams& p, cudaStream_t st)
 template<typename E>
 cudaError_t step_dispatch(const DeltaKernelParams& p, cudaStream_t st)
 {
-    const dim3 grid(p.d.heads, p.c.batch);
-    auto       rows = [&](int threads) { return (p.d.dim + threads / p.d.dim - 1) / (threads / p.d.dim); };
-    if (rows(512) <= 8) return launch_kernel(delta_step_kernel<E, 8, 512>, grid, dim3(512), 0, st, p.c.pdl, p);
-    if (rows(1024) <= 19) return launch_kernel(delta_step_kernel<E, 19, 1024>, grid, dim3(1024), 0, st, p.c.pdl, p);
-    return launch_kernel(delta_step_kernel<E, 0, 1024>, grid, dim3(1024), 0, st, p.c.pdl, p);
+    const dim3 grid(p.d.heads, p.c.batch), block(256);
+    switch (padded_dim(p.d.dim)) {
+        case 16: return launch_kernel(delta_step_kernel<E, 16>, grid, block, 0, st, p.c.pdl, p);
+        case 32: return launch_kernel(delta_step_kernel<E, 32>, grid, block, 0, st, p.c.pdl, p);
+        case 64: return launch_kernel(delta_step_kernel<E, 64>, grid, block, 0, st, p.c.pdl, p);
+        case 128: return launch_kernel(delta_step_kernel<E, 128>, grid, block, 0, st, p.c.pdl, p);
+        default: return launch_kernel(delta_step_kernel<E, 256>, grid, block, 0, st, p.c.pdl, p);
+    }
 }
 
 bool valid(const DeltaRule& d, const MixerCall& c)

@@ -6,9 +6,8 @@
 //   warp 1    allocates TMEM (two accumulators, so that one tile's epilogue overlaps the next tile's products); one lane
 //             issues four K16 MMAs per stage and commits the stage back to the loader
 //   warps 2-5 epilogue: lane = output column, so that every token's 32 columns leave in one contiguous store
-// Work split: whole tiles in full waves of one per CTA; the k blocks of the tiles that are left (all of them in a decode
-// step) are cut evenly over the CTAs, so that every SM streams the same number of bytes (stream-K).  A tile with several
-// CTAs: each publishes its fp32 part in scratch, the last one to arrive adds the parts up in CTA order (nobody waits, the
+// Work split (choose_plan): whole tiles dealt out to the CTAs; or, with few tiles (a decode step), the k blocks of all tiles
+// cut evenly over the CTAs, so that every SM streams the same number of bytes (stream-K).  A tile with several CTAs: each publishes its fp32 part in scratch, the last one to arrive adds the parts up in CTA order (nobody waits, the
 // sum does not depend on the order of arrival) and runs the epilogue.
 // Every wait is bounded: a barrier that does not complete sets a status bit, the CTA drains its copies and leaves.
 #include "gemm_dense.h"
@@ -41,8 +40,8 @@ struct DenseShared {
 struct DenseTcParams {
     int           tokens, n_out, k_blocks;
     int           token_tile, token_tiles, tiles;
-    int           whole_waves;   // tiles a CTA takes as a whole: blockIdx, blockIdx + grid, ...
-    int           cut_ctas;      // CTAs that share the k blocks of the tiles behind them; at most two tiles each
+    int           grid_tiles;  // tiles dealt out as a whole (all of them, or none)
+    int           cut_ctas;    // > 0: CTAs that share the k blocks of all tiles evenly
     int           stages, tmem_columns;
     float*        scratch;
     int*          tickets;
@@ -130,26 +129,17 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
 
     // segment i of this CTA -> tile and k blocks; false behind the last.  Token tiles vary fastest among tiles, so that
     // the CTAs of a wave share weight tiles and activations in the L2.
-    const int       first_cut = p.whole_waves * (int)gridDim.x;
-    const long long cut_total = (long long)(p.tiles - first_cut) * p.k_blocks;
+    const long long cut_total = (long long)p.tiles * p.k_blocks;
     auto            cut       = [&](int c) { return (long long)c * cut_total / p.cut_ctas; };
     auto            segment   = [&](int i, int& tile, int& kb0, int& kb1) {
-        if (i < p.whole_waves) {
+        if (p.cut_ctas == 0) {
             tile = i * (int)gridDim.x + (int)blockIdx.x, kb0 = 0, kb1 = p.k_blocks;
-            return true;
+            return tile < p.grid_tiles;
         }
-        if ((int)blockIdx.x >= p.cut_ctas || cut_total == 0) return false;
-        long long       begin = cut(blockIdx.x);
-        const long long end   = cut(blockIdx.x + 1);
-        for (int n = p.whole_waves; begin < end; ++n) {
-            const long long t = begin / p.k_blocks, stop = min(end, (t + 1) * p.k_blocks);
-            if (n == i) {
-                tile = first_cut + (int)t, kb0 = (int)(begin - t * p.k_blocks), kb1 = (int)(stop - t * p.k_blocks);
-                return true;
-            }
-            begin = stop;
-        }
-        return false;
+        const long long begin = cut(blockIdx.x), end = cut(blockIdx.x + 1), t = begin / p.k_blocks + i;
+        if (t * p.k_blocks >= end) return false;
+        tile = (int)t, kb0 = (int)(max(begin, t * p.k_blocks) - t * p.k_blocks), kb1 = (int)(min(end, (t + 1) * p.k_blocks) - t * p.k_blocks);
+        return true;
     };
 
     if (warp == 0) {
@@ -286,9 +276,9 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
             int            parts = 1, part0 = 0;  // CTAs that share this tile: part0, part0 + 1, ...
             const size_t   slot_floats = (size_t)NT * kDenseTile;
             // slot of a CTA's part of the tile: two per CTA, the second for the tile its range ends in
-            auto slot_of = [&](int c) { return p.scratch + (size_t)(2 * c + (cut(c) / p.k_blocks == tile - first_cut ? 0 : 1)) * slot_floats; };
+            auto slot_of = [&](int c) { return p.scratch + (size_t)(2 * c + (cut(c) / p.k_blocks == tile ? 0 : 1)) * slot_floats; };
             if (kb1 - kb0 < p.k_blocks) {
-                const long long lo = (long long)(tile - first_cut) * p.k_blocks, hi = lo + p.k_blocks - 1;
+                const long long lo = (long long)tile * p.k_blocks, hi = lo + p.k_blocks - 1;
                 part0 = (int)(lo * p.cut_ctas / cut_total);
                 while (cut(part0 + 1) <= lo) ++part0;
                 while (cut(part0) > lo) --part0;
@@ -308,7 +298,7 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                 __threadfence();
                 named_bar_sync(kEpiBar, 128);
                 if (etid == 0) {
-                    int*      ticket = p.tickets + (tile - first_cut);
+                    int*      ticket = p.tickets + tile;
                     const int before = atomicAdd(ticket, 1);
                     sh->last         = before == parts - 1;
                     if (sh->last) *ticket = 0;
@@ -325,11 +315,20 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                     if (parts > 1) {
 #pragma unroll
                         for (int i = 0; i < 16; ++i) v[i] = 0.f;
-                        for (int c = part0; c < part0 + parts; ++c) {
-                            const float* src = slot_of(c) + (size_t)c0 * kDenseTile + col;
+                        // four parts on their way at a time (a row beyond `live` is scratch of the same slot)
+                        for (int c = part0; c < part0 + parts; c += 4) {
+                            float x[4][16];
 #pragma unroll
-                            for (int i = 0; i < 16; ++i) {
-                                if (i < live) v[i] += __ldcg(src + (size_t)i * kDenseTile);
+                            for (int j = 0; j < 4; ++j) {
+                                const float* src = slot_of(min(c + j, part0 + parts - 1)) + (size_t)c0 * kDenseTile + col;
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) x[j][i] = __ldcg(src + (size_t)i * kDenseTile);
+                            }
+#pragma unroll
+                            for (int j = 0; j < 4; ++j) {
+                                if (c + j >= part0 + parts) break;
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] += x[j][i];
                             }
                         }
                     }
@@ -461,6 +460,29 @@ cudaError_t dense_prepare(int max_smem)
 }
 const KernelPreparation g_prepare(dense_prepare);
 
+struct Plan {
+    int  token_tile;
+    bool cut;
+};
+// Tile height and whether the tiles are cut, by a model of the launch's time in microseconds: a k block takes what its
+// bytes or its products need, cutting costs the exchange of the parts.
+Plan choose_plan(int tokens, int n_out, int k_blocks, int sms)
+{
+    Plan   best{0, false};
+    double best_cost = 1e30;
+    const int first = tokens >= kMaxTokens ? kMaxTokens : (tokens + 15) / 16 * 16;
+    const int last  = tokens >= kMaxTokens ? 128 : first;
+    for (int nt = first; nt >= last; nt -= 16) {
+        const long long tiles = (long long)((n_out + kDenseTile - 1) / kDenseTile) * ((tokens + nt - 1) / nt);
+        const double    block = std::max(0.4, 0.45 * nt / 256);
+        const double    whole = (double)((tiles + sms - 1) / sms) * (k_blocks * block + 1.0);
+        const double    cut   = (double)tiles * k_blocks / sms * block + 3.0 + 0.06 * nt;
+        if (whole < best_cost - 1e-9) best_cost = whole, best = {nt, false};
+        if (tiles < 2 * sms && cut < best_cost - 1e-9) best_cost = cut, best = {nt, true};
+    }
+    return best;
+}
+
 int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
 {
     static const EncodeTiled encode = lookup_encode_tiled();
@@ -471,22 +493,23 @@ int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
     p.tokens       = g.tokens;
     p.n_out        = g.n_out;
     p.k_blocks     = (g.k + kKBlock - 1) / kKBlock;
-    p.token_tile   = g.tokens >= kMaxTokens ? kMaxTokens : (g.tokens + 15) / 16 * 16;
-    p.token_tiles  = (g.tokens + p.token_tile - 1) / p.token_tile;
-    p.tiles        = (g.n_out + kDenseTile - 1) / kDenseTile * p.token_tiles;
+    const Plan plan = choose_plan(g.tokens, g.n_out, p.k_blocks, h->sm_count);
+    p.token_tile    = plan.token_tile;
+    p.token_tiles   = (g.tokens + p.token_tile - 1) / p.token_tile;
+    p.tiles         = (g.n_out + kDenseTile - 1) / kDenseTile * p.token_tiles;
     p.tmem_columns = 32;
     while (p.tmem_columns < 2 * p.token_tile) p.tmem_columns *= 2;
     const size_t stage_b = (size_t)kDenseTile * 128 + (size_t)p.token_tile * 128;
     p.stages             = (int)(((size_t)h->max_smem - 1024 - sizeof(DenseShared)) / stage_b);
     if (p.stages > kMaxStages) p.stages = kMaxStages;
     if (p.stages < 2) return TM_ERR_UNSUPPORTED;
-    // whole tiles in full waves, the rest cut; each CTA of the cut part gets at least four k blocks
     const int sms = h->sm_count;
-    p.whole_waves = p.tiles / sms;
-    int rest      = p.tiles - p.whole_waves * sms;
-    p.cut_ctas    = (int)std::min<long long>(sms, std::max<long long>(1, (long long)rest * p.k_blocks / 4));
-    if (p.cut_ctas < rest || (size_t)2 * p.cut_ctas * p.token_tile * kDenseTile * 4 > h->scratch_bytes) p.cut_ctas = std::max(1, rest);
-    const int grid_ctas = p.whole_waves > 0 ? sms : std::max(1, p.cut_ctas);
+    if (plan.cut && (size_t)2 * sms * p.token_tile * kDenseTile * 4 <= h->scratch_bytes) {
+        // each CTA gets at least four k blocks
+        p.cut_ctas = (int)std::min<long long>(sms, std::max<long long>(1, (long long)p.tiles * p.k_blocks / 4));
+    }
+    p.grid_tiles        = p.cut_ctas > 0 ? 0 : p.tiles;
+    const int grid_ctas = p.cut_ctas > 0 ? p.cut_ctas : std::min(sms, p.tiles);
     p.scratch  = static_cast<float*>(h->scratch);
     p.tickets  = h->counters;
     p.status   = h->status;

@@ -58,7 +58,7 @@ struct DeltaRule {
     float        norm_eps = 0.f;
     float        unit_eps = 1e-6f;     // u = k / sqrt(sum k^2 + unit_eps)
     float        decay_scale = 0.60653065971263342f;  // decay = exp(-decay_scale * sigmoid(.)); here exp(-1/2)
-    size_t       state_off = 0;        // bytes in the slab: float [head][key dim][value dim]
+    size_t       state_off = 0;        // bytes in the slab: float [head][value dim][key dim]
     int          r_col = 0, k_col = 0, v_col = 0, a_col = 0, g_col = 0, w1_col = 0;  // columns of the projections; w1 after tanh
 };
 // scratch of a prefill, fp32: so many floats per token

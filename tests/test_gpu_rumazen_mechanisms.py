@@ -270,7 +270,7 @@ def test_delta_rule_whole_portions_and_decoding(dtype, heads, dim, rank):
             at, i = at + m, i + 1
         assert np.abs(np.concatenate(got) - want).max() <= tol, (sizes, np.abs(np.concatenate(got) - want).max())
         # the state is fp32 in both precisions, and exact to fp32
-        held = slab[256:].view(torch.float32).cpu().numpy().reshape(state.shape)
+        held = slab[256:].view(torch.float32).cpu().numpy().reshape(state.shape).transpose(0, 2, 1)   # [head][value][key]
         assert np.abs(held - state).max() <= 2e-5 * np.abs(state).max(), sizes
 
 
