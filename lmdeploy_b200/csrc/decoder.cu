@@ -39,11 +39,32 @@ __global__ void __launch_bounds__(256) rows_kernel(float* x, E* xb, float* ssq, 
     E*        br = xb + (size_t)t * x_ld;
     const E*  er = ids ? embed + (size_t)min(max(ids[t], 0), vocab - 1) * width : nullptr;
     float     sq = 0.f;
-    for (int i = threadIdx.x; i < width; i += 256) {
-        const float v = er ? to_f32(er[i]) * scale : xr[i];
-        if (er) xr[i] = v;
-        br[i] = from_f32<E>(v);
-        sq += v * v;
+    if (width % 4 == 0 && x_ld % 4 == 0) {
+        for (int i = 4 * threadIdx.x; i < width; i += 1024) {
+            float4 v;
+            if (er) {
+                v = make_float4(to_f32(er[i]) * scale, to_f32(er[i + 1]) * scale, to_f32(er[i + 2]) * scale, to_f32(er[i + 3]) * scale);
+                *reinterpret_cast<float4*>(xr + i) = v;
+            }
+            else {
+                v = *reinterpret_cast<const float4*>(xr + i);
+            }
+            if constexpr (sizeof(E) == 2) {
+                *reinterpret_cast<uint2*>(br + i) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+            }
+            else {
+                *reinterpret_cast<float4*>(br + i) = v;
+            }
+            sq += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+        }
+    }
+    else {
+        for (int i = threadIdx.x; i < width; i += 256) {
+            const float v = er ? to_f32(er[i]) * scale : xr[i];
+            if (er) xr[i] = v;
+            br[i] = from_f32<E>(v);
+            sq += v * v;
+        }
     }
     sq = warp_sum(sq);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = sq;

@@ -25,23 +25,52 @@ struct DeltaKernelParams {
     long long    max_wait;
 };
 
-// DP: head size rounded up to 16, 32, ..., 256.
-// What the scan reads of a (head, token), made by delta_gates_kernel:
-//   u (first token of a pair) or u * w of the token before (second)  |  b = a u  |  w  |  k  |  r  |  v  |  beta, kappa
+// DP: head size rounded up to 32, 64, 128 or 256 in the prefill, from 16 on in the step.
+// What the scan reads of a (head, token), made by delta_gates_kernel (b = a u):
+//   u (first token of a pair) or u * w of the token before (second)  |  -b  |  w  |  k  |  r  |  v  |  beta, kappa
 // Tokens go in pairs, counted from the start of the span.  With z = u^T S read before the token's own update, the second
 // token's z follows from the state before the FIRST one:
 //   z1 = (u1 * w0)^T S - (u1 . b0) z0 + (u1 . k0) v0 = ... - beta z0 + kappa v0
 // so that both products with the state are in flight together.
 template<int DP>
 struct ScanShape {
-    static constexpr int kLanes   = DP / 8;              // lanes that own a column of S, eight rows each in registers
-    static constexpr int kThreads = 256;
-    static constexpr int kColumns = kThreads / kLanes;   // columns of one CTA
-    static constexpr int kRecord  = 6 * DP + 4;          // floats
+    static constexpr int kRows    = DP == 256 ? 8 : 4;    // rows of S per lane
+    static constexpr int kLanes   = DP / kRows;           // lanes that share columns
+    static constexpr int kPerLane = DP == 256 ? 2 : 4;    // columns of a lane (all lanes of a group have the same ones)
+    static constexpr int kThreads = 128;
+    static constexpr int kColumns = kThreads / kLanes * kPerLane;  // columns of one CTA
+    static constexpr int kRecord  = 6 * DP + 4;                    // floats
     static constexpr int kChunk   = DP <= 64 ? 16 : (DP == 128 ? 8 : 4);  // tokens of a stage
     static constexpr int kStages  = 3;
     static constexpr int kSmem    = kStages * kChunk * kRecord * 4;
 };
+
+// two fp32 values side by side: one instruction works on both
+using f32x2 = unsigned long long;
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c)
+{
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b)
+{
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 pair_of(float lo, float hi)
+{
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+    return d;
+}
+__device__ __forceinline__ float2 halves(f32x2 x)
+{
+    float2 f;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(x));
+    return f;
+}
 
 // one warp per (pair of tokens, head)
 template<typename E, int DP>
@@ -89,7 +118,7 @@ __global__ void __launch_bounds__(128) delta_gates_kernel(const DeltaKernelParam
                 kappa += u * k0[e];
                 first = u * w0[e];
             }
-            if (c < DP) rec[c] = first, rec[DP + c] = b, rec[2 * DP + c] = w, rec[3 * DP + c] = k[e], rec[4 * DP + c] = r[e], rec[5 * DP + c] = v[e];
+            if (c < DP) rec[c] = first, rec[DP + c] = -b, rec[2 * DP + c] = w, rec[3 * DP + c] = k[e], rec[4 * DP + c] = r[e], rec[5 * DP + c] = v[e];
             w0[e] = w, b0[e] = b, k0[e] = k[e];
         }
         if (t == 1) {
@@ -134,69 +163,113 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
     if (tid == 0) {
         for (int ch = 0; ch < min(S::kStages, chunks); ++ch) fetch(ch);
     }
-    // lane's rows of its column: 4 at 4 * part and 4 at DP / 2 + 4 * part (conflict-free 16-byte reads)
-    const int part = tid % S::kLanes, col = c0 + tid / S::kLanes, v_at = min(col, DP - 1);
-    float*    state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * dim;
-    float     st[8];
-    auto      row_of = [&](int i) { return (i < 4 ? 0 : DP / 2) + 4 * part + (i & 3); };
+    // Lanes of a group (kLanes of them) share kPerLane columns; lane `part` holds rows [part * kRows, ...) of each, in pairs.
+    constexpr int R2 = S::kRows / 2, NC = S::kPerLane, NV = 2 * NC, kBits = NV == 8 ? 3 : 2;
+    const int     part = tid % S::kLanes, col0 = c0 + tid / S::kLanes * NC, row0 = part * S::kRows;
+    float*        state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * dim;
+    f32x2         st[NC][R2];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        const int r = row_of(i);
-        st[i]       = s.history > 0 && r < dim && col < dim ? state[(size_t)col * dim + r] : 0.f;
+    for (int c = 0; c < NC; ++c) {
+#pragma unroll
+        for (int i = 0; i < R2; ++i) {
+            const int    r   = row0 + 2 * i;
+            const float* at  = state + (size_t)(col0 + c) * dim + r;
+            const bool   on  = s.history > 0 && col0 + c < dim;
+            st[c][i]         = pair_of(on && r < dim ? at[0] : 0.f, on && r + 1 < dim ? at[1] : 0.f);
+        }
     }
-    float* o_out = p.o + (size_t)s.tok0 * d.heads * dim + h * dim + col;
+    // A lane ends up with one of the NV = 2 x NC sums of a pair of tokens: token `b0`, column `mine`
+    const int b0 = part & 1, mine = NC == 4 ? ((part >> 1) & 1) * 2 + ((part >> 2) & 1) : (part >> 1) & 1;
+    const int v_mine = min(col0 + mine, DP - 1);
+    // sums over the lanes of the group of x[0..NV): each lane gets sum number b0 * NC + mine
+    auto scatter_sums = [&](float (&x)[NV]) {
+#pragma unroll
+        for (int level = 0; level < kBits; ++level) {
+            const int  half = NV >> (level + 1);
+            const bool up   = (part >> level) & 1;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float keep = up ? x[i + half] : x[i], send = up ? x[i] : x[i + half];
+                x[i] = keep + __shfl_xor_sync(0xffffffffu, send, 1 << level);
+            }
+        }
+#pragma unroll
+        for (int m = 1 << kBits; m < S::kLanes; m *= 2) x[0] += __shfl_xor_sync(0xffffffffu, x[0], m);
+        return x[0];
+    };
+    // the way back: all NV values to every lane
+    auto gather = [&](float f, float (&x)[NV]) {
+        x[0] = f;
+#pragma unroll
+        for (int level = kBits - 1; level >= 0; --level) {
+            const int  half = NV >> (level + 1);
+            const bool up   = (part >> level) & 1;
+#pragma unroll
+            for (int i = 0; i < half; ++i) {
+                const float other = __shfl_xor_sync(0xffffffffu, x[i], 1 << level), own = x[i];
+                x[i]              = up ? other : own;
+                x[i + half]       = up ? own : other;
+            }
+        }
+    };
+    float* o_out = p.o + (size_t)s.tok0 * d.heads * dim + h * dim + col0 + mine;
     bool   ok    = true;
     int    ch    = 0;
     for (; ch < chunks; ++ch) {
         ok           = mbar_wait(&full[ch % S::kStages], (ch / S::kStages) & 1, p.max_wait);
         const int nt = min(S::kChunk, s.n - ch * S::kChunk);
         for (int t = 0; t < nt; t += 2) {
-            const float* rec = sm + (size_t)((ch % S::kStages) * S::kChunk + t) * S::kRecord;
-            auto vec = [&](const float* r, int which, float (&x)[8]) {
-                const float4 lo = *reinterpret_cast<const float4*>(r + which * DP + 4 * part);
-                const float4 hi = *reinterpret_cast<const float4*>(r + which * DP + DP / 2 + 4 * part);
-                x[0] = lo.x, x[1] = lo.y, x[2] = lo.z, x[3] = lo.w, x[4] = hi.x, x[5] = hi.y, x[6] = hi.z, x[7] = hi.w;
-            };
-            auto dot = [&](const float (&x)[8]) {
-                float a = x[0] * st[0], b = x[1] * st[1];
-#pragma unroll
-                for (int i = 2; i < 8; i += 2) a = fmaf(x[i], st[i], a), b = fmaf(x[i + 1], st[i + 1], b);
-                return a + b;
-            };
-            auto update = [&](const float* r, float z, float v) {
-                float b[8], w[8], k[8];
-                vec(r, 1, b), vec(r, 2, w), vec(r, 3, k);
-#pragma unroll
-                for (int i = 0; i < 8; ++i) st[i] = fmaf(w[i], st[i], fmaf(k[i], v, -b[i] * z));
-            };
-            // two sums over the lanes of the column at the price of one: even lanes end up with the first, odd lanes with
-            // the second
-            auto reduce2 = [&](float a, float b) {
-                const bool odd = part & 1;
-                float      x   = odd ? b : a;
-                x += __shfl_xor_sync(0xffffffffu, odd ? a : b, 1);
-#pragma unroll
-                for (int m = 2; m < S::kLanes; m *= 2) x += __shfl_xor_sync(0xffffffffu, x, m);
-                return x;
-            };
             const bool   two  = t + 1 < nt;
+            const float* rec  = sm + (size_t)((ch % S::kStages) * S::kChunk + t) * S::kRecord;
             const float* rec1 = two ? rec + S::kRecord : rec;
-            float        u0[8], u1[8], r0[8], r1[8];
-            vec(rec, 0, u0), vec(rec1, 0, u1);
-            const float v0 = rec[5 * DP + v_at], v1 = rec1[5 * DP + v_at];
-            const float mine = reduce2(dot(u0), dot(u1)), other = __shfl_xor_sync(0xffffffffu, mine, 1);
-            const float z0 = part & 1 ? other : mine, y1 = part & 1 ? mine : other;
-            update(rec, z0, v0);
-            vec(rec, 4, r0);
-            const float o0 = dot(r0);
-            float       o1 = 0.f;
+            auto vec = [&](const float* r, int which, f32x2 (&x)[R2]) {
+#pragma unroll
+                for (int i = 0; i < R2; i += 2) {
+                    const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(r + which * DP + row0 + 2 * i);
+                    x[i] = q.x, x[i + 1] = q.y;
+                }
+            };
+            auto dots = [&](const f32x2 (&x)[R2], float* out) {
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    f32x2 a = mul2(x[0], st[c][0]);
+#pragma unroll
+                    for (int i = 1; i < R2; ++i) a = fma2(x[i], st[c][i], a);
+                    const float2 f = halves(a);
+                    out[c]         = f.x + f.y;
+                }
+            };
+            auto update = [&](const float* r, const float* z) {
+                f32x2 b[R2], w[R2], k[R2];
+                vec(r, 1, b), vec(r, 2, w), vec(r, 3, k);
+                float v[NC];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) v[c] = r[5 * DP + min(col0 + c, DP - 1)];
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    const f32x2 zz = pair_of(z[c], z[c]), vv = pair_of(v[c], v[c]);
+#pragma unroll
+                    for (int i = 0; i < R2; ++i) st[c][i] = fma2(w[i], st[c][i], fma2(k[i], vv, mul2(b[i], zz)));
+                }
+            };
+            f32x2 x0[R2], x1[R2];
+            float sums[NV], z[NV];
+            vec(rec, 0, x0), vec(rec1, 0, x1);
+            dots(x0, sums), dots(x1, sums + NC);
+            float       f     = scatter_sums(sums);
+            const float first = __shfl_xor_sync(0xffffffffu, f, 1);  // the same column's sum of the other token
+            if (b0) f = f - rec1[6 * DP] * first + rec1[6 * DP + 1] * rec[5 * DP + v_mine];
+            gather(f, z);
+            update(rec, z);
+            vec(rec, 4, x0);
+            dots(x0, sums);
             if (two) {
-                update(rec1, y1 - rec1[6 * DP] * z0 + rec1[6 * DP + 1] * v0, v1);
-                vec(rec1, 4, r1);
-                o1 = dot(r1);
+                update(rec1, z + NC);
+                vec(rec1, 4, x1);
             }
-            const float o = reduce2(o0, o1);
-            if (part < 2 && (part == 0 || two) && col < dim) o_out[(size_t)(ch * S::kChunk + t + part) * d.heads * dim] = o;
+            dots(x1, sums + NC);
+            const float o = scatter_sums(sums);
+            if (part < NV && (b0 == 0 || two) && col0 + mine < dim) o_out[(size_t)(ch * S::kChunk + t + b0) * d.heads * dim] = o;
         }
         // everybody is through with the stage; one outcome for the whole CTA
         if (!__syncthreads_and(ok)) break;
@@ -211,40 +284,72 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
         return;
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-        const int r = row_of(i);
-        if (r < dim && col < dim) state[(size_t)col * dim + r] = st[i];
+    for (int c = 0; c < NC; ++c) {
+#pragma unroll
+        for (int i = 0; i < R2; ++i) {
+            const int    r   = row0 + 2 * i;
+            float*       dst = state + (size_t)(col0 + c) * dim + r;
+            const float2 f   = halves(st[c][i]);
+            if (col0 + c < dim && r < dim) dst[0] = f.x;
+            if (col0 + c < dim && r + 1 < dim) dst[1] = f.y;
+        }
     }
 }
 
-// Head outputs over their root mean square, times the norm weight and the output gate: one warp per (token, head)
-template<typename E>
+// Head outputs over their root mean square, times the norm weight and the output gate: a warp takes a head of four tokens
+constexpr int kFinishTokens = 4;
+template<typename E, int PER>  // PER: dimensions per lane
 __global__ void __launch_bounds__(256) delta_finish_kernel(const DeltaKernelParams p)
 {
     pdl_wait();
     pdl_launch_dependents();
     const DeltaRule& d    = p.d;
-    const int        lane = threadIdx.x & 31, t = blockIdx.x, h = blockIdx.y * 8 + (threadIdx.x >> 5);
-    const E*         row  = static_cast<const E*>(p.c.proj) + (size_t)t * p.c.proj_ld;
-    E*               out  = static_cast<E*>(p.c.out) + (size_t)t * p.c.out_ld;
+    const int        lane = threadIdx.x & 31, t0 = blockIdx.x * kFinishTokens, h = blockIdx.y * 8 + (threadIdx.x >> 5);
+    const int        nt   = min(kFinishTokens, p.c.tokens - t0);
     if (blockIdx.y == 0) {
-        for (int n = d.heads * d.dim + threadIdx.x; n < p.c.out_pad; n += 256) out[n] = from_f32<E>(0.f);
+        for (int t = 0; t < nt; ++t) {
+            E* out = static_cast<E*>(p.c.out) + (size_t)(t0 + t) * p.c.out_ld;
+            for (int n = d.heads * d.dim + threadIdx.x; n < p.c.out_pad; n += 256) out[n] = from_f32<E>(0.f);
+        }
     }
     if (h >= d.heads) return;
-    const float* o = p.o + ((size_t)t * d.heads + h) * d.dim;
-    float        x[kMaxDim / 32], sq = 0.f;
+    float x[kFinishTokens][PER], g[kFinishTokens][PER], nw[PER];
 #pragma unroll
-    for (int e = 0; e < kMaxDim / 32; ++e) {
-        const int c = lane + 32 * e;
-        x[e]        = c < d.dim ? o[c] : 0.f;
-        sq += x[e] * x[e];
-    }
-    const float inv = 1.f / sqrtf(warp_sum(sq) / (float)d.dim + d.norm_eps);
+    for (int e = 0; e < PER; ++e) nw[e] = lane + 32 * e < d.dim ? d.norm[h * d.dim + lane + 32 * e] : 0.f;
 #pragma unroll
-    for (int e = 0; e < kMaxDim / 32; ++e) {
-        const int c = lane + 32 * e, n = h * d.dim + c;
-        if (c < d.dim) out[n] = from_f32<E>(x[e] * inv * d.norm[n] * sigmoid_f32(to_f32(row[d.g_col + n])));
+    for (int t = 0; t < kFinishTokens; ++t) {
+        const float* o   = p.o + ((size_t)(t0 + t) * d.heads + h) * d.dim;
+        const E*     row = static_cast<const E*>(p.c.proj) + (size_t)(t0 + t) * p.c.proj_ld + d.g_col + h * d.dim;
+#pragma unroll
+        for (int e = 0; e < PER; ++e) {
+            const int  c  = lane + 32 * e;
+            const bool on = t < nt && c < d.dim;
+            x[t][e] = on ? o[c] : 0.f, g[t][e] = on ? to_f32(row[c]) : 0.f;
+        }
     }
+#pragma unroll
+    for (int t = 0; t < kFinishTokens; ++t) {
+        float sq = 0.f;
+#pragma unroll
+        for (int e = 0; e < PER; ++e) sq += x[t][e] * x[t][e];
+        const float inv = 1.f / sqrtf(warp_sum(sq) / (float)d.dim + d.norm_eps);
+        if (t >= nt) break;
+        E* out = static_cast<E*>(p.c.out) + (size_t)(t0 + t) * p.c.out_ld + h * d.dim;
+#pragma unroll
+        for (int e = 0; e < PER; ++e) {
+            if (lane + 32 * e < d.dim) out[lane + 32 * e] = from_f32<E>(x[t][e] * inv * nw[e] * sigmoid_f32(g[t][e]));
+        }
+    }
+}
+
+template<typename E>
+cudaError_t finish_launch(const DeltaKernelParams& p, cudaStream_t st)
+{
+    const dim3 grid((p.c.tokens + kFinishTokens - 1) / kFinishTokens, (p.d.heads + 7) / 8);
+    if (p.d.dim <= 32) return launch_kernel(delta_finish_kernel<E, 1>, grid, dim3(256), 0, st, p.c.pdl, p);
+    if (p.d.dim <= 64) return launch_kernel(delta_finish_kernel<E, 2>, grid, dim3(256), 0, st, p.c.pdl, p);
+    if (p.d.dim <= 128) return launch_kernel(delta_finish_kernel<E, 4>, grid, dim3(256), 0, st, p.c.pdl, p);
+    return launch_kernel(delta_finish_kernel<E, 8>, grid, dim3(256), 0, st, p.c.pdl, p);
 }
 
 // One new token per sequence, one CTA per (head, sequence): decay projection, step, head norm and gate in one kernel.
@@ -426,11 +531,15 @@ int padded_dim(int dim)
     return dp;
 }
 
+int scan_dim(int dim)
+{
+    return padded_dim(dim) < 32 ? 32 : padded_dim(dim);
+}
+
 template<typename E>
 cudaError_t scan_dispatch(const DeltaKernelParams& p, cudaStream_t st)
 {
-    switch (padded_dim(p.d.dim)) {
-        case 16: return scan_launch<E, 16>(p, st);
+    switch (scan_dim(p.d.dim)) {
         case 32: return scan_launch<E, 32>(p, st);
         case 64: return scan_launch<E, 64>(p, st);
         case 128: return scan_launch<E, 128>(p, st);
@@ -461,7 +570,7 @@ bool valid(const DeltaRule& d, const MixerCall& c)
 // decay pre-activations, later the outputs, to a multiple of four floats; behind them the records
 size_t delta_rule_scratch_floats(const DeltaRule& d)
 {
-    return (size_t)(d.heads * d.dim + 3) / 4 * 4 + (size_t)d.heads * (6 * padded_dim(d.dim) + 4);
+    return (size_t)(d.heads * d.dim + 3) / 4 * 4 + (size_t)d.heads * (6 * scan_dim(d.dim) + 4);
 }
 
 int delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, float* scratch, cudaStream_t st)
@@ -479,9 +588,7 @@ int delta_rule_prefill(tm_handle* h, const DeltaRule& d, const MixerCall& c, flo
     const DeltaKernelParams p{d, c, scratch, records, scratch, h->status, kMaxWaitCycles};
     cudaError_t             e = c.f32 ? scan_dispatch<float>(p, st) : scan_dispatch<__nv_bfloat16>(p, st);
     if (e == cudaSuccess) {
-        const dim3 grid(c.tokens, (d.heads + 7) / 8);
-        e = c.f32 ? launch_kernel(delta_finish_kernel<float>, grid, dim3(256), 0, st, c.pdl, p) :
-                    launch_kernel(delta_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, c.pdl, p);
+        e = c.f32 ? finish_launch<float>(p, st) : finish_launch<__nv_bfloat16>(p, st);
     }
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;
