@@ -180,7 +180,6 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
     }
     // A lane ends up with one of the NV = 2 x NC sums of a pair of tokens: token `b0`, column `mine`
     const int b0 = part & 1, mine = NC == 4 ? ((part >> 1) & 1) * 2 + ((part >> 2) & 1) : (part >> 1) & 1;
-    const int v_mine = min(col0 + mine, DP - 1);
     // sums over the lanes of the group of x[0..NV): each lane gets sum number b0 * NC + mine
     auto scatter_sums = [&](float (&x)[NV]) {
 #pragma unroll
@@ -197,24 +196,17 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
         for (int m = 1 << kBits; m < S::kLanes; m *= 2) x[0] += __shfl_xor_sync(0xffffffffu, x[0], m);
         return x[0];
     };
-    // the way back: all NV values to every lane
-    auto gather = [&](float f, float (&x)[NV]) {
-        x[0] = f;
-#pragma unroll
-        for (int level = kBits - 1; level >= 0; --level) {
-            const int  half = NV >> (level + 1);
-            const bool up   = (part >> level) & 1;
-#pragma unroll
-            for (int i = 0; i < half; ++i) {
-                const float other = __shfl_xor_sync(0xffffffffu, x[i], 1 << level), own = x[i];
-                x[i]              = up ? other : own;
-                x[i + half]       = up ? own : other;
-            }
-        }
-    };
     float* o_out = p.o + (size_t)s.tok0 * d.heads * dim + h * dim + col0 + mine;
-    bool   ok    = true;
-    int    ch    = 0;
+    int    v_at[NC], held = -1;  // held: first token of the pair whose outputs wait in `sums`
+    float  sums[NV] = {};
+    bool   held_two = false, ok = true;
+#pragma unroll
+    for (int c = 0; c < NC; ++c) v_at[c] = 5 * DP + min(col0 + c, DP - 1);
+    auto store_outputs = [&]() {
+        const float o = scatter_sums(sums);
+        if (held >= 0 && part < NV && (b0 == 0 || held_two) && col0 + mine < dim) o_out[(size_t)(held + b0) * d.heads * dim] = o;
+    };
+    int ch = 0;
     for (; ch < chunks; ++ch) {
         ok           = mbar_wait(&full[ch % S::kStages], (ch / S::kStages) & 1, p.max_wait);
         const int nt = min(S::kChunk, s.n - ch * S::kChunk);
@@ -239,37 +231,38 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
                     out[c]         = f.x + f.y;
                 }
             };
-            auto update = [&](const float* r, const float* z) {
-                f32x2 b[R2], w[R2], k[R2];
-                vec(r, 1, b), vec(r, 2, w), vec(r, 3, k);
-                float v[NC];
+            // everything the pair needs from shared memory is on its way before the first sum
+            f32x2 x0[R2], x1[R2], b[2][R2], w[2][R2], k[2][R2], r0[R2], r1[R2];
+            float v[2][NC], z[NV];
+            vec(rec, 0, x0), vec(rec1, 0, x1);
+            vec(rec, 1, b[0]), vec(rec, 2, w[0]), vec(rec, 3, k[0]), vec(rec, 4, r0);
+            vec(rec1, 1, b[1]), vec(rec1, 2, w[1]), vec(rec1, 3, k[1]), vec(rec1, 4, r1);
 #pragma unroll
-                for (int c = 0; c < NC; ++c) v[c] = r[5 * DP + min(col0 + c, DP - 1)];
+            for (int c = 0; c < NC; ++c) v[0][c] = rec[v_at[c]], v[1][c] = rec1[v_at[c]];
+            const float beta = rec1[6 * DP], kappa = rec1[6 * DP + 1];
+            dots(x0, z), dots(x1, z + NC);
+            // all sums in every lane; the outputs of the pair before are summed in the shadow of these exchanges
+#pragma unroll
+            for (int m = 1; m < S::kLanes; m *= 2) {
+#pragma unroll
+                for (int i = 0; i < NV; ++i) z[i] += __shfl_xor_sync(0xffffffffu, z[i], m);
+            }
+            store_outputs();
+#pragma unroll
+            for (int c = 0; c < NC; ++c) z[NC + c] = z[NC + c] - beta * z[c] + kappa * v[0][c];
+            auto update = [&](int j) {
 #pragma unroll
                 for (int c = 0; c < NC; ++c) {
-                    const f32x2 zz = pair_of(z[c], z[c]), vv = pair_of(v[c], v[c]);
+                    const f32x2 zz = pair_of(z[j * NC + c], z[j * NC + c]), vv = pair_of(v[j][c], v[j][c]);
 #pragma unroll
-                    for (int i = 0; i < R2; ++i) st[c][i] = fma2(w[i], st[c][i], fma2(k[i], vv, mul2(b[i], zz)));
+                    for (int i = 0; i < R2; ++i) st[c][i] = fma2(w[j][i], st[c][i], fma2(k[j][i], vv, mul2(b[j][i], zz)));
                 }
             };
-            f32x2 x0[R2], x1[R2];
-            float sums[NV], z[NV];
-            vec(rec, 0, x0), vec(rec1, 0, x1);
-            dots(x0, sums), dots(x1, sums + NC);
-            float       f     = scatter_sums(sums);
-            const float first = __shfl_xor_sync(0xffffffffu, f, 1);  // the same column's sum of the other token
-            if (b0) f = f - rec1[6 * DP] * first + rec1[6 * DP + 1] * rec[5 * DP + v_mine];
-            gather(f, z);
-            update(rec, z);
-            vec(rec, 4, x0);
-            dots(x0, sums);
-            if (two) {
-                update(rec1, z + NC);
-                vec(rec1, 4, x1);
-            }
-            dots(x1, sums + NC);
-            const float o = scatter_sums(sums);
-            if (part < NV && (b0 == 0 || two) && col0 + mine < dim) o_out[(size_t)(ch * S::kChunk + t + b0) * d.heads * dim] = o;
+            update(0);
+            dots(r0, sums);
+            if (two) update(1);
+            dots(r1, sums + NC);
+            held = ch * S::kChunk + t, held_two = two;
         }
         // everybody is through with the stage; one outcome for the whole CTA
         if (!__syncthreads_and(ok)) break;
@@ -283,6 +276,7 @@ __global__ void __launch_bounds__(ScanShape<DP>::kThreads) delta_scan_kernel(con
         }
         return;
     }
+    store_outputs();
 #pragma unroll
     for (int c = 0; c < NC; ++c) {
 #pragma unroll
