@@ -358,7 +358,7 @@ struct StepShape {
 };
 
 template<typename E, int DP>
-__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaKernelParams p)
+__global__ void __launch_bounds__(256, DP <= 64 ? 4 : 1) delta_step_kernel(const DeltaKernelParams p)
 {
     using S = StepShape<DP>;
     constexpr int kVec = 16 / sizeof(E);
@@ -412,15 +412,25 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaKernelParams
     const float vc = on ? to_f32(row[d.v_col + n + c]) : 0.f, ac = on ? to_f32(row[d.a_col + n + c]) : 0.f;
     const float gate = tid < dim ? to_f32(row[d.g_col + n + tid]) : 0.f;
     // ---- decay pre-activation: w2 . tanh(w1 h)
-    float x = 0.f;
+    const bool aligned = (reinterpret_cast<uintptr_t>(row + d.w1_col) & 15) == 0;
+    float      x       = 0.f;
     for (int i = 0;; ++i) {
         const int m = (sub + i * S::kPer) * kVec;
         if (m >= d.rank) break;
         const uint4 a = i == 0 ? w2[0] : i == 1 ? w2[1] : i == 2 ? w2[2] : i == 3 ? w2[3] : *reinterpret_cast<const uint4*>(w2_row + m);
         const E*    wa = reinterpret_cast<const E*>(&a);
+        const E*    xa = row + d.w1_col + m;
+        if (m + kVec <= d.rank && aligned) {
+            const uint4 c16 = *reinterpret_cast<const uint4*>(xa);
+            const E*    xe  = reinterpret_cast<const E*>(&c16);
 #pragma unroll
-        for (int e = 0; e < kVec; ++e) {
-            if (m + e < d.rank) x = fmaf(to_f32(wa[e]), to_f32(row[d.w1_col + m + e]), x);
+            for (int e = 0; e < kVec; ++e) x = fmaf(to_f32(wa[e]), to_f32(xe[e]), x);
+        }
+        else {
+#pragma unroll
+            for (int e = 0; e < kVec; ++e) {
+                if (m + e < d.rank) x = fmaf(to_f32(wa[e]), to_f32(xa[e]), x);
+            }
         }
     }
     // the threads of a channel are neighbours; up to 16 of them

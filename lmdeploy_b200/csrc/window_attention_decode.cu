@@ -18,7 +18,7 @@
 namespace tmb {
 namespace {
 
-constexpr int   kWarps = 4, kThreads = kWarps * 32, kKeys = 16, kHeads = 16, kStages = 3;
+constexpr int   kWarps = 4, kThreads = kWarps * 32, kKeys = 16, kHeads = 16, kStages = 3, kMaxSplits = 32;
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct StepParams {
@@ -59,6 +59,12 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+__device__ __forceinline__ float ex2(float x)
+{
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 // byte offset of 16-byte chunk `chunk` of row `row`
 template<int D>
 __device__ __forceinline__ uint32_t sw(int row, int chunk)
@@ -73,6 +79,7 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
     using E = __nv_bfloat16;
     extern __shared__ __align__(128) unsigned char sm[];
     __shared__ float cs[128], sn[128], k_new[D], v_new[D], self_score[kHeads];
+    __shared__ float s_m[kHeads][kMaxSplits], s_l[kHeads][kMaxSplits], s_top[kHeads], s_sum[kHeads];
     __shared__ int   s_last;
     const WindowAttention& a    = p.a;
     const int              tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -165,14 +172,15 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
         __syncthreads();
     }
     auto score = [&](float s) {  // in units of log2
-        return p.cap_log2 > 0.f ? p.cap_log2 - 2.f * p.cap_log2 / (1.f + exp2f(s * p.cap_in)) : s * p.scale_log2;
+        return p.cap_log2 > 0.f ? fmaf(-2.f * p.cap_log2, __fdividef(1.f, 1.f + ex2(s * p.cap_in)), p.cap_log2) : s * p.scale_log2;
     };
 
     // ---- online softmax over this warp's blocks; fragment rows r and r + 8 are heads
     uint32_t q[D / 16][4];
 #pragma unroll
     for (int k = 0; k < D / 16; ++k) ldsm4(sm_b + sw<D>(lane & 15, 2 * k + (lane >> 4)), q[k]);
-    const int r = lane >> 2, c2 = 2 * (lane & 3);
+    const int  r = lane >> 2, c2 = 2 * (lane & 3);
+    const bool upper = heads > 8;  // the fragments' rows 8..15 hold heads
     float     m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, o[D / 8][4];
 #pragma unroll
     for (int n = 0; n < D / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
@@ -203,6 +211,7 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
         for (int t = 0; t < 2; ++t) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
+                if (e >= 2 && !upper) continue;
                 const bool in = b * kKeys + 8 * t + c2 + (e & 1) < total;
                 s[t][e]       = in ? score(s[t][e]) : -INFINITY;
                 mx[e >> 1]    = fmaxf(mx[e >> 1], s[t][e]);
@@ -211,10 +220,12 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
         float alpha[2];
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
+            alpha[e] = 1.f;
+            if (e == 1 && !upper) continue;
             mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
             mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
             const float top = fmaxf(m[e], mx[e]);
-            alpha[e]        = exp2f(m[e] - top);
+            alpha[e]        = ex2(m[e] - top);
             m[e]            = top;
             l[e] *= alpha[e];
         }
@@ -222,7 +233,8 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
         for (int t = 0; t < 2; ++t) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                s[t][e] = exp2f(s[t][e] - m[e >> 1]);
+                if (e >= 2 && !upper) continue;  // products of zero rows of Q: finite, and read by nobody
+                s[t][e] = ex2(s[t][e] - m[e >> 1]);
                 l[e >> 1] += s[t][e];
             }
         }
@@ -258,41 +270,70 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
     const float* all   = reinterpret_cast<const float*>(sm + L::kQ);
     const size_t item  = ((size_t)blockIdx.z * a.kv_heads + g) * p.head_blocks + hb;
     float*       recs  = p.scratch + item * p.splits * kHeads * (D + 2);
-    auto merge = [&](const float* src, size_t stride, int parts, int hh, int d, bool shared_mem, float& top, float& sum) {
-        top = -INFINITY, sum = 0.f;
-        float y = 0.f;
-        for (int w = 0; w < parts; ++w) top = fmaxf(top, shared_mem ? src[w * stride + hh * (D + 2)] : __ldcg(src + w * stride + hh * (D + 2)));
-        for (int w = 0; w < parts; ++w) {
-            const float* x = src + w * stride + hh * (D + 2);
-            const float  f = top == -INFINITY ? 0.f : exp2f((shared_mem ? x[0] : __ldcg(x)) - top);
-            sum += f * (shared_mem ? x[1] : __ldcg(x + 1));
-            y += f * (shared_mem ? x[2 + d] : __ldcg(x + 2 + d));
+    // merge of `parts` results per head: factors first (one thread per head and part), then the sums over the parts
+    auto factors = [&](const float* src, int parts, bool divide) {
+        for (int w = tid; w < heads * parts; w += kThreads) {
+            const float* x    = src + ((size_t)(w % parts) * kHeads + w / parts) * (D + 2);
+            s_m[w / parts][w % parts] = __ldcg(x), s_l[w / parts][w % parts] = __ldcg(x + 1);
         }
+        __syncthreads();
+        if (tid < heads) {
+            float top = -INFINITY, sum = 0.f;
+            for (int w = 0; w < parts; ++w) top = fmaxf(top, s_m[tid][w]);
+            for (int w = 0; w < parts; ++w) {
+                const float f = top == -INFINITY ? 0.f : ex2(s_m[tid][w] - top);
+                sum += f * s_l[tid][w];
+                s_m[tid][w] = f;
+            }
+            const float scale = divide ? sigmoid_f32(to_f32(row[a.g_col + h0 + tid])) / sum : 1.f;
+            for (int w = 0; w < parts; ++w) s_m[tid][w] *= scale;
+            s_top[tid] = top, s_sum[tid] = sum;
+        }
+        __syncthreads();
+    };
+    auto combine = [&](const float* src, int parts, int hh, int d) {
+        float y = 0.f;
+#pragma unroll 8
+        for (int w = 0; w < parts; ++w) y = fmaf(s_m[hh][w], __ldcg(src + ((size_t)w * kHeads + hh) * (D + 2) + 2 + d), y);
         return y;
     };
-    auto store = [&](int hh, int d, float y, float sum) {
-        const float gate = sigmoid_f32(to_f32(row[a.g_col + h0 + hh]));
-        static_cast<E*>(p.c.out)[(size_t)sp.tok0 * p.c.out_ld + (h0 + hh) * a.vdim + d] = from_f32<E>(y / sum * gate);
+    auto store = [&](int hh, int d, float y) {
+        static_cast<E*>(p.c.out)[(size_t)sp.tok0 * p.c.out_ld + (h0 + hh) * a.vdim + d] = from_f32<E>(y);
+    };
+    // the warps' results, in shared memory
+    for (int w = tid; w < heads * kWarps; w += kThreads) {
+        const float* x = all + ((size_t)(w % kWarps) * kHeads + w / kWarps) * (D + 2);
+        s_m[w / kWarps][w % kWarps] = x[0], s_l[w / kWarps][w % kWarps] = x[1];
+    }
+    __syncthreads();
+    if (tid < heads) {
+        float top = -INFINITY, sum = 0.f;
+        for (int w = 0; w < kWarps; ++w) top = fmaxf(top, s_m[tid][w]);
+        for (int w = 0; w < kWarps; ++w) {
+            const float f = top == -INFINITY ? 0.f : ex2(s_m[tid][w] - top);
+            sum += f * s_l[tid][w];
+            s_m[tid][w] = f;
+        }
+        const float scale = p.splits == 1 ? sigmoid_f32(to_f32(row[a.g_col + h0 + tid])) / sum : 1.f;
+        for (int w = 0; w < kWarps; ++w) s_m[tid][w] *= scale;
+        s_top[tid] = top, s_sum[tid] = sum;
+    }
+    __syncthreads();
+    auto of_warps = [&](int hh, int d) {
+        float y = 0.f;
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) y = fmaf(s_m[hh][w], all[((size_t)w * kHeads + hh) * (D + 2) + 2 + d], y);
+        return y;
     };
     if (p.splits == 1) {
-        for (int w = tid; w < heads * a.vdim; w += kThreads) {
-            float       top, sum;
-            const int   hh = w / a.vdim, d = w % a.vdim;
-            const float y = merge(all, (size_t)kHeads * (D + 2), kWarps, hh, d, true, top, sum);
-            store(hh, d, y, sum);
-        }
+        for (int w = tid; w < heads * a.vdim; w += kThreads) store(w / a.vdim, w % a.vdim, of_warps(w / a.vdim, w % a.vdim));
     }
     else {
         float* mine = recs + (size_t)blockIdx.x * kHeads * (D + 2);
-        for (int w = tid; w < heads * D; w += kThreads) {
-            float       top, sum;
-            const int   hh = w / D, d = w % D;
-            const float y = merge(all, (size_t)kHeads * (D + 2), kWarps, hh, d, true, top, sum);
-            __stcg(mine + hh * (D + 2) + 2 + d, y);
-            if (d == 0) {
-                __stcg(mine + hh * (D + 2), top);
-                __stcg(mine + hh * (D + 2) + 1, sum);
-            }
+        for (int w = tid; w < heads * D; w += kThreads) __stcg(mine + (w / D) * (D + 2) + 2 + w % D, of_warps(w / D, w % D));
+        if (tid < heads) {
+            __stcg(mine + tid * (D + 2), s_top[tid]);
+            __stcg(mine + tid * (D + 2) + 1, s_sum[tid]);
         }
         __threadfence();
         __syncthreads();
@@ -303,12 +344,8 @@ __global__ void __launch_bounds__(kThreads) window_step_kernel(const StepParams 
         __syncthreads();
         if (s_last) {
             __threadfence();
-            for (int w = tid; w < heads * a.vdim; w += kThreads) {
-                float       top, sum;
-                const int   hh = w / a.vdim, d = w % a.vdim;
-                const float y = merge(recs, (size_t)kHeads * (D + 2), p.splits, hh, d, false, top, sum);
-                store(hh, d, y, sum);
-            }
+            factors(recs, p.splits, true);
+            for (int w = tid; w < heads * a.vdim; w += kThreads) store(w / a.vdim, w % a.vdim, combine(recs, p.splits, w / a.vdim, w % a.vdim));
         }
     }
 
@@ -362,12 +399,15 @@ int window_attention_step(tm_handle* h, const WindowAttention& a, const MixerCal
     p.cap_in      = a.softcap > 0.f ? 2.f * kLog2e * a.scale / a.softcap : 0.f;
     p.head_blocks = (a.heads / a.kv_heads + kHeads - 1) / kHeads;
     const int D   = a.dim <= 64 && a.vdim <= 64 ? 64 : 128;
-    // about two CTAs per SM, each with at least four blocks of keys per warp; the bound on the visible keys is the host's
+    // the bound on the visible keys is the host's
     const long long items = (long long)c.batch * a.kv_heads * p.head_blocks;
     const long long keys  = a.window > 0 ? (long long)a.window + (a.pool > 0 ? c.max_context / a.pool : 0) : c.max_context;
-    long long splits = (2ll * h->sm_count + items - 1) / items;
-    splits           = std::min(splits, std::max(1ll, keys / (kKeys * kWarps * 4)));
-    splits           = std::min(splits, (long long)(h->attn_scratch_bytes / (items * kHeads * (D + 2) * 4)));
+    // two CTAs fit an SM; a CTA's set-up and the merge cost as much as hundreds of keys, so sequences are split only to
+    // occupy SMs that would idle, each warp with at least two blocks of keys
+    const long long most = std::min<long long>(kMaxSplits, std::max(1ll, keys / (kKeys * kWarps * 2)));
+    long long splits     = std::min((2ll * h->sm_count + items - 1) / items, most);
+    if (items >= h->sm_count) splits = 1;
+    splits = std::min(splits, (long long)(h->attn_scratch_bytes / (items * kHeads * (D + 2) * 4)));
     if (splits < 1 || items > (long long)h->attn_counter_ints) splits = 1;
     p.splits  = (int)splits;
     p.scratch = static_cast<float*>(h->attn_scratch);
