@@ -32,8 +32,8 @@ def config(vocab, width, layers, eps=1e-5, scale=1.0):
 
 
 # sizes no power of two, every width different, a layer without feed-forward, two windows
-ODD = config(331, 152, [
-    layer("general_delta", dict(heads=3, dim=24), 88),
+ODD = config(331, 150, [
+    layer("general_delta", dict(heads=3, dim=24), 87),
     layer("attention", attention(6, 2, 40, 28, rot=24, base=700.0, factor=2.5, scale=0.21, softcap=9.0, size=19, pool=5), 104),
     layer("general_delta", dict(heads=5, dim=12), 0),
     layer("attention", attention(4, 4, 36, 52, rot=36, base=5000.0, scale=0.15, softcap=40.0, size=33, pool=7), 0),
@@ -162,6 +162,34 @@ class Runner:
 
     def close(self):
         self.model.close()
+
+
+def first_token_margin(cfg, w, token):
+    """At its first token a delta-rule head gives (r . k) v over its own root mean square, that is v with the SIGN of r . k:
+    rounding decides where r and k are all but orthogonal.  -> the smallest |cos(r, k)| of any head for this first token."""
+    seen = [1.0]
+    m = rumazen.Model(cfg, w)
+    mix = m.general_delta
+
+    def watched(l, spec, h):
+        r, k = ((h @ m.w[f"l{l}.mix.{x}"].T).reshape(spec["heads"], spec["dim"]) for x in "rk")
+        seen.append(np.abs((r * k).sum(-1) / np.linalg.norm(r, axis=-1) / np.linalg.norm(k, axis=-1)).min())
+        return mix(l, spec, h)
+
+    m.general_delta = watched
+    m.forward([token])
+    return min(seen)
+
+
+def prompts(cfg, w, lengths, seed=5):
+    """random token ids whose first token is well conditioned (first_token_margin)"""
+    rng, out = np.random.default_rng(seed), []
+    for n in lengths:
+        ids = list(map(int, rng.integers(0, cfg["vocab"], n)))
+        while first_token_margin(cfg, w, ids[0]) < 0.02:
+            ids[0] = int(rng.integers(0, cfg["vocab"]))
+        out.append(ids)
+    return out
 
 
 def oracle_logits(cfg, w, ids):

@@ -26,8 +26,7 @@ def checkpoints(tmp_path_factory):
         w = u.weights(cfg, seed=len(name), sharp=1.6)
         folder = str(tmp_path_factory.mktemp(name))
         u.write_checkpoint(folder, cfg, w)
-        rng = np.random.default_rng(5)
-        ids = [list(map(int, rng.integers(0, cfg["vocab"], n))) for n in (LENGTH[name], 37, 61, 2)]
+        ids = u.prompts(cfg, w, (LENGTH[name], 37, 61, 2))
         made[name] = dict(cfg=cfg, w=w, folder=folder, ids=ids, want=[u.oracle_logits(cfg, w, x) for x in ids])
     return made
 

@@ -85,7 +85,7 @@ class Attention:
 TOL = dict(float32=3e-5, bfloat16=2e-2)
 both = pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 SHAPES = [dict(heads=6, kv=2, dim=20, vdim=12, rot=12, factor=2.0, scale=0.3, softcap=4.0, size=13, pool=3),
-          dict(heads=4, kv=1, dim=64, vdim=64, rot=64, base=5000.0, scale=0.125, softcap=30.0, size=40, pool=8),
+          dict(heads=6, kv=3, dim=64, vdim=64, rot=64, base=5000.0, scale=0.11, softcap=22.0, size=40, pool=9),
           dict(heads=8, kv=2, dim=128, vdim=128, rot=64, base=300.0, factor=4.0, scale=0.1, softcap=12.0, size=129, pool=16),
           dict(heads=2, kv=2, dim=64, vdim=128, scale=0.2, size=100),
           dict(heads=3, kv=3, dim=33, vdim=70, rot=32, scale=0.2, softcap=2.0),
