@@ -24,7 +24,8 @@ LIB = os.path.join(OUT_DIR, "libtm_b200.so")
 # Libraries with a part of the framework, for programs that need no more: <name> -> source files of csrc/
 COMPONENTS = {
     "decoder": ["handle", "model", "replay", "cache_manager", "decoder", "decoder_config", "gemm_dense", "window_attention",
-                "window_attention_tc", "window_attention_decode", "delta_rule", "step_kernels"],
+                "window_attention_tc", "window_attention_decode", "delta_rule", "chunk_attention", "chunk_attention_tc",
+                "chunk_attention_decode", "gated_linear", "moe", "step_kernels"],
 }
 
 NVCC_FLAGS = [

@@ -125,6 +125,15 @@ __global__ void random_kernel(E* dst, long long rows, long long cols, long long 
     }
 }
 
+// talk [heads][heads] -> fp16 [pad][pad], zeros beyond
+__global__ void talk_half_kernel(__half* dst, const float* talk, int heads, int pad)
+{
+    for (int i = threadIdx.x; i < pad * pad; i += blockDim.x) {
+        const int h = i / pad, g = i % pad;
+        dst[i] = __float2half_rn(h < heads && g < heads ? talk[h * heads + g] : 0.f);
+    }
+}
+
 float half_to_float(uint16_t h)
 {
     const int   e = (h >> 10) & 31, m = h & 1023;
@@ -216,6 +225,15 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
     };
     auto at = [&](void* base, int64_t row, int64_t ld, int64_t col = 0) { return static_cast<char*>(base) + (size_t)(row * ld + col) * es; };
 
+    const bool gated = c.form == LayerForm::kGatedBranches;
+    // longest chunk of any layer that reads a layer's keys: the ring has to keep it
+    std::vector<int> reach(c.layers.size(), 0);
+    for (size_t i = 0; i < c.layers.size(); ++i) {
+        const MixerSpec& m = c.layers[i].mixer;
+        int&             r = reach[m.kv_from >= 0 ? (size_t)m.kv_from : i];
+        r                  = std::max(r, m.chunk > 0 ? m.chunk : session_len);
+    }
+    int top_max = 0, ff_max = 0, experts_max = 0, router_max = 0;
     layers.resize(c.layers.size());
     for (size_t i = 0; i < layers.size() && ok; ++i) {
         DecoderLayer&     L = layers[i];
@@ -254,7 +272,7 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
             ok = ok && alloc((void**)&L.inv_freq, f.size() * 4) && cudaMemcpy(L.inv_freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice) == cudaSuccess;
             a.inv_freq = L.inv_freq;
         }
-        else {
+        else if (m.type == MixerType::kGeneralDelta) {
             DeltaRule& d = L.delta;
             const int  n = m.heads * m.dim;
             d.heads = m.heads, d.dim = m.dim, d.rank = m.rank, d.norm_eps = (float)c.norm_eps;
@@ -270,6 +288,89 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
             vec(mp + "norm", n, &L.norm, 1.f, 0.f);
             d.w2 = L.w2, d.w0 = L.w0, d.a_bias = L.a_bias, d.norm = L.norm;
             delta_floats = std::max(delta_floats, delta_rule_scratch_floats(d));
+        }
+        else if (m.type == MixerType::kChunkAttention) {
+            ChunkAttention& a = L.chunk;
+            a.heads = m.heads, a.kv_heads = m.kv_heads, a.dim = m.dim, a.vdim = m.vdim, a.scale = (float)m.scale, a.chunk = m.chunk;
+            a.writes = m.kv_from < 0;
+            a.q_col  = segment(m.heads * m.dim);
+            parts    = {{"q", m.heads * m.dim, a.q_col}};
+            if (a.writes) {
+                a.k_col = segment(m.kv_heads * m.dim), a.v_col = segment(m.kv_heads * m.vdim);
+                parts.push_back({"k", m.kv_heads * m.dim, a.k_col});
+                parts.push_back({"v", m.kv_heads * m.vdim, a.v_col});
+                a.ring  = round_up((int)std::min<long long>((long long)reach[i] + max_prefill, session_len), 128);
+                a.k_off = take((size_t)m.kv_heads * a.ring * m.dim * es);
+                a.v_off = take((size_t)m.kv_heads * a.ring * m.vdim * es);
+            }
+            else {
+                const ChunkAttention& o = layers[m.kv_from].chunk;
+                a.ring = o.ring, a.k_off = o.k_off, a.v_off = o.v_off;
+            }
+            const int pad = talk_pad(m.heads);
+            ok = ok && alloc((void**)&L.talk, (size_t)m.heads * m.heads * 4) && alloc(&L.talk_half, (size_t)pad * pad * 2);
+            vec(mp + "pb", m.heads, &L.bias, -3.f, 1.f);
+            target(mp + "talk", m.heads, m.heads, L.talk, m.heads).f32 = true;
+            a.bias = L.bias, a.talk = L.talk, a.talk_half = L.talk_half;
+            attention_weights_bytes = std::max(attention_weights_bytes, chunk_attention_scratch(a, session_len, f32));
+        }
+        else {
+            GatedLinear& d = L.linear;
+            const int    n = m.heads * m.dim, nv = m.heads * m.vdim;
+            d.heads = m.heads, d.dim = m.dim, d.vdim = m.vdim, d.rank = m.rank, d.norm_eps = (float)c.norm_eps, d.tau = (float)m.tau;
+            d.scale = (float)(1.0 / std::sqrt((double)m.dim));
+            d.q_col = segment(n), d.k_col = segment(n), d.v_col = segment(nv), d.g_col = segment(nv), d.a_col = segment(m.rank);
+            parts   = {{"q", n, d.q_col}, {"k", n, d.k_col}, {"v", nv, d.v_col}, {"g", nv, d.g_col}, {"a1", m.rank, d.a_col}};
+            d.w2_ld     = round_up(m.rank, 8);
+            d.state_off = take((size_t)m.heads * m.dim * m.vdim * 4);
+            ok          = ok && alloc(&L.w2, (size_t)n * d.w2_ld * es);
+            target(mp + "a2", n, m.rank, L.w2, d.w2_ld);
+            vec(mp + "a2.b", n, &L.a_bias, 2.f, 1.f);
+            vec(mp + "norm", m.vdim, &L.norm, 1.f, 0.f);
+            d.w2 = L.w2, d.bias = L.a_bias, d.norm = L.norm;
+            delta_floats = std::max(delta_floats, gated_linear_scratch_floats(d));
+        }
+        if (gated) {
+            const MoeSpec& e = L.spec.moe;
+            L.rg1_col        = segment(W);
+            L.in_rows        = round_up(cols, kDenseTile);
+            if (e.experts > 0) {
+                L.x2_from = cols = L.in_rows;
+                L.rg2_col = segment(W), L.router_col = segment(e.experts + e.identity);
+                L.in_rows = cols;
+            }
+            L.mix_pad = round_up(m.out_width(), 8);
+            L.out_k   = L.mix_pad;
+            ok = ok && alloc(&L.w_in, (size_t)L.in_rows * x_ld * es) && alloc(&L.w_out, (size_t)W * L.out_k * es);
+            if (!ok) break;
+            vec(p + "norm1", W, &L.norm1, 1.f, 0.1f);
+            for (const Part& q : parts) target(mp + q.name, q.rows, W, at(L.w_in, q.col, x_ld), x_ld);
+            target(mp + "o", W, m.out_width(), L.w_out, L.out_k);
+            target(p + "rg1", W, W, at(L.w_in, L.rg1_col, x_ld), x_ld);
+            vec(p + "rg1.b", W, &L.rg1_bias, 0.f, 1.f);
+            if (e.experts > 0) {
+                const int n = e.experts + e.identity, down_ld = round_up(e.ff, 8);
+                L.router = {e.experts, e.identity, e.top, e.groups, e.keep, nullptr};
+                ok = ok && alloc(&L.w_experts, (size_t)e.experts * 2 * e.ff * x_ld * es) && alloc(&L.w_down, (size_t)e.experts * W * down_ld * es);
+                if (!ok) break;
+                vec(p + "norm2", W, &L.norm2, 1.f, 0.1f);
+                target(p + "rg2", W, W, at(L.w_in, L.rg2_col, x_ld), x_ld);
+                vec(p + "rg2.b", W, &L.rg2_bias, 0.f, 1.f);
+                target(p + "mlp.router", n, W, at(L.w_in, L.router_col, x_ld), x_ld);
+                vec(p + "mlp.correction", n, &L.correction, 0.f, 0.f);
+                L.router.correction = L.correction;
+                for (int x = 0; x < e.experts; ++x) {
+                    const std::string ep = p + "mlp.e" + std::to_string(x) + ".";
+                    target(ep + "gate", e.ff, W, at(L.w_experts, (int64_t)x * 2 * e.ff, x_ld), 2 * x_ld);
+                    target(ep + "up", e.ff, W, at(L.w_experts, (int64_t)x * 2 * e.ff + 1, x_ld), 2 * x_ld);
+                    target(ep + "down", W, e.ff, at(L.w_down, (int64_t)x * W, down_ld), down_ld);
+                }
+                top_max = std::max(top_max, e.top), ff_max = std::max(ff_max, e.ff), experts_max = std::max(experts_max, e.experts);
+                router_max = std::max(router_max, n);
+            }
+            proj_ld = std::max(proj_ld, round_up(L.x2_from > 0 ? L.router_col : L.in_rows, 8));
+            y_ld    = std::max(y_ld, L.out_k);
+            continue;
         }
         L.mixer_cols = round_up(cols, kDenseTile);
         L.in_rows    = L.mixer_cols + 2 * ff;
@@ -293,7 +394,12 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
     if (ok) {
         target("embed", c.vocab, W, embed, W).init_std = 1.f;
         target("head", c.vocab, W, head, x_ld);
-        gain("final.norm", &final_gain);
+        if (gated) {
+            vec("final.norm", W, &final_norm, 1.f, 0.1f);
+        }
+        else {
+            gain("final.norm", &final_gain);
+        }
     }
     ssq_stride            = round_up(tokens, 8);
     const size_t T        = (size_t)tokens, column_tiles = (size_t)(W + kDenseTile - 1) / kDenseTile;
@@ -302,6 +408,23 @@ int tm_decoder::init(tm_handle* handle, const DecoderConfig& c, const tm_model_o
          && alloc(&proj, T * proj_ld * es) && alloc(&y, T * y_ld * es) && alloc((void**)&delta_scratch, (size_t)max_prefill * delta_floats * 4) && alloc((void**)&logits, logit_rows * c.vocab * 4)
          && alloc(&want_xb, (size_t)kWantRows * x_ld * es) && alloc((void**)&want_ssq, (size_t)kWantRows * 4) && alloc((void**)&ids, T * 4)
          && alloc((void**)&want, T * 4) && alloc((void**)&picked, T * 4) && alloc((void**)&inactive, T) && alloc((void**)&spans, T * sizeof(SeqSpan));
+    if (gated) {
+        const size_t rows = T * std::max(1, top_max);
+        router_ld = round_up(std::max(1, router_max), 4), act_ld = round_up(std::max(1, ff_max), 8);
+        moe_rows.ld = x_ld;
+        // as many query tiles at a time as a pass has, within 1 GB
+        const size_t most = T / 128 + max_batch_size;
+        if (attention_weights_bytes > 0) attention_weights_bytes *= std::max<size_t>(1, std::min(most, ((size_t)1 << 30) / attention_weights_bytes));
+        ok = ok && alloc(&xb2, T * x_ld * es) && alloc((void**)&tiles, T * sizeof(QueryTile));
+        if (top_max > 0) {
+            ok = ok && alloc(&expert_act, rows * act_ld * es) && alloc(&expert_out, rows * W * es) && alloc((void**)&router_logits, T * router_ld * 4)
+                 && alloc((void**)&moe_rows.counts, (size_t)experts_max * 4) && alloc((void**)&moe_rows.offsets, (size_t)(experts_max + 1) * 4)
+                 && alloc((void**)&moe_rows.slots, rows * 4) && alloc((void**)&moe_rows.weights, rows * 4) && alloc((void**)&moe_rows.ranks, rows * 4)
+                 && alloc(&moe_rows.sorted, rows * x_ld * es);
+        }
+        if (attention_weights_bytes > 0) ok = ok && alloc(&attention_weights, attention_weights_bytes);
+        for (DecoderLayer& L : layers) L.chunk.weights = attention_weights, L.chunk.weights_bytes = attention_weights_bytes;
+    }
     const cudaError_t e = cudaGetLastError();
     cudaSetDevice(prev);
     if (!ok) {
@@ -365,8 +488,18 @@ int tm_decoder::load(const std::string& path, std::string* why)
             break;
         }
     }
+    if (rc == TM_OK) rc = derive_weights();
     cudaSetDevice(prev);
     return rc;
+}
+
+// what kernels want in another form than the checkpoint has it
+int tm_decoder::derive_weights()
+{
+    for (const DecoderLayer& L : layers) {
+        if (L.talk_half) talk_half_kernel<<<1, 256>>>(static_cast<__half*>(L.talk_half), L.talk, L.chunk.heads, talk_pad(L.chunk.heads));
+    }
+    return cudaDeviceSynchronize() == cudaSuccess ? TM_OK : TM_ERR_CUDA;
 }
 
 int tm_decoder::random_weights(unsigned long long seed)
@@ -384,9 +517,9 @@ int tm_decoder::random_weights(unsigned long long seed)
             random_kernel<__nv_bfloat16><<<1024, 256>>>(static_cast<__nv_bfloat16*>(t.dst), t.rows, t.cols, t.row_stride, t.init_mean, t.init_std, k);
         }
     }
-    const cudaError_t e = cudaDeviceSynchronize();
+    const int rc = derive_weights();
     cudaSetDevice(prev);
-    return e == cudaSuccess ? TM_OK : TM_ERR_CUDA;
+    return rc;
 }
 
 int tm_decoder::new_cache(tm_cache_manager** out, size_t max_entry_count, size_t chunk_size) const
@@ -403,10 +536,104 @@ struct tm_decoder::Pass {
     float* const* residual_rows = nullptr;  // [batch] destination of each span's rows of layer 0
     size_t        residual_layer_stride = 0;
     const SeqSpan* host_spans = nullptr;
+    int            tile_count = 0;          // prefill: query tiles on the device
 };
+
+int tm_decoder::run_mixer(const DecoderLayer& L, const Pass& p, cudaStream_t s)
+{
+    MixerCall c;
+    c.proj = proj, c.proj_ld = proj_ld, c.out = y, c.out_ld = y_ld, c.out_pad = L.mix_pad, c.spans = spans, c.batch = p.batch;
+    c.tokens = p.tokens, c.max_n = p.max_n, c.max_context = session_len, c.f32 = f32, c.pdl = p.pdl;
+    if (tiles && !p.decode) c.tiles = tiles, c.tile_count = p.tile_count;
+    switch (L.spec.mixer.type) {
+        case MixerType::kAttention: return p.decode ? window_attention_decode(h, L.attention, c, s) : window_attention_prefill(h, L.attention, c, s);
+        case MixerType::kGeneralDelta: return p.decode ? delta_rule_decode(h, L.delta, c, s) : delta_rule_prefill(h, L.delta, c, delta_scratch, s);
+        case MixerType::kChunkAttention: return p.decode ? chunk_attention_decode(h, L.chunk, c, s) : chunk_attention_prefill(h, L.chunk, c, s);
+        default: return p.decode ? gated_linear_decode(h, L.linear, c, s) : gated_linear_prefill(h, L.linear, c, delta_scratch, s);
+    }
+}
+
+int tm_decoder::copy_residual(const Pass& p, size_t layer, cudaStream_t s)
+{
+    for (int b = 0; p.residual_rows && b < p.batch; ++b) {
+        if (cudaMemcpyAsync(p.residual_rows[b] + layer * p.residual_layer_stride, x + (size_t)p.host_spans[b].tok0 * cfg.width,
+                            (size_t)p.host_spans[b].n * cfg.width * 4, cudaMemcpyDeviceToDevice, s)
+            != cudaSuccess) {
+            return TM_ERR_CUDA;
+        }
+    }
+    return TM_OK;
+}
+
+// LayerForm::kGatedBranches; leaves the final norm's rows in xb
+int tm_decoder::run_gated_layers(const Pass& p, cudaStream_t s)
+{
+    const int    W   = cfg.width;
+    const size_t es  = f32 ? 4 : 2;
+    const bool   pdl = p.pdl;
+    const float  mult = (float)cfg.residual_mult;
+    // the rows kernel ahead of layer `next` (the output behind the last), with what the layer before leaves to add
+    auto rows = [&](size_t next) {
+        RowsCall c;
+        c.x = x, c.tokens = p.tokens, c.width = W, c.eps = (float)cfg.norm_eps, c.out_a = xb, c.out_ld = x_ld;
+        if (next == 0) {
+            c.embed = embed, c.ids = ids, c.vocab = cfg.vocab;
+        }
+        else if (layers[next - 1].router.experts > 0) {
+            const DecoderLayer& L = layers[next - 1];
+            c.expert_rows = expert_out, c.input = xb2, c.input_ld = x_ld, c.slots = moe_rows.slots, c.weights = moe_rows.weights, c.top = L.router.top;
+            c.gate = static_cast<char*>(proj) + (size_t)L.rg2_col * es, c.gate_ld = proj_ld, c.gate_bias = L.rg2_bias, c.mult = mult;
+        }
+        c.weight_a = next < layers.size() ? layers[next].norm1 : final_norm;
+        if (next < layers.size() && layers[next].router.experts > 0) c.weight_b = layers[next].norm2, c.out_b = xb2;
+        c.clear = moe_rows.counts;
+        for (const DecoderLayer& L : layers) c.clear_count = std::max(c.clear_count, L.router.experts);
+        return norm_rows(h, c, f32, s, pdl);
+    };
+    int rc = rows(0);
+    for (size_t l = 0; l < layers.size() && rc == TM_OK; ++l) {
+        const DecoderLayer& L = layers[l];
+        DenseGemm           g;
+        g.w = L.w_in, g.ldw = x_ld, g.x = xb, g.ldx = x_ld, g.tokens = p.tokens, g.n_out = L.in_rows, g.k = W;
+        g.ep.kind = DenseKind::kStore, g.ep.out = proj, g.ep.out_ld = proj_ld;
+        if (L.x2_from > 0) {
+            g.x2 = xb2, g.x2_from = L.x2_from;
+            g.ep.f32_out = router_logits, g.ep.f32_from = L.router_col, g.ep.f32_ld = router_ld;
+            g.n_out = L.router_col + L.router.outputs();
+        }
+        if ((rc = dense_gemm(h, g, f32, s, pdl)) != TM_OK) break;
+        rc = run_mixer(L, p, s);
+        if (rc != TM_OK || (l + 1 == layers.size() && !p.need_output)) break;
+
+        DenseGemm o;
+        o.w = L.w_out, o.ldw = L.out_k, o.x = y, o.ldx = y_ld, o.tokens = p.tokens, o.n_out = W, o.k = L.out_k;
+        o.ep.kind = DenseKind::kResidual, o.ep.residual = x, o.ep.residual_ld = W, o.ep.mult = mult;
+        o.ep.gate = static_cast<char*>(proj) + (size_t)L.rg1_col * es, o.ep.gate_ld = proj_ld, o.ep.gate_bias = L.rg1_bias;
+        if ((rc = dense_gemm(h, o, f32, s, pdl)) != TM_OK) break;
+        if (L.router.experts > 0) {
+            const MoeSpec& e = L.spec.moe;
+            if ((rc = moe_dispatch(h, L.router, moe_rows, router_logits, router_ld, xb2, p.tokens, W, f32, s, pdl)) != TM_OK) break;
+            DenseGemm u;
+            u.w = L.w_experts, u.ldw = x_ld, u.x = moe_rows.sorted, u.ldx = x_ld, u.tokens = p.tokens * e.top, u.n_out = 2 * e.ff, u.k = W;
+            u.groups.count = e.experts, u.groups.offsets = moe_rows.offsets;
+            u.ep.kind = DenseKind::kInput, u.ep.split = 0, u.ep.act = expert_act, u.ep.act_ld = act_ld;
+            u.ep.activation = DenseActivation::kClampedSwish, u.ep.limit = (float)e.limit, u.ep.slope = kSwishSlope;
+            if ((rc = dense_gemm(h, u, f32, s, pdl)) != TM_OK) break;
+            DenseGemm d;
+            d.w = L.w_down, d.ldw = round_up(e.ff, 8), d.x = expert_act, d.ldx = act_ld, d.tokens = u.tokens, d.n_out = W, d.k = e.ff;
+            d.groups = u.groups;
+            d.ep.kind = DenseKind::kStore, d.ep.out = expert_out, d.ep.out_ld = W;
+            if ((rc = dense_gemm(h, d, f32, s, pdl)) != TM_OK) break;
+        }
+        if ((rc = rows(l + 1)) != TM_OK) break;
+        rc = copy_residual(p, l, s);
+    }
+    return rc;
+}
 
 int tm_decoder::run_layers(const Pass& p, cudaStream_t s)
 {
+    if (cfg.form == LayerForm::kGatedBranches) return run_gated_layers(p, s);
     const int  W   = cfg.width;
     const bool pdl = p.pdl;
     auto rows = [&](const int* token_ids) {
@@ -437,15 +664,7 @@ int tm_decoder::run_layers(const Pass& p, cudaStream_t s)
         g.ep.act = static_cast<char*>(y) + (size_t)L.mix_pad * (f32 ? 4 : 2), g.ep.act_ld = y_ld;
         if ((rc = dense_gemm(h, g, f32, s, pdl)) != TM_OK) break;
 
-        MixerCall c;
-        c.proj = proj, c.proj_ld = proj_ld, c.out = y, c.out_ld = y_ld, c.out_pad = L.mix_pad, c.spans = spans, c.batch = p.batch;
-        c.tokens = p.tokens, c.max_n = p.max_n, c.max_context = session_len, c.f32 = f32, c.pdl = pdl;
-        if (L.spec.mixer.type == MixerType::kAttention) {
-            rc = p.decode ? window_attention_decode(h, L.attention, c, s) : window_attention_prefill(h, L.attention, c, s);
-        }
-        else {
-            rc = p.decode ? delta_rule_decode(h, L.delta, c, s) : delta_rule_prefill(h, L.delta, c, delta_scratch, s);
-        }
+        rc = run_mixer(L, p, s);
         if (rc != TM_OK || (last && !p.need_output)) break;
 
         DenseGemm o;
@@ -456,15 +675,7 @@ int tm_decoder::run_layers(const Pass& p, cudaStream_t s)
             ssq_parts = (W + kDenseTile - 1) / kDenseTile;
         }
         if ((rc = dense_gemm(h, o, f32, s, pdl)) != TM_OK) break;
-        if (p.residual_rows) {
-            for (int b = 0; b < p.batch; ++b) {
-                if (cudaMemcpyAsync(p.residual_rows[b] + l * p.residual_layer_stride, x + (size_t)p.host_spans[b].tok0 * W,
-                                    (size_t)p.host_spans[b].n * W * 4, cudaMemcpyDeviceToDevice, s)
-                    != cudaSuccess) {
-                    return TM_ERR_CUDA;
-                }
-            }
-        }
+        if ((rc = copy_residual(p, l, s)) != TM_OK) break;
         if (!p.fold) rc = rows(nullptr);
     }
     return rc;
@@ -504,9 +715,15 @@ int tm_decoder::prefill(const tm_model_prefill_state& st, cudaStream_t s)
         p.batch       = (int)sp.size();
         p.need_output = !wanted.empty() || st.residual_out != nullptr;
         p.host_spans  = sp.data();
+        std::vector<QueryTile> query_tiles;
+        for (int b = 0; tiles && b < p.batch; ++b) {
+            for (int q = 0; q < sp[b].n; q += 128) query_tiles.push_back({b, q});
+        }
+        p.tile_count = (int)query_tiles.size();
         if (st.residual_out) p.residual_rows = res_rows.data(), p.residual_layer_stride = (size_t)total * W;
         if (cudaMemcpyAsync(spans, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess
             || cudaMemcpyAsync(ids, tok.data(), tok.size() * 4, cudaMemcpyHostToDevice, s) != cudaSuccess
+            || (tiles && cudaMemcpyAsync(tiles, query_tiles.data(), query_tiles.size() * sizeof(QueryTile), cudaMemcpyHostToDevice, s) != cudaSuccess)
             || (!wanted.empty() && cudaMemcpyAsync(want, wanted.data(), wanted.size() * 4, cudaMemcpyHostToDevice, s) != cudaSuccess)) {
             return TM_ERR_CUDA;
         }
@@ -526,8 +743,10 @@ int tm_decoder::prefill(const tm_model_prefill_state& st, cudaStream_t s)
                 DenseGemm g;
                 g.w = head, g.ldw = x_ld, g.x = want_xb, g.ldx = x_ld, g.tokens = n, g.n_out = cfg.vocab, g.k = cfg.width;
                 g.ep.kind = DenseKind::kF32, g.ep.out = logit_rows[b] + (size_t)(w - want_seq_begin[b]) * V, g.ep.out_ld = cfg.vocab;
-                g.ep.ssq = want_ssq, g.ep.ssq_parts = 1, g.ep.ssq_stride = kWantRows, g.ep.inv_width = 1.f / (float)W, g.ep.eps = (float)cfg.norm_eps;
-                g.ep.gain = final_gain;
+                if (cfg.form == LayerForm::kScalarNorm) {
+                    g.ep.ssq = want_ssq, g.ep.ssq_parts = 1, g.ep.ssq_stride = kWantRows, g.ep.inv_width = 1.f / (float)W, g.ep.eps = (float)cfg.norm_eps;
+                    g.ep.gain = final_gain;
+                }
                 rc        = dense_gemm(h, g, f32, s, false);
             }
         }
@@ -550,8 +769,10 @@ int tm_decoder::step(const tm_llama_decode_state& st, cudaStream_t s, unsigned l
     DenseGemm g;
     g.w = head, g.ldw = x_ld, g.x = xb, g.ldx = x_ld, g.tokens = B, g.n_out = cfg.vocab, g.k = cfg.width;
     g.ep.kind = DenseKind::kF32, g.ep.out = out, g.ep.out_ld = cfg.vocab;
-    g.ep.ssq = ssq, g.ep.ssq_parts = p.fold ? (cfg.width + kDenseTile - 1) / kDenseTile : 1, g.ep.ssq_stride = ssq_stride;
-    g.ep.inv_width = 1.f / (float)cfg.width, g.ep.eps = (float)cfg.norm_eps, g.ep.gain = final_gain;
+    if (cfg.form == LayerForm::kScalarNorm) {
+        g.ep.ssq = ssq, g.ep.ssq_parts = p.fold ? (cfg.width + kDenseTile - 1) / kDenseTile : 1, g.ep.ssq_stride = ssq_stride;
+        g.ep.inv_width = 1.f / (float)cfg.width, g.ep.eps = (float)cfg.norm_eps, g.ep.gain = final_gain;
+    }
     if ((rc = dense_gemm(h, g, f32, s, p.pdl)) != TM_OK) return rc;
     if (step_argmax(out, picked, st.output_ids, st.step, inactive, B, cfg.vocab, 1, st.max_steps, s) != cudaSuccess
         || step_advance(st.step, st.sequence_lengths, inactive, B, s) != cudaSuccess) {

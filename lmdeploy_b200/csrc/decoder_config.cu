@@ -62,8 +62,6 @@ bool read_text(const std::string& path, std::string* out)
     return true;
 }
 
-}  // namespace
-
 bool read_rumazen_config(const Json& j, DecoderConfig* c, std::string* why)
 {
     Reader       r{why};
@@ -119,8 +117,109 @@ bool read_rumazen_config(const Json& j, DecoderConfig* c, std::string* why)
         if (!r.ok) return false;
         c->layers.push_back(s);
     }
-    c->architecture = "Rumazen";
     return true;
+}
+
+bool read_fopinex_config(const Json& j, DecoderConfig* c, std::string* why)
+{
+    Reader       r{why};
+    const double one = 1.0, zero = 0.0;
+    const Json * norm = r.object(j, "norm", false), *layers = j.find("layers");
+    c->form  = LayerForm::kGatedBranches;
+    c->vocab = r.integer(j, "vocab", 1);
+    c->width = r.integer(j, "width", 1);
+    if (norm) c->norm_eps = r.number(*norm, "eps");
+    c->residual_mult = r.number(j, "residual_mult", &one);
+    if (!layers || layers->kind != Json::kArray || layers->items.empty()) r.fail("missing: layers");
+    if (!r.ok) return false;
+    for (const Json& l : layers->items) {
+        LayerSpec   s;
+        const Json *type = l.find("type"), *mixer = r.object(l, "mixer", false), *mlp = r.object(l, "mlp", true);
+        if (!mixer || !type) return r.fail("a layer without type or mixer"), false;
+        MixerSpec& m = s.mixer;
+        m.heads      = r.integer(*mixer, "heads", 1);
+        m.dim        = r.integer(*mixer, "dim", 1);
+        const double dim = m.dim, heads = m.heads, dflt_scale = 1.0 / std::sqrt(dim > 0 ? dim : 1.0);
+        m.vdim = r.integer(*mixer, "vdim", 1, &dim);
+        if (m.dim > 256 || m.vdim > 256) r.fail("heads larger than 256");
+        if (type->text == "attention") {
+            const double own = -1;
+            m.type     = MixerType::kChunkAttention;
+            m.kv_heads = r.integer(*mixer, "kv_heads", 1, &heads);
+            m.scale    = r.number(*mixer, "scale", &dflt_scale);
+            m.kv_from  = r.integer(*mixer, "kv_from", -1, &own);
+            if (const Json* mask = r.object(*mixer, "mask", true)) m.chunk = r.integer(*mask, "size", 1);
+            if (r.ok && m.heads % m.kv_heads) r.fail("kv_heads does not divide heads");
+            if (r.ok && m.kv_from >= 0) {
+                const MixerSpec* o = m.kv_from < (int)c->layers.size() ? &c->layers[m.kv_from].mixer : nullptr;
+                if (!o || o->type != MixerType::kChunkAttention || o->kv_from >= 0 || o->kv_heads != m.kv_heads || o->dim != m.dim || o->vdim != m.vdim) {
+                    r.fail("kv_from: not an earlier attention layer with keys and values of the same shape");
+                }
+            }
+        }
+        else if (type->text == "gla") {
+            const double rank = 16;
+            m.type            = MixerType::kGatedLinear;
+            m.tau             = r.number(*mixer, "tau");
+            m.rank            = r.integer(*mixer, "rank", 1, &rank);
+            if (r.ok && m.tau <= 0) r.fail("out of range: tau");
+        }
+        else {
+            r.fail("unknown layer type: " + type->text);
+        }
+        if (mlp) {
+            const Json *kind = mlp->find("kind"), *expert = r.object(*mlp, "expert", false), *router = r.object(*mlp, "router", false);
+            if (!kind || kind->text != "moe") r.fail("unknown feed-forward kind");
+            if (expert && router) {
+                MoeSpec& e = s.moe;
+                e.ff       = r.integer(*expert, "ff", 1);
+                e.limit    = r.number(*expert, "limit");
+                e.experts  = r.integer(*router, "experts", 1);
+                e.identity = r.integer(*router, "identity", 0, &zero);
+                e.top      = r.integer(*router, "top", 1);
+                if (const Json* groups = r.object(*router, "groups", true)) {
+                    e.groups = r.integer(*groups, "count", 1);
+                    e.keep   = r.integer(*groups, "keep", 1);
+                }
+                const int n = e.experts + e.identity;
+                if (r.ok && (n > kMaxRouterOutputs || e.top > kMaxRouterTop || n % e.groups || e.keep > e.groups || e.top > e.keep * (n / e.groups))) {
+                    r.fail("router sizes that do not fit together");
+                }
+            }
+        }
+        if (!r.ok) return false;
+        c->layers.push_back(s);
+    }
+    return true;
+}
+
+struct DecoderArchitecture {
+    const char* name;
+    bool (*read)(const Json& j, DecoderConfig* c, std::string* why);
+    const char* decay_rank;  // tensor of a recurrent mixer whose rows are the rank of its decay projection
+};
+const DecoderArchitecture kArchitectures[] = {{"Rumazen", read_rumazen_config, "w1"}, {"Fopinex", read_fopinex_config, "a1"}};
+
+const DecoderArchitecture* architecture_of(const Json& j)
+{
+    const Json* a = j.find("architecture");
+    for (const DecoderArchitecture& d : kArchitectures) {
+        if (a && a->text == d.name) return &d;
+    }
+    return nullptr;
+}
+
+}  // namespace
+
+bool read_decoder_config(const Json& j, DecoderConfig* c, std::string* why)
+{
+    const DecoderArchitecture* a = architecture_of(j);
+    if (!a) {
+        *why = "unknown architecture";
+        return false;
+    }
+    c->architecture = a->name;
+    return a->read(j, c, why);
 }
 
 namespace {
@@ -131,20 +230,20 @@ bool read_config_file(const std::string& dir, Json* j)
     return read_text(dir + "/config.json", &text) && Json::parse(text, j) && j->kind == Json::kObject;
 }
 
-bool rumazen_claims(const std::string& dir)
+template<int I>
+bool claims(const std::string& dir)
 {
-    Json        j;
-    const Json* a = nullptr;
-    return read_config_file(dir, &j) && (a = j.find("architecture")) && a->text == "Rumazen";
+    Json j;
+    return read_config_file(dir, &j) && architecture_of(j) == &kArchitectures[I];
 }
 
-int rumazen_open(tm_model** out, tm_handle* h, const std::string& dir, const tm_model_options& opt)
+int decoder_open(tm_model** out, tm_handle* h, const std::string& dir, const tm_model_options& opt)
 {
     Json          j;
     DecoderConfig c;
     g_open_error.clear();
     if (!read_config_file(dir, &j)) return TM_ERR_IO;
-    if (!read_rumazen_config(j, &c, &g_open_error)) return TM_ERR_INVALID_ARG;
+    if (!read_decoder_config(j, &c, &g_open_error)) return TM_ERR_INVALID_ARG;
     const std::string path = dir + "/model.safetensors";
     {
         // the ranks of the decay projections are given by their tensors
@@ -155,10 +254,11 @@ int rumazen_open(tm_model** out, tm_handle* h, const std::string& dir, const tm_
         }
         for (size_t i = 0; i < c.layers.size(); ++i) {
             MixerSpec& m = c.layers[i].mixer;
-            if (m.type != MixerType::kGeneralDelta) continue;
-            const SafeTensor* t = st.find("l" + std::to_string(i) + ".mix.w1");
+            if (m.type != MixerType::kGeneralDelta && m.type != MixerType::kGatedLinear) continue;
+            const std::string name = "l" + std::to_string(i) + ".mix." + architecture_of(j)->decay_rank;
+            const SafeTensor* t    = st.find(name);
             if (!t || t->shape.size() != 2 || t->shape[0] < 1 || t->shape[0] > 65536) {
-                g_open_error = "missing: l" + std::to_string(i) + ".mix.w1";
+                g_open_error = "missing: " + name;
                 return TM_ERR_IO;
             }
             m.rank = (int)t->shape[0];
@@ -176,7 +276,8 @@ int rumazen_open(tm_model** out, tm_handle* h, const std::string& dir, const tm_
     return TM_OK;
 }
 
-const ArchitectureRegistration g_rumazen({"Rumazen", rumazen_claims, rumazen_open});
+const ArchitectureRegistration g_rumazen({kArchitectures[0].name, claims<0>, decoder_open});
+const ArchitectureRegistration g_fopinex({kArchitectures[1].name, claims<1>, decoder_open});
 
 }  // namespace
 }  // namespace tmb
@@ -196,7 +297,7 @@ extern "C" int tm_decoder_create_random(tm_model** out, tm_handle* h, const char
     Json          j;
     DecoderConfig c;
     g_open_error.clear();
-    if (!Json::parse(config_json, &j) || !read_rumazen_config(j, &c, &g_open_error)) return TM_ERR_INVALID_ARG;
+    if (!Json::parse(config_json, &j) || !read_decoder_config(j, &c, &g_open_error)) return TM_ERR_INVALID_ARG;
     tm_decoder* m = new (std::nothrow) tm_decoder();
     if (!m) return TM_ERR_CUDA;
     int rc = m->init(h, c, *opt);

@@ -5,6 +5,7 @@
 // prefill kernel splits over lanes, warps and CTAs; the keys' side (u, a u, w, k, r) is shared by all columns of a head.
 // A column is contiguous in memory.
 #include "common.cuh"
+#include "f32x2.cuh"
 #include "gemm_dense.h"
 #include "mixers.h"
 #include "numeric.cuh"
@@ -44,33 +45,6 @@ struct ScanShape {
     static constexpr int kStages  = 3;
     static constexpr int kSmem    = kStages * kChunk * kRecord * 4;
 };
-
-// two fp32 values side by side: one instruction works on both
-using f32x2 = unsigned long long;
-__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c)
-{
-    f32x2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b)
-{
-    f32x2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-__device__ __forceinline__ f32x2 pair_of(float lo, float hi)
-{
-    f32x2 d;
-    asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-    return d;
-}
-__device__ __forceinline__ float2 halves(f32x2 x)
-{
-    float2 f;
-    asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(x));
-    return f;
-}
 
 // one warp per (pair of tokens, head)
 template<typename E, int DP>

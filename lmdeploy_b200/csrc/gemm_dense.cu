@@ -9,6 +9,8 @@
 // Work split (choose_plan): whole tiles dealt out to the CTAs; or, with few tiles (a decode step), the k blocks of all tiles
 // cut evenly over the CTAs, so that every SM streams the same number of bytes (stream-K).  A tile with several CTAs: each publishes its fp32 part in scratch, the last one to arrive adds the parts up in CTA order (nobody waits, the
 // sum does not depend on the order of arrival) and runs the epilogue.
+// Groups (a mixture of experts): the rows of a group are known on the device only, so every CTA makes the tile table itself
+// from the groups' offsets; a tile is (group, weight tile, token tile), the rest is the same.
 // Every wait is bounded: a barrier that does not complete sets a status bit, the CTA drains its copies and leaves.
 #include "gemm_dense.h"
 #include "numeric.cuh"
@@ -36,6 +38,13 @@ struct DenseShared {
     float    scale[kMaxTokens];
     float    red[4][kMaxTokens];
 };
+// behind DenseShared, groups only: first tile of every group, [groups + 1]
+
+template<bool FAST>
+__device__ __forceinline__ float activate(const DenseEpilogue& ep, float gate, float up)
+{
+    return ep.activation == DenseActivation::kGeluTanh ? gelu_tanh_f32<FAST>(gate) * up : clamped_swish_f32<FAST>(gate, up, ep.limit, ep.slope);
+}
 
 struct DenseTcParams {
     int           tokens, n_out, k_blocks;
@@ -43,6 +52,9 @@ struct DenseTcParams {
     int           grid_tiles;  // tiles dealt out as a whole (all of them, or none)
     int           cut_ctas;    // > 0: CTAs that share the k blocks of all tiles evenly
     int           stages, tmem_columns;
+    int           x2_tile;     // weight tiles from here on multiply the second operand
+    int           column_tiles;
+    DenseGroups   groups;
     float*        scratch;
     int*          tickets;
     unsigned*     status;
@@ -59,10 +71,18 @@ __device__ __forceinline__ void epilogue16(const DenseEpilogue& ep, const float 
         float r[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) r[i] = i < live && col ? ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] : 0.f;
+        float f[16];
+        if (ep.gate) {
+            const float b = col ? ep.gate_bias[n] : 0.f;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) f[i] = i < live && col ? to_f32(static_cast<const E*>(ep.gate)[(size_t)(t0 + i) * ep.gate_ld + n]) + b : 0.f;
+#pragma unroll
+            for (int i = 0; i < 16; ++i) f[i] = __fdividef(ep.mult, 1.f + __expf(-f[i]));
+        }
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
             const bool on = i < live && col;
-            r[i]          = on ? r[i] + y[i] : 0.f;
+            r[i]          = on ? r[i] + (ep.gate ? f[i] * y[i] : y[i]) : 0.f;
             sq[i]         = r[i] * r[i];
             if (on) ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] = r[i];
             if (on && ep.cast) static_cast<E*>(ep.cast)[(size_t)(t0 + i) * ep.cast_ld + n] = from_f32<E>(r[i]);
@@ -85,7 +105,14 @@ __device__ __forceinline__ void epilogue16(const DenseEpilogue& ep, const float 
             const float other = __shfl_xor_sync(0xffffffffu, odd ? y[i] : y[i + 1], 1);
             const float gate = odd ? other : y[i], up = odd ? y[i + 1] : other;
             const int   t = i + (odd ? 1 : 0);
-            if (t < live && col) dst[(size_t)(t0 + t) * ep.act_ld] = from_f32<E>(gelu_tanh_f32<true>(gate) * up);
+            if (t < live && col) dst[(size_t)(t0 + t) * ep.act_ld] = from_f32<E>(activate<true>(ep, gate, up));
+        }
+        return;
+    }
+    if (ep.f32_out && n >= ep.f32_from) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            if (i < live && col) ep.f32_out[(size_t)(t0 + i) * ep.f32_ld + n - ep.f32_from] = y[i];
         }
         return;
     }
@@ -96,8 +123,10 @@ __device__ __forceinline__ void epilogue16(const DenseEpilogue& ep, const float 
     }
 }
 
+template<bool GROUPS>
 __global__ void __launch_bounds__(kThreads, 1)
-dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map)
+dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map,
+                const __grid_constant__ CUtensorMap x2_map)
 {
     extern __shared__ unsigned char smem_dyn[];
     const uint32_t raw  = smem_u32(smem_dyn);
@@ -122,20 +151,67 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
         fence_mbar_init();
     }
     if (warp == 1) tmem_alloc(&sh->tmem_base, p.tmem_columns);
+    int* const first_tile = reinterpret_cast<int*>(sh + 1);
+    if (GROUPS) {
+        pdl_wait();  // the offsets come from a kernel ahead
+        pdl_launch_dependents();
+        if (warp == 0) {
+            int sum = 0;
+            for (int g0 = 0; g0 < p.groups.count; g0 += 32) {
+                const int g = g0 + lane;
+                int       n = g < p.groups.count ? (p.groups.offsets[g + 1] - p.groups.offsets[g] + NT - 1) / NT * p.column_tiles : 0;
+                const int own = n;
+#pragma unroll
+                for (int m = 1; m < 32; m *= 2) {
+                    const int x = __shfl_up_sync(0xffffffffu, n, m);
+                    if (lane >= m) n += x;
+                }
+                if (g < p.groups.count) first_tile[g] = sum + n - own;
+                sum += __shfl_sync(0xffffffffu, n, 31);
+            }
+            if (lane == 0) first_tile[p.groups.count] = sum;
+        }
+    }
     tcgen05_before_sync();
     __syncthreads();
     tcgen05_after_sync();
     const uint32_t tmem = sh->tmem_base;
+    const int      tiles = GROUPS ? first_tile[p.groups.count] : p.tiles;
+    // CTAs that share the k blocks; with groups at least four k blocks each, as the host cannot tell how many there are
+    const int cut_ctas = GROUPS && p.cut_ctas > 0 ? max(1, min(p.cut_ctas, (int)min((long long)tiles * p.k_blocks / 4, 1ll << 20))) : p.cut_ctas;
+    // tile -> weight tile, first row of its tokens, how many there are, first weight row, token tile (the key of `scale`)
+    struct Place {
+        int ct, t0, rows, w_row, tt;
+    };
+    auto place = [&](int tile) {
+        Place q;
+        if (GROUPS) {
+            int lo = 0, hi = p.groups.count;  // first_tile[lo] <= tile < first_tile[hi]
+            while (hi - lo > 1) {
+                const int mid = (lo + hi) >> 1;
+                (first_tile[mid] <= tile ? lo : hi) = mid;
+            }
+            const int begin = p.groups.offsets[lo], n = p.groups.offsets[lo + 1] - begin, tts = (n + NT - 1) / NT, in = tile - first_tile[lo];
+            q.ct = in / tts, q.tt = in - q.ct * tts;
+            q.t0 = begin + q.tt * NT, q.rows = min(NT, n - q.tt * NT), q.w_row = lo * p.n_out + q.ct * kDenseTile;
+        }
+        else {
+            q.ct = tile / p.token_tiles, q.tt = tile - q.ct * p.token_tiles;
+            q.t0 = q.tt * NT, q.rows = min(NT, p.tokens - q.t0), q.w_row = q.ct * kDenseTile;
+        }
+        return q;
+    };
 
     // segment i of this CTA -> tile and k blocks; false behind the last.  Token tiles vary fastest among tiles, so that
     // the CTAs of a wave share weight tiles and activations in the L2.
-    const long long cut_total = (long long)p.tiles * p.k_blocks;
-    auto            cut       = [&](int c) { return (long long)c * cut_total / p.cut_ctas; };
+    const long long cut_total = (long long)tiles * p.k_blocks;
+    auto            cut       = [&](int c) { return (long long)c * cut_total / cut_ctas; };
     auto            segment   = [&](int i, int& tile, int& kb0, int& kb1) {
         if (p.cut_ctas == 0) {
             tile = i * (int)gridDim.x + (int)blockIdx.x, kb0 = 0, kb1 = p.k_blocks;
-            return tile < p.grid_tiles;
+            return tile < (GROUPS ? tiles : p.grid_tiles);
         }
+        if (GROUPS && (int)blockIdx.x >= cut_ctas) return false;
         const long long begin = cut(blockIdx.x), end = cut(blockIdx.x + 1), t = begin / p.k_blocks + i;
         if (t * p.k_blocks >= end) return false;
         tile = (int)t, kb0 = (int)(max(begin, t * p.k_blocks) - t * p.k_blocks), kb1 = (int)(min(end, (t + 1) * p.k_blocks) - t * p.k_blocks);
@@ -147,23 +223,25 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
         if (lane == 0) {
             int  issued = 0;
             bool ok = true, waited = false;
-            auto load_w = [&](int kb, int ct, int s) {
+            auto load_w = [&](int kb, const Place& q, int s) {
                 mbar_arrive_expect_tx(&sh->full[s], stage_b);
-                tma_load_2d(base + s * stage_b, &w_map, kb * kKBlock, ct * kDenseTile, &sh->full[s]);
+                tma_load_2d(base + s * stage_b, &w_map, kb * kKBlock, q.w_row, &sh->full[s]);
             };
-            auto load_x = [&](int kb, int tt, int s) { tma_load_2d(base + s * stage_b + w_bytes, &x_map, kb * kKBlock, tt * NT, &sh->full[s]); };
+            auto load_x = [&](int kb, const Place& q, int s) {
+                tma_load_2d(base + s * stage_b + w_bytes, q.ct >= p.x2_tile ? &x2_map : &x_map, kb * kKBlock, q.t0, &sh->full[s]);
+            };
             int tile, kb0, kb1;
             for (int seg = 0; ok && segment(seg, tile, kb0, kb1); ++seg) {
-                const int ct = tile / p.token_tiles, tt = tile - ct * p.token_tiles;
+                const Place q = place(tile);
                 int       kb = kb0;
                 if (!waited) {
                     // weights are written by no kernel: the first boxes go out before the kernel ahead is complete
                     const int pre = min(ST, kb1 - kb0);
-                    for (int i = 0; i < pre; ++i) load_w(kb0 + i, ct, i);
+                    for (int i = 0; i < pre; ++i) load_w(kb0 + i, q, i);
                     pdl_wait();
                     pdl_launch_dependents();
                     waited = true;
-                    for (int i = 0; i < pre; ++i) load_x(kb0 + i, tt, i);
+                    for (int i = 0; i < pre; ++i) load_x(kb0 + i, q, i);
                     issued = pre;
                     kb += pre;
                 }
@@ -175,8 +253,8 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                         ok = false;
                         break;
                     }
-                    load_w(kb, ct, s);
-                    load_x(kb, tt, s);
+                    load_w(kb, q, s);
+                    load_x(kb, q, s);
                 }
             }
             if (!waited) {
@@ -239,11 +317,9 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
         bool      ok = true;
         int       tile, kb0, kb1;
         for (; ok && segment(local, tile, kb0, kb1); ++local) {
-            const int ct = tile / p.token_tiles, tt = tile - ct * p.token_tiles;
-            const int a    = local & 1;
-            const int t0   = tt * NT;
-            const int rows = min(NT, p.tokens - t0);
-            const int n    = ct * kDenseTile + col;
+            const Place at = place(tile);
+            const int   ct = at.ct, tt = at.tt, a = local & 1, t0 = at.t0, rows = at.rows;
+            const int   n = ct * kDenseTile + col;
             if (p.ep.ssq && scaled_tile != tt) {
                 // 1 / rms of every token of the tile, once per token tile
                 named_bar_sync(kEpiBar, 128);
@@ -279,10 +355,10 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
             auto slot_of = [&](int c) { return p.scratch + (size_t)(2 * c + (cut(c) / p.k_blocks == tile ? 0 : 1)) * slot_floats; };
             if (kb1 - kb0 < p.k_blocks) {
                 const long long lo = (long long)tile * p.k_blocks, hi = lo + p.k_blocks - 1;
-                part0 = (int)(lo * p.cut_ctas / cut_total);
+                part0 = (int)(lo * cut_ctas / cut_total);
                 while (cut(part0 + 1) <= lo) ++part0;
                 while (cut(part0) > lo) --part0;
-                int last = (int)(hi * p.cut_ctas / cut_total);
+                int last = (int)(hi * cut_ctas / cut_total);
                 while (cut(last + 1) <= hi) ++last;
                 while (cut(last) > hi) --last;
                 parts       = last - part0 + 1;
@@ -375,10 +451,17 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(DenseGemm g)
     __shared__ float xs[kSimtK][kSimtTile + 4], ws[kSimtK][kSimtTile + 4];
     pdl_wait();
     pdl_launch_dependents();
-    const int    t0 = blockIdx.y * kSimtTile, n0 = blockIdx.x * kSimtTile;
-    const int    tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-    const float* x = static_cast<const float*>(g.x);
+    const int n0 = blockIdx.x * kSimtTile;
+    int       t0 = blockIdx.y * kSimtTile;
+    const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const float* x = static_cast<const float*>(g.x2 && n0 >= g.x2_from ? g.x2 : g.x);
     const float* w = static_cast<const float*>(g.w);
+    if (g.groups.count > 0) {
+        t0 += g.groups.offsets[blockIdx.z];
+        g.tokens = g.groups.offsets[blockIdx.z + 1];
+        w += (size_t)blockIdx.z * g.n_out * g.ldw;
+        if (t0 >= g.tokens) return;
+    }
     float        acc[4][4] = {};
     for (int k0 = 0; k0 < g.k; k0 += kSimtK) {
         for (int i = threadIdx.x; i < kSimtTile * kSimtK; i += 256) {
@@ -414,13 +497,17 @@ __global__ void __launch_bounds__(256) dense_f32_kernel(DenseGemm g)
             if (n >= g.n_out) continue;
             const float y = acc[i][j] * scale;
             if (ep.kind == DenseKind::kResidual) {
-                ep.residual[(size_t)t * ep.residual_ld + n] += y;
+                const float f = ep.gate ? ep.mult * sigmoid_f32(static_cast<const float*>(ep.gate)[(size_t)t * ep.gate_ld + n] + ep.gate_bias[n]) : 1.f;
+                ep.residual[(size_t)t * ep.residual_ld + n] += f * y;
             }
             else if (ep.kind == DenseKind::kInput && n >= ep.split) {
                 if ((j & 1) == 0) {
                     const float up = n + 1 < g.n_out ? acc[i][j + 1] * scale : 0.f;
-                    static_cast<float*>(ep.act)[(size_t)t * ep.act_ld + ((n - ep.split) >> 1)] = gelu_tanh_f32<false>(y) * up;
+                    static_cast<float*>(ep.act)[(size_t)t * ep.act_ld + ((n - ep.split) >> 1)] = activate<false>(ep, y, up);
                 }
+            }
+            else if (ep.f32_out && n >= ep.f32_from) {
+                ep.f32_out[(size_t)t * ep.f32_ld + n - ep.f32_from] = y;
             }
             else {
                 const bool th = ep.kind == DenseKind::kInput && n >= ep.tanh_lo && n < ep.tanh_hi;
@@ -456,7 +543,8 @@ bool encode_rows(EncodeTiled encode, CUtensorMap* map, const void* ptr, int rows
 
 cudaError_t dense_prepare(int max_smem)
 {
-    return cudaFuncSetAttribute(dense_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+    const cudaError_t e = cudaFuncSetAttribute(dense_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem);
+    return e == cudaSuccess ? cudaFuncSetAttribute(dense_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, max_smem) : e;
 }
 const KernelPreparation g_prepare(dense_prepare);
 
@@ -483,44 +571,65 @@ Plan choose_plan(int tokens, int n_out, int k_blocks, int sms)
     return best;
 }
 
+// The same for groups, whose rows are spread in a way the host does not know: tiles twice as high as the average group
+// (an uneven spread seldom needs a second tile of the same weights), cut unless there are many.
+Plan choose_group_plan(int rows, int groups, int n_out, int sms)
+{
+    const int       average = (rows + groups - 1) / groups;
+    const int       nt      = std::min(kMaxTokens, (2 * average + 15) / 16 * 16);
+    const long long tiles   = (long long)((n_out + kDenseTile - 1) / kDenseTile) * std::min(rows, groups + rows / nt);
+    return {nt, tiles < 4 * sms};
+}
+
 int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
 {
     static const EncodeTiled encode = lookup_encode_tiled();
     if (!encode) return TM_ERR_CUDA;
     if (g.ldw % 8 || g.ldx % 8 || (reinterpret_cast<uintptr_t>(g.w) & 15) || (reinterpret_cast<uintptr_t>(g.x) & 15)) return TM_ERR_INVALID_ARG;
     if (g.ep.kind == DenseKind::kInput && g.ep.split % kDenseTile) return TM_ERR_INVALID_ARG;
+    if (g.x2 && (g.x2_from % kDenseTile || (reinterpret_cast<uintptr_t>(g.x2) & 15))) return TM_ERR_INVALID_ARG;
+    if (g.groups.count > kMaxDenseGroups || (g.groups.count > 0 && (g.ep.ssq || g.ep.ssq_out || g.x2))) return TM_ERR_UNSUPPORTED;
     DenseTcParams p{};
     p.tokens       = g.tokens;
     p.n_out        = g.n_out;
     p.k_blocks     = (g.k + kKBlock - 1) / kKBlock;
-    const Plan plan = choose_plan(g.tokens, g.n_out, p.k_blocks, h->sm_count);
+    const bool grouped = g.groups.count > 0;
+    const Plan plan    = grouped ? choose_group_plan(g.tokens, g.groups.count, g.n_out, h->sm_count) : choose_plan(g.tokens, g.n_out, p.k_blocks, h->sm_count);
+    p.groups           = g.groups;
+    p.x2_tile          = g.x2 ? g.x2_from / kDenseTile : 1 << 30;
+    p.column_tiles     = (g.n_out + kDenseTile - 1) / kDenseTile;
     p.token_tile    = plan.token_tile;
     p.token_tiles   = (g.tokens + p.token_tile - 1) / p.token_tile;
     p.tiles         = (g.n_out + kDenseTile - 1) / kDenseTile * p.token_tiles;
     p.tmem_columns = 32;
     while (p.tmem_columns < 2 * p.token_tile) p.tmem_columns *= 2;
     const size_t stage_b = (size_t)kDenseTile * 128 + (size_t)p.token_tile * 128;
-    p.stages             = (int)(((size_t)h->max_smem - 1024 - sizeof(DenseShared)) / stage_b);
+    const size_t shared  = sizeof(DenseShared) + (grouped ? (size_t)(g.groups.count + 1) * sizeof(int) : 0);
+    p.stages             = (int)(((size_t)h->max_smem - 1024 - shared) / stage_b);
     if (p.stages > kMaxStages) p.stages = kMaxStages;
     if (p.stages < 2) return TM_ERR_UNSUPPORTED;
     const int sms = h->sm_count;
-    if (plan.cut && (size_t)2 * sms * p.token_tile * kDenseTile * 4 <= h->scratch_bytes) {
+    // tiles that tickets have to be there for
+    const long long most = grouped ? (long long)p.column_tiles * std::min(g.tokens, g.groups.count + g.tokens / p.token_tile) : p.tiles;
+    if (plan.cut && most <= (long long)h->counter_ints && (size_t)2 * sms * p.token_tile * kDenseTile * 4 <= h->scratch_bytes) {
         // each CTA gets at least four k blocks
-        p.cut_ctas = (int)std::min<long long>(sms, std::max<long long>(1, (long long)p.tiles * p.k_blocks / 4));
+        p.cut_ctas = grouped ? sms : (int)std::min<long long>(sms, std::max<long long>(1, (long long)p.tiles * p.k_blocks / 4));
     }
     p.grid_tiles        = p.cut_ctas > 0 ? 0 : p.tiles;
-    const int grid_ctas = p.cut_ctas > 0 ? p.cut_ctas : std::min(sms, p.tiles);
+    const int grid_ctas = p.cut_ctas > 0 ? p.cut_ctas : (int)std::min<long long>(sms, most);
     p.scratch  = static_cast<float*>(h->scratch);
     p.tickets  = h->counters;
     p.status   = h->status;
     p.max_wait = h->gemm_wait_cycles > 0 ? h->gemm_wait_cycles : kMaxWaitCycles;
     p.ep       = g.ep;
-    CUtensorMap w_map, x_map;
-    if (!encode_rows(encode, &w_map, g.w, g.n_out, g.k, g.ldw, kDenseTile)) return TM_ERR_CUDA;
+    CUtensorMap w_map, x_map, x2_map;
+    if (!encode_rows(encode, &w_map, g.w, g.n_out * std::max(1, g.groups.count), g.k, g.ldw, kDenseTile)) return TM_ERR_CUDA;
     if (!encode_rows(encode, &x_map, g.x, g.tokens, g.k, g.ldx, p.token_tile)) return TM_ERR_CUDA;
-    const size_t smem = 1024 + (size_t)p.stages * stage_b + sizeof(DenseShared);
+    if (!encode_rows(encode, &x2_map, g.x2 ? g.x2 : g.x, g.tokens, g.k, g.ldx, p.token_tile)) return TM_ERR_CUDA;
+    const size_t smem = 1024 + (size_t)p.stages * stage_b + shared;
     const dim3   grid(grid_ctas);
-    const cudaError_t e = launch_kernel(dense_tc_kernel, grid, dim3(kThreads), smem, st, pdl, p, w_map, x_map);
+    const cudaError_t e = grouped ? launch_kernel(dense_tc_kernel<true>, grid, dim3(kThreads), smem, st, pdl, p, w_map, x_map, x2_map) :
+                                    launch_kernel(dense_tc_kernel<false>, grid, dim3(kThreads), smem, st, pdl, p, w_map, x_map, x2_map);
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;
         return TM_ERR_CUDA;
@@ -536,7 +645,8 @@ int dense_gemm(tm_handle* h, const DenseGemm& g, bool f32, cudaStream_t st, bool
     if (!g.w || !g.x || g.tokens <= 0 || g.n_out <= 0 || g.k <= 0 || g.ldw < g.k || g.ldx < g.k) return TM_ERR_INVALID_ARG;
     if (!f32) return dense_tc(h, g, st, pdl);
     if (g.ep.kind == DenseKind::kResidual && (g.ep.cast || g.ep.ssq_out)) return TM_ERR_UNSUPPORTED;
-    const dim3 grid((g.n_out + kSimtTile - 1) / kSimtTile, (g.tokens + kSimtTile - 1) / kSimtTile);
+    if (g.x2 && g.x2_from % kSimtTile) return TM_ERR_INVALID_ARG;
+    const dim3 grid((g.n_out + kSimtTile - 1) / kSimtTile, (g.tokens + kSimtTile - 1) / kSimtTile, std::max(1, g.groups.count));
     const cudaError_t e = launch_kernel(dense_f32_kernel, grid, dim3(256), 0, st, pdl, g);
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;

@@ -14,9 +14,14 @@ enum class DenseKind : int {
     kF32,       // out[t][n] in fp32
     kInput,     // a layer's input projections: columns [0, split) are stored in the element type (those in
                 // [tanh_lo, tanh_hi) through tanh); from `split` on, columns come in (gate, up) pairs and
-                // act[t][(n - split) / 2] = gelu_tanh(gate) * up
-    kResidual,  // residual[t][n] += y (fp32); optionally also cast[t][n] = residual in the element type and the tile's
-                // part of the row's sum of squares
+                // act[t][(n - split) / 2] = activation(gate, up)
+    kResidual,  // residual[t][n] += y (fp32), or += mult * sigmoid(gate[t][n] + gate_bias[n]) * y where there is a gate;
+                // optionally also cast[t][n] = residual in the element type and the tile's part of the row's sum of squares
+};
+
+enum class DenseActivation : int {
+    kGeluTanh,      // gelu_tanh(gate) * up
+    kClampedSwish,  // g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(slope * g) * (u + 1)
 };
 
 struct DenseEpilogue {
@@ -33,6 +38,11 @@ struct DenseEpilogue {
     int   tanh_lo = 0, tanh_hi = 0, split = 0;
     void* act     = nullptr;
     int   act_ld  = 0;
+    DenseActivation activation = DenseActivation::kGeluTanh;
+    float           limit = 0.f, slope = 0.f;
+    // kStore, kInput: columns from f32_from on go to f32_out[t][n - f32_from] in fp32 instead (0: none)
+    float* f32_out  = nullptr;
+    int    f32_from = 0, f32_ld = 0;
 
     float* residual    = nullptr;
     int    residual_ld = 0;
@@ -40,13 +50,30 @@ struct DenseEpilogue {
     int    cast_ld     = 0;
     float* ssq_out     = nullptr;  // [column tile of 128][ssq_out_stride]
     int    ssq_out_stride = 0;
+    const void*  gate      = nullptr;
+    int          gate_ld   = 0;
+    const float* gate_bias = nullptr;
+    float        mult      = 1.f;
 };
+
+// Products of several row groups, each with a weight of its own (the experts of a mixture): group g's rows are
+// [offsets[g], offsets[g + 1]) of x and of the output, its weight rows [g * n_out, (g + 1) * n_out) of w.  The offsets are
+// read on the device; `tokens` of the call is an upper bound on offsets[groups].
+struct DenseGroups {
+    int        count   = 0;  // 0: a plain product
+    const int* offsets = nullptr;
+};
+constexpr int kMaxDenseGroups = 1024;
 
 struct DenseGemm {
     const void* w = nullptr;  // [n_out][ldw]
     const void* x = nullptr;  // [tokens][ldx]
     int         ldw = 0, ldx = 0;
     int         tokens = 0, n_out = 0, k = 0;
+    // output columns from x2_from on (a multiple of kDenseTile; 0: none) are products with x2 instead, rows as far apart as x's
+    const void* x2      = nullptr;
+    int         x2_from = 0;
+    DenseGroups   groups;
     DenseEpilogue ep;
 };
 

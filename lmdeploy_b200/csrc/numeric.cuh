@@ -32,6 +32,13 @@ template<bool FAST> __device__ __forceinline__ float gelu_tanh_f32(float z)
     return FAST ? __fdividef(z, 1.f + __expf(-u2)) : z / (1.f + expf(-u2));
 }
 
+// g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(slope * g) * (u + 1)
+template<bool FAST> __device__ __forceinline__ float clamped_swish_f32(float gate, float up, float limit, float slope)
+{
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit) + 1.f;
+    return (FAST ? __fdividef(g, 1.f + __expf(-slope * g)) : g / (1.f + expf(-slope * g))) * u;
+}
+
 __device__ __forceinline__ float warp_sum(float v)
 {
 #pragma unroll

@@ -261,12 +261,18 @@ int attend(tm_handle* h, const WindowKernelParams& p, cudaStream_t st)
 
 }  // namespace
 
-int window_attention_prefill(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st)
+int window_attention_write(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st)
 {
     if (!valid(a, c)) return TM_ERR_UNSUPPORTED;
     const WindowKernelParams p{a, c};
-    int rc = c.f32 ? write_and_pool<float>(h, p, st) : write_and_pool<__nv_bfloat16>(h, p, st);
+    return c.f32 ? write_and_pool<float>(h, p, st) : write_and_pool<__nv_bfloat16>(h, p, st);
+}
+
+int window_attention_prefill(tm_handle* h, const WindowAttention& a, const MixerCall& c, cudaStream_t st)
+{
+    const int rc = window_attention_write(h, a, c, st);
     if (rc != TM_OK) return rc;
+    const WindowKernelParams p{a, c};
     if (window_attention_tc_supported(a, c)) return window_attention_tc(h, a, c, st);
     return c.f32 ? attend<float>(h, p, st) : attend<__nv_bfloat16>(h, p, st);
 }
@@ -275,9 +281,9 @@ int window_attention_decode(tm_handle* h, const WindowAttention& a, const MixerC
 {
     if (!valid(a, c)) return TM_ERR_UNSUPPORTED;
     if (window_attention_step_supported(a, c)) return window_attention_step(h, a, c, st);
-    const WindowKernelParams p{a, c};
-    const int rc = c.f32 ? write_and_pool<float>(h, p, st) : write_and_pool<__nv_bfloat16>(h, p, st);
+    const int rc = window_attention_write(h, a, c, st);
     if (rc != TM_OK) return rc;
+    const WindowKernelParams p{a, c};
     return c.f32 ? attend<float>(h, p, st) : attend<__nv_bfloat16>(h, p, st);
 }
 
