@@ -598,6 +598,8 @@ TM_API int tm_llama_check_status(tm_llama* m, void* stream, unsigned* word);
  * (lmdeploy_b200/generate.py) and the trace replay (bin/trace_run) use.  tm_model_open chooses by what the folder holds:
  *   config.json with "architecture": "Rumazen" and model.safetensors   the config-driven decoder (window attention with
  *       pooled blocks, generalised delta rule, parallel layers); bf16, or everything in fp32
+ *   ... with "architecture": "Fopinex"   the same decoder with gated branches (attention within chunks with sigmoid weights
+ *       mixed across heads, gated linear attention, mixture of experts); bf16, or everything in fp32
  *   config.ini and weight files                                        a TurboMind W4A16 workspace (tm_llama)
  * tm_model_close frees what tm_model_open and tm_decoder_create_random made; a tm_llama keeps its own functions, and
  * tm_llama_as_model lends its tm_model.
@@ -656,7 +658,7 @@ TM_API int tm_replay_destroy(tm_replay* r);
 TM_API int tm_replay_step(tm_replay* r, uint64_t id, const int* tokens, int count, const int* want, int want_count, float* logits);
 TM_API int tm_replay_end(tm_replay* r, uint64_t id);
 /* A config-driven decoder with random weights (seeded, on the device), for measurements: `config_json` is the text of a
- * config.json; a delta-rule mixer then names the rank of its decay projection itself ("rank", default 16). */
+ * config.json; a recurrent mixer then names the rank of its decay projection itself ("rank", default 16). */
 TM_API int tm_decoder_create_random(tm_model** out, tm_handle* h, const char* config_json, const tm_model_options* opt,
                                     unsigned long long seed);
 
@@ -703,6 +705,57 @@ typedef struct tm_delta_rule_params {
     int          r_col, k_col, v_col, a_col, g_col, w1_col;
 } tm_delta_rule_params;
 TM_API int tm_delta_rule(tm_handle* h, const tm_delta_rule_params* d, const tm_mixer_call* c, void* stream);
+/* Attention without a softmax: position i sees the tokens from the start of its chunk of `chunk` positions (0: from the first)
+ * to itself; head g gives key j the weight sigmoid(scale q.k + bias[g]); head h applies sum_g talk[h][g] weight_g to the
+ * values of its own kv head (h / (heads / kv_heads)).  reads_only: the rows of the new tokens are in the cache already (keys
+ * and values of another layer), nothing is written.  Position p is cached in row p % ring of [kv head][ring][dim or vdim]. */
+typedef struct tm_chunk_attention_params {
+    int          heads, kv_heads, dim, vdim;
+    float        scale;
+    int          chunk;
+    const float *bias, *talk;  /* device [heads], [heads][heads] */
+    const void*  talk_half;    /* device fp16 [P][P], P = heads rounded up to 16, zeros beyond the heads; null: made by the call */
+    int          reads_only, ring;
+    size_t       k_off, v_off;
+    int          q_col, k_col, v_col;
+    int          query_tiles;  /* tiles of 128 queries the tensor-core prefill works on at a time (0: all)               */
+} tm_chunk_attention_params;
+TM_API int tm_chunk_attention(tm_handle* h, const tm_chunk_attention_params* a, const tm_mixer_call* c, void* stream);
+/* Gated linear attention, fp32 state float [head][value dim][key dim] (zero at history 0):
+ *   S <- diag(sigmoid(w2 . a + bias)^(1 / tau)) S + k v^T,   o = S^T (scale q);   out = o / rms(o) * norm * silu(g) per head */
+typedef struct tm_gated_linear_params {
+    int          heads, dim, vdim, rank;
+    const void*  w2; /* device [heads * dim][w2_ld] */
+    int          w2_ld;
+    const float *bias, *norm; /* device [heads * dim], [vdim] */
+    float        norm_eps, scale, tau;
+    size_t       state_off;
+    int          q_col, k_col, v_col, g_col, a_col;
+} tm_gated_linear_params;
+TM_API int tm_gated_linear(tm_handle* h, const tm_gated_linear_params* d, const tm_mixer_call* c, void* stream);
+/* Mixture of experts behind an elementwise gate: s = softmax(logits); of the experts + identity router outputs, `top` are
+ * chosen by s + correction out of the `keep` of `groups` groups of neighbours with the highest best choice score;
+ *   x += mult * sigmoid(gate + gate_bias) * sum over the chosen e of s_e f_e(input)
+ * f_e(h) = down_e(g sigmoid(slope g) (u + 1)), g = min(gate_e h, limit), u = clamp(up_e h, -limit, limit); the last `identity`
+ * outputs are f(h) = h.  w_experts: rows (gate 0, up 0, gate 1, ...) of every expert in turn; norm_out (optional) =
+ * x / sqrt(mean x^2 + norm_eps) * norm_weight.  x, logits, vectors in fp32, the rest in `dtype`; ld multiples of 8. */
+typedef struct tm_moe_params {
+    int          tokens, width, ff, experts, identity, top, groups, keep;
+    float        limit, slope, mult, norm_eps;
+    float*       x;          /* [tokens][width] */
+    const float* logits;     /* [tokens][logits_ld] */
+    int          logits_ld;
+    const void*  input;      /* [tokens][input_ld] */
+    int          input_ld;
+    const void*  gate;       /* [tokens][gate_ld] */
+    int          gate_ld;
+    const float *gate_bias, *correction, *norm_weight;
+    const void*  w_experts;  /* [experts][2 ff][input_ld] */
+    const void*  w_down;     /* [experts][width][ff rounded up to 8] */
+    void*        norm_out;   /* [tokens][input_ld] */
+    int          dtype;
+} tm_moe_params;
+TM_API int tm_moe(tm_handle* h, const tm_moe_params* m, void* stream);
 /* out[t][n] = sum_k x[t][k] * w[n][k]: bf16 on the tcgen05 tensor core (ld multiples of 8, 16-byte aligned; out in bf16, or
  * in fp32 with out_f32), or fp32 throughout */
 TM_API int tm_gemm_dense(tm_handle* h, void* out, int out_ld, int out_f32, const void* x, int x_ld, const void* w, int w_ld, int tokens,

@@ -791,13 +791,26 @@ int tm_decoder::decode(const tm_llama_decode_state& st, int n_steps, bool use_gr
 // ---------------------------------------------------------------------------------------------------- mechanisms alone
 namespace {
 
-// Spans of a call on the device, and `extra` bytes of scratch behind them, in the handle's operator buffer
+// `bytes` of the handle's operator buffer, on 256-byte boundaries
+bool operator_buffer(tm_handle* h, size_t bytes)
+{
+    if (bytes <= h->op_buffer_bytes) return true;
+    if (h->op_buffer) cudaFree(h->op_buffer);  // waits for the work that uses it
+    h->op_buffer = nullptr, h->op_buffer_bytes = 0;
+    if (cudaMalloc(&h->op_buffer, bytes) != cudaSuccess) return false;
+    h->op_buffer_bytes = bytes;
+    return true;
+}
+
+// Spans and query tiles of a call on the device, and scratch behind them, in the handle's operator buffer
 struct DeviceSpans {
     MixerCall c;
     void*     scratch = nullptr;
     int       rc      = TM_OK;
 
-    DeviceSpans(tm_handle* h, const tm_mixer_call& call, size_t extra_per_token, cudaStream_t s)
+    // scratch_bytes(call) -> bytes, asked when the call's sizes are known
+    template<typename Bytes>
+    DeviceSpans(tm_handle* h, const tm_mixer_call& call, cudaStream_t s, Bytes scratch_bytes)
     {
         if (!call.proj || !call.out || call.batch <= 0 || !call.history || !call.n || !call.slabs
             || (call.dtype != TM_DTYPE_BF16 && call.dtype != TM_DTYPE_F32)) {
@@ -815,21 +828,25 @@ struct DeviceSpans {
         }
         if (rc == TM_OK && c.tokens == 0) rc = TM_ERR_INVALID_ARG;
         if (rc != TM_OK) return;
-        const size_t spans_bytes = round_up_bytes(sp.size() * sizeof(SeqSpan)), need = spans_bytes + extra_per_token * c.tokens;
-        if (need > h->op_buffer_bytes) {
-            if (h->op_buffer) cudaFree(h->op_buffer);  // waits for the work that uses it
-            h->op_buffer = nullptr, h->op_buffer_bytes = 0;
-            if (cudaMalloc(&h->op_buffer, need) != cudaSuccess) {
-                rc = TM_ERR_CUDA;
-                return;
-            }
-            h->op_buffer_bytes = need;
+        std::vector<QueryTile> tiles;
+        for (int b = 0; !call.decode && b < call.batch; ++b) {
+            for (int q = 0; q < call.n[b]; q += 128) tiles.push_back({b, q});
+        }
+        c.proj = call.proj, c.proj_ld = call.proj_ld, c.out = call.out, c.out_ld = call.out_ld, c.batch = call.batch;
+        c.f32 = call.dtype == TM_DTYPE_F32, c.tile_count = (int)tiles.size();
+        const size_t spans_bytes = round_up_bytes(sp.size() * sizeof(SeqSpan)), tiles_bytes = round_up_bytes(tiles.size() * sizeof(QueryTile));
+        if (!operator_buffer(h, spans_bytes + tiles_bytes + scratch_bytes(c))) {
+            rc = TM_ERR_CUDA;
+            return;
         }
         SeqSpan* d = static_cast<SeqSpan*>(h->op_buffer);
-        scratch    = static_cast<char*>(h->op_buffer) + spans_bytes;
-        if (cudaMemcpyAsync(d, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess) rc = TM_ERR_CUDA;
-        c.proj = call.proj, c.proj_ld = call.proj_ld, c.out = call.out, c.out_ld = call.out_ld, c.spans = d, c.batch = call.batch;
-        c.f32 = call.dtype == TM_DTYPE_F32;
+        void* const t = static_cast<char*>(h->op_buffer) + spans_bytes;
+        scratch       = static_cast<char*>(t) + tiles_bytes;
+        c.spans = d, c.tiles = static_cast<QueryTile*>(t);
+        if (cudaMemcpyAsync(d, sp.data(), sp.size() * sizeof(SeqSpan), cudaMemcpyHostToDevice, s) != cudaSuccess
+            || (!tiles.empty() && cudaMemcpyAsync(t, tiles.data(), tiles.size() * sizeof(QueryTile), cudaMemcpyHostToDevice, s) != cudaSuccess)) {
+            rc = TM_ERR_CUDA;
+        }
     }
 };
 
@@ -839,7 +856,7 @@ extern "C" int tm_window_attention(tm_handle* h, const tm_window_attention_param
 {
     if (!h || !q || !call) return TM_ERR_INVALID_ARG;
     const cudaStream_t s = (cudaStream_t)stream;
-    DeviceSpans        sp(h, *call, 0, s);
+    DeviceSpans        sp(h, *call, s, [](const MixerCall&) { return (size_t)0; });
     if (sp.rc != TM_OK) return sp.rc;
     WindowAttention a;
     a.heads = q->heads, a.kv_heads = q->kv_heads, a.dim = q->dim, a.vdim = q->vdim, a.rot_dims = q->rot_dims, a.inv_freq = q->inv_freq;
@@ -862,7 +879,94 @@ extern "C" int tm_delta_rule(tm_handle* h, const tm_delta_rule_params* q, const 
     d.heads = q->heads, d.dim = q->dim, d.rank = q->rank, d.w2 = q->w2, d.w2_ld = q->w2_ld, d.w0 = q->w0, d.a_bias = q->a_bias, d.norm = q->norm;
     d.norm_eps = q->norm_eps, d.unit_eps = q->unit_eps, d.decay_scale = q->decay_scale, d.state_off = q->state_off;
     d.r_col = q->r_col, d.k_col = q->k_col, d.v_col = q->v_col, d.a_col = q->a_col, d.g_col = q->g_col, d.w1_col = q->w1_col;
-    DeviceSpans sp(h, *call, call->decode ? 0 : delta_rule_scratch_floats(d) * sizeof(float), s);
+    DeviceSpans sp(h, *call, s, [&](const MixerCall& c) { return call->decode ? 0 : delta_rule_scratch_floats(d) * sizeof(float) * c.tokens; });
     if (sp.rc != TM_OK) return sp.rc;
     return call->decode ? delta_rule_decode(h, d, sp.c, s) : delta_rule_prefill(h, d, sp.c, static_cast<float*>(sp.scratch), s);
+}
+
+extern "C" int tm_chunk_attention(tm_handle* h, const tm_chunk_attention_params* q, const tm_mixer_call* call, void* stream)
+{
+    if (!h || !q || !call || !q->bias || !q->talk || q->heads <= 0 || q->heads > 1024) return TM_ERR_INVALID_ARG;
+    const cudaStream_t s = (cudaStream_t)stream;
+    ChunkAttention     a;
+    a.heads = q->heads, a.kv_heads = q->kv_heads, a.dim = q->dim, a.vdim = q->vdim, a.scale = q->scale, a.chunk = q->chunk, a.bias = q->bias;
+    a.talk = q->talk, a.writes = !q->reads_only, a.ring = q->ring, a.k_off = q->k_off, a.v_off = q->v_off;
+    a.q_col = q->q_col, a.k_col = q->k_col, a.v_col = q->v_col;
+    const int    pad        = talk_pad(a.heads);
+    const size_t talk_bytes = round_up_bytes((size_t)pad * pad * 2);
+    DeviceSpans  sp(h, *call, s, [&](const MixerCall& c) {
+        a.weights_bytes = call->decode ? 0 : chunk_attention_scratch(a, c.max_context, c.f32) * (q->query_tiles > 0 ? std::min(q->query_tiles, c.tile_count) : c.tile_count);
+        return talk_bytes + a.weights_bytes;
+    });
+    if (sp.rc != TM_OK) return sp.rc;
+    for (int b = 0; b < call->batch; ++b) {
+        // everything a query of the call may see has to be in the ring
+        const int end = call->history[b] + call->n[b], need = a.chunk > 0 ? std::min(end, a.chunk - 1 + call->n[b]) : end;
+        if (need > a.ring) return TM_ERR_INVALID_ARG;
+    }
+    a.talk_half = q->talk_half;
+    if (!a.talk_half) {
+        a.talk_half = sp.scratch;
+        talk_half_kernel<<<1, 256, 0, s>>>(static_cast<__half*>(sp.scratch), a.talk, a.heads, pad);
+    }
+    a.weights = static_cast<char*>(sp.scratch) + talk_bytes;
+    return call->decode ? chunk_attention_decode(h, a, sp.c, s) : chunk_attention_prefill(h, a, sp.c, s);
+}
+
+extern "C" int tm_gated_linear(tm_handle* h, const tm_gated_linear_params* q, const tm_mixer_call* call, void* stream)
+{
+    if (!h || !q || !call || !q->w2 || !q->bias || !q->norm || !(q->tau > 0.f)) return TM_ERR_INVALID_ARG;
+    const cudaStream_t s = (cudaStream_t)stream;
+    GatedLinear        d;
+    d.heads = q->heads, d.dim = q->dim, d.vdim = q->vdim, d.rank = q->rank, d.w2 = q->w2, d.w2_ld = q->w2_ld, d.bias = q->bias, d.norm = q->norm;
+    d.norm_eps = q->norm_eps, d.scale = q->scale, d.tau = q->tau, d.state_off = q->state_off;
+    d.q_col = q->q_col, d.k_col = q->k_col, d.v_col = q->v_col, d.g_col = q->g_col, d.a_col = q->a_col;
+    DeviceSpans sp(h, *call, s, [&](const MixerCall& c) { return call->decode ? 0 : gated_linear_scratch_floats(d) * sizeof(float) * c.tokens; });
+    if (sp.rc != TM_OK) return sp.rc;
+    return call->decode ? gated_linear_decode(h, d, sp.c, s) : gated_linear_prefill(h, d, sp.c, static_cast<float*>(sp.scratch), s);
+}
+
+extern "C" int tm_moe(tm_handle* h, const tm_moe_params* q, void* stream)
+{
+    if (!h || !q || !q->x || !q->logits || !q->input || !q->gate || !q->gate_bias || !q->correction || !q->w_experts || !q->w_down || q->tokens < 0
+        || q->experts <= 0 || q->top <= 0 || (q->dtype != TM_DTYPE_BF16 && q->dtype != TM_DTYPE_F32)) {
+        return TM_ERR_INVALID_ARG;
+    }
+    if (q->tokens == 0) return TM_OK;
+    const cudaStream_t s   = (cudaStream_t)stream;
+    const bool         f32 = q->dtype == TM_DTYPE_F32;
+    const size_t       es = f32 ? 4 : 2, T = (size_t)q->tokens, rows = T * q->top;
+    const int          act_ld = round_up(q->ff, 8);
+    size_t             at     = 0;
+    auto take = [&](size_t bytes) {
+        const size_t begin = at;
+        at += round_up_bytes(bytes);
+        return begin;
+    };
+    const size_t counts = take((size_t)q->experts * 4), offsets = take((size_t)(q->experts + 1) * 4), slots = take(rows * 4), weights = take(rows * 4),
+                 ranks = take(rows * 4), sorted = take(rows * q->input_ld * es), act = take(rows * act_ld * es), out = take(rows * q->width * es);
+    if (!operator_buffer(h, at)) return TM_ERR_CUDA;
+    char* const base = static_cast<char*>(h->op_buffer);
+    MoeRows     m;
+    m.counts = (int*)(base + counts), m.offsets = (int*)(base + offsets), m.slots = (int*)(base + slots), m.weights = (float*)(base + weights);
+    m.ranks = (int*)(base + ranks), m.sorted = base + sorted, m.ld = q->input_ld;
+    const MoeRouter r{q->experts, q->identity, q->top, q->groups, q->keep, q->correction};
+    if (cudaMemsetAsync(m.counts, 0, (size_t)q->experts * 4, s) != cudaSuccess) return TM_ERR_CUDA;
+    int rc = moe_dispatch(h, r, m, q->logits, q->logits_ld, q->input, q->tokens, q->width, f32, s, false);
+    if (rc != TM_OK) return rc;
+    DenseGemm u;
+    u.w = q->w_experts, u.ldw = q->input_ld, u.x = m.sorted, u.ldx = m.ld, u.tokens = (int)rows, u.n_out = 2 * q->ff, u.k = q->width;
+    u.groups.count = q->experts, u.groups.offsets = m.offsets;
+    u.ep.kind = DenseKind::kInput, u.ep.act = base + act, u.ep.act_ld = act_ld;
+    u.ep.activation = DenseActivation::kClampedSwish, u.ep.limit = q->limit, u.ep.slope = q->slope;
+    if ((rc = dense_gemm(h, u, f32, s, false)) != TM_OK) return rc;
+    DenseGemm d;
+    d.w = q->w_down, d.ldw = act_ld, d.x = base + act, d.ldx = act_ld, d.tokens = (int)rows, d.n_out = q->width, d.k = q->ff, d.groups = u.groups;
+    d.ep.kind = DenseKind::kStore, d.ep.out = base + out, d.ep.out_ld = q->width;
+    if ((rc = dense_gemm(h, d, f32, s, false)) != TM_OK) return rc;
+    RowsCall c;
+    c.x = q->x, c.tokens = q->tokens, c.width = q->width, c.expert_rows = base + out, c.input = q->input, c.input_ld = q->input_ld, c.slots = m.slots;
+    c.weights = m.weights, c.top = q->top, c.gate = q->gate, c.gate_ld = q->gate_ld, c.gate_bias = q->gate_bias, c.mult = q->mult;
+    c.weight_a = q->norm_weight, c.out_a = q->norm_weight ? q->norm_out : nullptr, c.out_ld = q->input_ld, c.eps = q->norm_eps;
+    return norm_rows(h, c, f32, s, false);
 }

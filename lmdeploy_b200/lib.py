@@ -199,6 +199,29 @@ class TmDeltaRuleParams(C.Structure):
         + [(n, C.c_int) for n in ("r_col", "k_col", "v_col", "a_col", "g_col", "w1_col")]
 
 
+class TmChunkAttentionParams(C.Structure):
+    """ctypes mirror of ``tm_chunk_attention_params``."""
+    _fields_ = [(n, C.c_int) for n in ("heads", "kv_heads", "dim", "vdim")] + [("scale", C.c_float), ("chunk", C.c_int)] \
+        + [(n, C.c_void_p) for n in ("bias", "talk", "talk_half")] + [("reads_only", C.c_int), ("ring", C.c_int)] \
+        + [("k_off", C.c_size_t), ("v_off", C.c_size_t)] + [(n, C.c_int) for n in ("q_col", "k_col", "v_col", "query_tiles")]
+
+
+class TmGatedLinearParams(C.Structure):
+    """ctypes mirror of ``tm_gated_linear_params``."""
+    _fields_ = [(n, C.c_int) for n in ("heads", "dim", "vdim", "rank")] + [("w2", C.c_void_p), ("w2_ld", C.c_int), ("bias", C.c_void_p),
+                ("norm", C.c_void_p), ("norm_eps", C.c_float), ("scale", C.c_float), ("tau", C.c_float), ("state_off", C.c_size_t)] \
+        + [(n, C.c_int) for n in ("q_col", "k_col", "v_col", "g_col", "a_col")]
+
+
+class TmMoeParams(C.Structure):
+    """ctypes mirror of ``tm_moe_params``."""
+    _fields_ = [(n, C.c_int) for n in ("tokens", "width", "ff", "experts", "identity", "top", "groups", "keep")] \
+        + [(n, C.c_float) for n in ("limit", "slope", "mult", "norm_eps")] \
+        + [("x", C.c_void_p), ("logits", C.c_void_p), ("logits_ld", C.c_int), ("input", C.c_void_p), ("input_ld", C.c_int),
+           ("gate", C.c_void_p), ("gate_ld", C.c_int)] \
+        + [(n, C.c_void_p) for n in ("gate_bias", "correction", "norm_weight", "w_experts", "w_down", "norm_out")] + [("dtype", C.c_int)]
+
+
 # name -> (restype, argtypes); must list every symbol declared in include/tm_b200.h
 SIGNATURES = {
     "tm_create": (_i, [C.POINTER(_vp), _i]),
@@ -238,6 +261,9 @@ SIGNATURES = {
     "tm_decoder_create_random": (_i, [C.POINTER(_vp), _vp, C.c_char_p, C.POINTER(TmModelOptions), C.c_ulonglong]),
     "tm_window_attention": (_i, [_vp, C.POINTER(TmWindowAttentionParams), C.POINTER(TmMixerCall), _vp]),
     "tm_delta_rule": (_i, [_vp, C.POINTER(TmDeltaRuleParams), C.POINTER(TmMixerCall), _vp]),
+    "tm_chunk_attention": (_i, [_vp, C.POINTER(TmChunkAttentionParams), C.POINTER(TmMixerCall), _vp]),
+    "tm_gated_linear": (_i, [_vp, C.POINTER(TmGatedLinearParams), C.POINTER(TmMixerCall), _vp]),
+    "tm_moe": (_i, [_vp, C.POINTER(TmMoeParams), _vp]),
     "tm_gemm_dense": (_i, [_vp, _vp, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _vp]),
     "tm_batch_destroy": (_i, [_vp]),
     "tm_batch_submit": (_i, [_vp, C.POINTER(TmRequest)]),
