@@ -740,6 +740,32 @@ def device_ms(fn, stream, steps, warmup, flush=None):
     return total / steps
 
 
+class KernelTable:
+    """Timings of single kernels as shares of the measured peak that bounds them (HBM or bf16 GEMM)."""
+
+    def __init__(self, peaks, like_key):
+        self.peaks, self.like_key, self.rows = peaks, like_key, []
+
+    def add(self, name, ms, flops=0.0, nbytes=0.0, like=False):
+        tf, gb, peaks = flops / ms * 1e-9, nbytes / ms * 1e-6, self.peaks
+        bound = "tensor" if flops / (peaks["bf16_tflops"] * 1e12) > nbytes / (peaks["hbm_gbs"] * 1e9) else "hbm"
+        frac = tf / peaks["bf16_tflops"] if bound == "tensor" else gb / peaks["hbm_gbs"]
+        self.rows.append({"kernel": name, self.like_key: like, "us": round(ms * 1e3, 2), "bound": bound, "tflops": round(tf, 1), "gbs": round(gb, 1),
+                          "frac": round(frac, 3)})
+
+
+def mixer_call(proj, ld, out, out_ld, hist, n, slabs, decode):
+    """-> (tm_mixer_call over these tensors, what has to stay alive with it)"""
+    import ctypes as C
+    from lmdeploy_b200 import lib as l
+    c = l.TmMixerCall()
+    c.proj, c.proj_ld, c.out, c.out_ld, c.batch = proj.data_ptr(), ld, out.data_ptr(), out_ld, len(n)
+    c.history, c.n = (C.c_int * len(n))(*hist), (C.c_int * len(n))(*n)
+    c.slabs = (C.c_void_p * len(n))(*[s.data_ptr() for s in slabs])
+    c.dtype, c.decode = l.TM_DTYPE_BF16, int(decode)
+    return c, (proj, out, slabs)
+
+
 def rumazen_kernels(device, stream, args, peaks, flush):
     """The kernels of the Rumazen layers one at a time, each with the like kernel of the W4A16 LLaMA beside it at equal
     size: achieved share of the measured peak (HBM for decode, bf16 GEMM for prefill contractions)."""
@@ -751,15 +777,9 @@ def rumazen_kernels(device, stream, args, peaks, flush):
     st = C.c_void_p(stream.cuda_stream)
     W, FF, H, G, D = 4096, 11008, 32, 8, 128
     K, Wm = args.steps, args.warmup
-    bf, rows = torch.bfloat16, []
+    bf, table = torch.bfloat16, KernelTable(peaks, "like_kernel_of_llama")
+    add, call = table.add, mixer_call
     g = torch.Generator(device=device).manual_seed(1)
-
-    def add(name, ms, flops=0.0, nbytes=0.0, like=False):
-        tf, gb = flops / ms * 1e-9, nbytes / ms * 1e-6
-        bound = "tensor" if flops / (peaks["bf16_tflops"] * 1e12) > nbytes / (peaks["hbm_gbs"] * 1e9) else "hbm"
-        frac = tf / peaks["bf16_tflops"] if bound == "tensor" else gb / peaks["hbm_gbs"]
-        rows.append(dict(kernel=name, like_kernel_of_llama=like, us=round(ms * 1e3, 2), bound=bound, tflops=round(tf, 1), gbs=round(gb, 1),
-                         frac=round(frac, 3)))
 
     # ---- dense GEMMs: gate/up-sized input projection and down-sized output projection
     for n, k in ((2 * FF, W), (W, FF)):
@@ -777,15 +797,6 @@ def rumazen_kernels(device, stream, args, peaks, flush):
         del w, lin
 
     # ---- window attention
-    def call(proj, ld, out, out_ld, hist, n, slabs, decode):
-        c = l.TmMixerCall()
-        keep = (proj, out, slabs)
-        c.proj, c.proj_ld, c.out, c.out_ld, c.batch = proj.data_ptr(), ld, out.data_ptr(), out_ld, len(n)
-        c.history, c.n = (C.c_int * len(n))(*hist), (C.c_int * len(n))(*n)
-        c.slabs = (C.c_void_p * len(n))(*[s.data_ptr() for s in slabs])
-        c.dtype, c.decode = l.TM_DTYPE_BF16, int(decode)
-        return c, keep
-
     def window(size, pool, softcap, context, portion):
         p = l.TmWindowAttentionParams()
         freq = (500000.0 ** (-2.0 * torch.arange(D // 2, dtype=torch.float64) / D)).float().to(device)
@@ -870,14 +881,191 @@ def rumazen_kernels(device, stream, args, peaks, flush):
         ms = device_ms(lambda: l.check(l.lib.tm_delta_rule(h.ptr, C.byref(p), C.byref(c), st), "delta"), stream, K, Wm, flush if decode else None)
         nbytes = B * (t * (ld * 2.0 + n * 2.0) + n * dim * 8.0) + n * rank * 2.0
         add(f"delta_step_kernel, batch {B}" if decode else f"delta rule prefill (decay GEMM + scan + finish), {B} x {t} tokens", ms, 0.0, nbytes)
-    return rows
+    return table.rows
+
+
+def decoder_throughput(cfg, device, stream, K, Wm, world, ctx, rng):
+    """A config-driven model with random weights: prefill, decode steps behind `ctx` tokens, and the step at batch 64 end to
+    end -> (table, ms of the step at batch 64, end-to-end tokens/s, kernels launched in the timed decode steps)"""
+    from lmdeploy_b200 import decoder
+    res, launches = {}, 0
+    model = decoder.Model.random(cfg, "bfloat16", 64, ctx + 512, 4096, device)
+    slabs = torch.zeros(64, -(-model.slab_bytes // 256) * 256, dtype=torch.uint8, device=device)
+    addr = [slabs[b].data_ptr() for b in range(64)]
+    prompt = list(map(int, rng.integers(0, cfg["vocab"], 4096)))
+    for B, t in ((1, 1024), (1, 4096), (4, 1024)):
+        ms = device_ms(lambda: model.prefill([prompt[:t]] * B, [0] * B, addr[:B]), stream, max(3, K // 4), Wm)
+        res[f"prefill {B} x {t}"] = dict(ms=round(ms, 3), tokens_per_s=round(B * t / ms * 1e3, 1))
+    for B in (1, 16, 64):
+        # every sequence goes its own way: its first token is forced
+        st = model.new_state(addr[:B], [ctx] * B, 400, [list(map(int, rng.integers(0, cfg["vocab"], B)))] + [[-1] * B] * 399)
+        model.decode(st, Wm, True, stream.cuda_stream)
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        barrier(world)
+        e0.record(stream)
+        model.decode(st, K, True, stream.cuda_stream)
+        e1.record(stream)
+        torch.cuda.synchronize()
+        ms = max_over_ranks(e0.elapsed_time(e1), world) / K
+        launches += model.last_launches()
+        res[f"decode batch {B} at {ctx}"] = dict(ms=round(ms, 4), tokens_per_s=round(B / ms * 1e3, 1), launches=model.last_launches() // K)
+    # end to end: the step's input tokens from pinned host memory, the drawn tokens back, every step
+    st = model.new_state(addr, [ctx] * 64, 400, np.full((400, 64), 0, np.int32))
+    host_in, host_out = torch.randint(0, cfg["vocab"], (64,), dtype=torch.int32).pin_memory(), torch.empty(64, dtype=torch.int32).pin_memory()
+
+    def e2e_step(i):
+        st.forced_ids[i].copy_(host_in, non_blocking=True)
+        model.decode(st, 1, True, stream.cuda_stream)
+        host_out.copy_(st.output_ids[i], non_blocking=True)
+        stream.synchronize()
+
+    for i in range(Wm):
+        e2e_step(i)
+    t0 = time.time()
+    for i in range(Wm, Wm + K):
+        e2e_step(i)
+    e2e = 64 * K / (time.time() - t0)
+    model.check_status()
+    model.close()
+    return res, ms, e2e, launches
+
+
+def fopinex_config(layers=8):
+    """the size of rumazen_config: same width, depth, attention heads, recurrent state and feed-forward columns per token"""
+    mlp = dict(kind="moe", expert=dict(ff=2752, limit=7.0), router=dict(experts=30, identity=2, top=4, groups=dict(count=4, keep=2)))
+    attn = dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=2048))
+    gla = dict(heads=32, dim=64, vdim=128, tau=16.0, rank=16)
+    return dict(architecture="Fopinex", vocab=32000, width=4096, norm=dict(eps=1e-6), residual_mult=0.5,
+                layers=[dict(type="gla" if i % 4 else "attention", mixer=gla if i % 4 else (dict(attn, kv_from=0) if i else attn), mlp=mlp)
+                        for i in range(layers)])
+
+
+def fopinex_kernels(device, stream, args, peaks, flush):
+    """The kernels of the Fopinex layers one at a time (bytes and products as the mechanism needs them at the least)."""
+    import ctypes as C
+    from lmdeploy_b200 import lib as l
+    h, st = l.default_handle(device), C.c_void_p(stream.cuda_stream)
+    W, H, G, D, K, Wm, bf = 4096, 32, 8, 128, args.steps, args.warmup, torch.bfloat16
+    table = KernelTable(peaks, "like_kernel_of_rumazen")
+    add = table.add
+    g = torch.Generator(device=device).manual_seed(2)
+
+    # ---- chunk attention
+    bias, talk = torch.randn(H, device=device, generator=g) - 4, torch.randn(H, H, device=device, generator=g)
+    half = talk.half()
+    ld = (H + 2 * G) * D
+
+    def attention(chunk, context, portion):
+        p = l.TmChunkAttentionParams()
+        p.heads, p.kv_heads, p.dim, p.vdim, p.scale, p.chunk = H, G, D, D, D ** -0.5, chunk
+        p.bias, p.talk, p.talk_half = bias.data_ptr(), talk.data_ptr(), half.data_ptr()
+        p.ring = -(-(min(context, chunk + portion) if chunk else context) // 128) * 128
+        p.v_off = G * p.ring * D * 2
+        p.q_col, p.k_col, p.v_col = 0, H * D, (H + G) * D
+        return p, 2 * p.v_off
+
+    for B, S in ((8, 2048), (1, 16384)):
+        p, nbytes = attention(2048, S, S)
+        slabs = [torch.zeros(nbytes, dtype=torch.uint8, device=device) for _ in range(B)]
+        proj, out = torch.randn(B * S, ld, device=device, generator=g).to(bf), torch.empty(B * S, H * D, dtype=bf, device=device)
+        c, keep = mixer_call(proj, ld, out, H * D, [0] * B, [S] * B, slabs, False)
+        ms = device_ms(lambda: l.check(l.lib.tm_chunk_attention(h.ptr, C.byref(p), C.byref(c), st), "attention"), stream, K, Wm)
+        pairs = B * S // 2048 * 2048 * 2049 / 2
+        add(f"chunk attention prefill (write + scores + mix + values), {B} x {S} tokens, chunks of 2048", ms, pairs * H * (4.0 * D + 2.0 * H))
+        del slabs, proj, out, keep
+    for B, ctx in ((1, 4096), (16, 4096), (64, 4096)):
+        p, nbytes = attention(4096, ctx, 1)
+        slabs = [torch.zeros(nbytes, dtype=torch.uint8, device=device) for _ in range(B)]
+        proj, out = torch.randn(B, ld, device=device, generator=g).to(bf), torch.empty(B, H * D, dtype=bf, device=device)
+        c, keep = mixer_call(proj, ld, out, H * D, [ctx - 1] * B, [1] * B, slabs, True)
+        ms = device_ms(lambda: l.check(l.lib.tm_chunk_attention(h.ptr, C.byref(p), C.byref(c), st), "attention"), stream, K, Wm, flush)
+        add(f"chunk_step_kernel, batch {B}, {ctx} keys", ms, 0.0, B * G * ctx * D * 4.0)
+        del slabs, keep
+
+    # ---- gated linear attention (bytes: projections, outputs, state)
+    HL, dim, vdim, rank = 32, 64, 128, 16
+    n, nv = HL * dim, HL * vdim
+    w2 = torch.randn(n, rank, device=device, generator=g).to(bf)
+    vec, norm = torch.randn(n, device=device, generator=g) + 2, torch.ones(vdim, device=device)
+    p = l.TmGatedLinearParams()
+    p.heads, p.dim, p.vdim, p.rank, p.w2, p.w2_ld, p.bias, p.norm = HL, dim, vdim, rank, w2.data_ptr(), rank, vec.data_ptr(), norm.data_ptr()
+    p.norm_eps, p.scale, p.tau = 1e-6, dim ** -0.5, 16.0
+    p.q_col, p.k_col, p.v_col, p.g_col, p.a_col = 0, n, 2 * n, 2 * n + nv, 2 * n + 2 * nv
+    ld = 2 * n + 2 * nv + rank
+    for B, t, dec in ((1, 4096, False), (4, 1024, False), (8, 2048, False), (1, 1, True), (16, 1, True), (64, 1, True)):
+        proj, out = torch.randn(B * t, ld, device=device, generator=g).to(bf), torch.empty(B * t, nv, dtype=bf, device=device)
+        slabs = [torch.zeros(n * vdim * 4, dtype=torch.uint8, device=device) for _ in range(B)]
+        c, keep = mixer_call(proj, ld, out, nv, [8 if dec else 0] * B, [t] * B, slabs, dec)
+        ms = device_ms(lambda: l.check(l.lib.tm_gated_linear(h.ptr, C.byref(p), C.byref(c), st), "gla"), stream, K, Wm, flush if dec else None)
+        nbytes = B * (t * (ld * 2.0 + nv * 2.0) + n * vdim * 8.0) + n * rank * 2.0
+        add(f"linear_step_kernel, batch {B}" if dec else f"gated linear attention prefill (decay GEMM + gates + scan + finish), {B} x {t} tokens", ms, 0.0, nbytes)
+
+    # ---- mixture of experts (bytes: the chosen experts once, rows in and out)
+    E, ident, top, FF = 30, 2, 4, 2752
+    we, wd = torch.randn(E, 2 * FF, W, device=device, generator=g).to(bf), torch.randn(E, W, FF, device=device, generator=g).to(bf)
+    corr, gb = torch.zeros(E + ident, device=device), torch.zeros(W, device=device)
+    for t in (1, 16, 64, 4096):
+        x, z = torch.zeros(t, W, device=device), torch.randn(t, E + ident, device=device, generator=g)
+        hh, gate, out = (torch.randn(t, W, device=device, generator=g).to(bf) for _ in range(3))
+        m = l.TmMoeParams()
+        m.tokens, m.width, m.ff, m.experts, m.identity, m.top, m.groups, m.keep = t, W, FF, E, ident, top, 4, 2
+        m.limit, m.slope, m.mult, m.norm_eps = 7.0, 1.702, 0.5, 1e-6
+        m.x, m.logits, m.logits_ld, m.input, m.input_ld, m.gate, m.gate_ld = x.data_ptr(), z.data_ptr(), E + ident, hh.data_ptr(), W, gate.data_ptr(), W
+        m.gate_bias, m.correction, m.norm_weight, m.w_experts, m.w_down = gb.data_ptr(), corr.data_ptr(), gb.data_ptr(), we.data_ptr(), wd.data_ptr()
+        m.norm_out, m.dtype = out.data_ptr(), l.TM_DTYPE_BF16
+        ms = device_ms(lambda: l.check(l.lib.tm_moe(h.ptr, C.byref(m), st), "moe"), stream, K, Wm, flush)
+        s = torch.softmax(z, 1).view(t, 4, -1)
+        best = s.max(2).values.topk(2, 1).indices
+        s = torch.where(torch.zeros(t, 4, device=device).scatter(1, best, 1.0)[:, :, None] > 0, s, torch.full_like(s, -1)).view(t, -1)
+        ids = s.topk(top, 1).indices
+        rows, used = int((ids < E).sum()), int(ids[ids < E].unique().numel())
+        add(f"mixture of experts (dispatch + two grouped GEMMs + rows), {t} tokens, {used} experts", ms, 6.0 * rows * FF * W,
+            used * 6.0 * FF * W + t * W * (8.0 + 3 * 2.0))
+    return table.rows
+
+
+def run_fopinex_workload(args, rank, world, device):
+    """Prefill and decode throughput of a random-weight Fopinex model with layers of a 7B-class size (8 layers, bf16) beside the
+    Rumazen model of the same width, depth, heads, recurrent state and feed-forward columns per token, and the kernels of both
+    one at a time.  value = tokens/s of a decode step at batch 64 behind 4096 tokens each."""
+    torch.cuda.set_device(device)
+    K, Wm, L, ctx = min(args.steps, 32), args.warmup, 8, 4096
+    peaks, stream = measured_peaks(), torch.cuda.Stream(device)
+    flush = torch.zeros(64 << 20, dtype=torch.int32, device=device)   # 256 MB, larger than L2
+    sampler, res = ClockSampler(device), {}
+    with torch.cuda.stream(stream):
+        sampler.start()
+        res["fopinex"], headline_ms, e2e, launches = decoder_throughput(fopinex_config(L), device, stream, K, Wm, world, ctx, np.random.default_rng(5 + rank))
+        torch.cuda.empty_cache()
+        res["rumazen"], _, _, _ = decoder_throughput(rumazen_config(L), device, stream, K, Wm, world, ctx, np.random.default_rng(5 + rank))
+        torch.cuda.empty_cache()
+        single = argparse.Namespace(steps=max(5, K // 2), warmup=Wm)
+        kernels = fopinex_kernels(device, stream, single, peaks, flush)
+        torch.cuda.empty_cache()
+        for r in rumazen_kernels(device, stream, single, peaks, flush):
+            if not r.pop("like_kernel_of_llama"):
+                kernels.append(dict(r, like_kernel_of_rumazen=True))
+        clocks = sampler.stop()
+    return {
+        "metric": "decode tokens/s Fopinex, 8 layers of a 7B-class size", "value": round(64 * world / headline_ms * 1e3, 1), "unit": "tokens/s",
+        "n_gpus": world, "steps": K, "warmup": Wm, "ms_per_step": round(headline_ms, 4), "higher_is_better": True, "scaling": "weak",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "fopinex", "model": "8 layers, width 4096, vocab 32000; 2 chunk attention (32 / 8 heads of 128, chunks of 2048, the second "
+                   "on the first's keys), 6 gated linear attention (32 heads of 64 x 128), experts 30 + 2 identity, 4 a token, ff 2752",
+                   "global_batch": 64 * world, "seq_len": ctx,
+                   "l2": "decode: weights and caches of a step larger than L2; single kernels: L2 flushed between launches (decode, experts), inputs "
+                   "larger than L2 (prefill)", "parallelism": "replicas only" if world > 1 else "single GPU"},
+        "throughput": res, "per_kernel": kernels, "clocks": clocks, "gpu_launches": int(launches),
+        "e2e": {"value": round(e2e * world, 1), "unit": "tokens/s", "h2d_bytes_per_step": 64 * 4, "d2h_bytes_per_step": 64 * 4},
+    }
 
 
 def run_rumazen_workload(args, rank, world, device):
     """Prefill and decode throughput of a random-weight Rumazen model with layers of a 7B-class size (8 layers, bf16), beside
     the W4A16 LLaMA of the same width, depth, feed-forward and attention heads, and the kernels of both one at a time.
     value = tokens/s of a decode step at batch 64 behind 4096 tokens each."""
-    from lmdeploy_b200 import decoder, llama
+    from lmdeploy_b200 import llama
     torch.cuda.set_device(device)
     K, Wm, L = min(args.steps, 32), args.warmup, 8
     cfg, peaks = rumazen_config(L), measured_peaks()
@@ -885,50 +1073,11 @@ def run_rumazen_workload(args, rank, world, device):
     flush = torch.zeros(64 << 20, dtype=torch.int32, device=device)   # 256 MB, larger than L2
     rng = np.random.default_rng(5 + rank)
     sampler = ClockSampler(device)
-    res, launches = {"rumazen": {}, "llama_w4a16": {}}, 0
-    ctx = 4096
+    res, ctx = {"rumazen": {}, "llama_w4a16": {}}, 4096
+    prompts = [list(map(int, np.random.default_rng(5 + rank).integers(0, cfg["vocab"], 4096)))]
     with torch.cuda.stream(stream):
         sampler.start()
-        model = decoder.Model.random(cfg, "bfloat16", 64, ctx + 512, 4096, device)
-        slabs = torch.zeros(64, -(-model.slab_bytes // 256) * 256, dtype=torch.uint8, device=device)
-        addr = [slabs[b].data_ptr() for b in range(64)]
-        prompts = [list(map(int, rng.integers(0, cfg["vocab"], 4096))) for _ in range(1)]
-        for B, t in ((1, 1024), (1, 4096), (4, 1024)):
-            ms = device_ms(lambda: model.prefill([prompts[0][:t]] * B, [0] * B, addr[:B]), stream, max(3, K // 4), Wm)
-            res["rumazen"][f"prefill {B} x {t}"] = dict(ms=round(ms, 3), tokens_per_s=round(B * t / ms * 1e3, 1))
-        for B in (1, 16, 64):
-            st = model.new_state(addr[:B], [ctx] * B, 400)
-            model.decode(st, Wm, True, stream.cuda_stream)
-            torch.cuda.synchronize()
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            barrier(world)
-            e0.record(stream)
-            model.decode(st, K, True, stream.cuda_stream)
-            e1.record(stream)
-            torch.cuda.synchronize()
-            ms = max_over_ranks(e0.elapsed_time(e1), world) / K
-            launches += model.last_launches()
-            res["rumazen"][f"decode batch {B} at {ctx}"] = dict(ms=round(ms, 4), tokens_per_s=round(B / ms * 1e3, 1), launches=model.last_launches() // K)
-        headline_ms = ms
-        # end to end: the step's input tokens from pinned host memory, the drawn tokens back, every step
-        st = model.new_state(addr, [ctx] * 64, 400, np.full((400, 64), 0, np.int32))
-        host_in, host_out = torch.randint(0, cfg["vocab"], (64,), dtype=torch.int32).pin_memory(), torch.empty(64, dtype=torch.int32).pin_memory()
-
-        def e2e_step(i):
-            st.forced_ids[i].copy_(host_in, non_blocking=True)
-            model.decode(st, 1, True, stream.cuda_stream)
-            host_out.copy_(st.output_ids[i], non_blocking=True)
-            stream.synchronize()
-
-        for i in range(Wm):
-            e2e_step(i)
-        t0 = time.time()
-        for i in range(Wm, Wm + K):
-            e2e_step(i)
-        e2e = 64 * K / (time.time() - t0)
-        model.check_status()
-        model.close()
-        del slabs, st
+        res["rumazen"], headline_ms, e2e, launches = decoder_throughput(cfg, device, stream, K, Wm, world, ctx, rng)
         lcfg = llama.LlamaConfig(32, 8, 11008, L, quant_policy=0, name="llama 8 layers")
         lm = llama.LlamaModel(lcfg, 64, ctx + 512, device, None)
         lm.random_init(seed=0)
@@ -1423,7 +1572,7 @@ def main():
     ap.add_argument("--steps", type=int, default=128)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--workload", default="decode",
-                    help="decode (7B at 1 GPU, 70B tensor-parallel at N > 1) | decode7b | decode70b | gemm | mmha | prefill | prefill7b | rumazen")
+                    help="decode (7B at 1 GPU, 70B tensor-parallel at N > 1) | decode7b | decode70b | gemm | mmha | prefill | prefill7b | rumazen | fopinex")
     ap.add_argument("--batch-override", type=int, default=0, help="smaller batch for smoke runs")
     ap.add_argument("--max-prompt", type=int, default=0, help="cap on the prompt length for smoke runs")
     ap.add_argument("--no-cpu", action="store_true", help="skip the CPU baseline leg")
@@ -1446,7 +1595,7 @@ def main():
             print(json.dumps({"impl": "reference", "unavailable": "whole-model prefill of the reference needs its engine and "
                               "CUTLASS flash attention; use --workload prefill for its kernels"}), flush=True)
         return
-    if args.impl == "reference" and args.workload == "rumazen":
+    if args.impl == "reference" and args.workload in ("rumazen", "fopinex"):
         if rank == 0:
             print(json.dumps({"impl": "reference", "unavailable": "the reference has no such model"}), flush=True)
         return
@@ -1476,6 +1625,8 @@ def main():
         out = run_prefill_model_workload(args, rank, world, local)
     elif args.workload == "rumazen":
         out = run_rumazen_workload(args, rank, world, local)
+    elif args.workload == "fopinex":
+        out = run_fopinex_workload(args, rank, world, local)
     else:
         raise SystemExit(f"unknown workload {args.workload}")
     if rank == 0:

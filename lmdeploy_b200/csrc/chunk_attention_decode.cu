@@ -7,8 +7,9 @@
 //   S[head, key] = Q K^T    mma.m16n8k16, Q fragments in registers, K rows through ldmatrix; sigmoid; fp16 into shared memory
 //   P[head, key] = talk W   the weights of all heads for the warp's keys, through ldmatrix.trans
 //   O[head, d]  += P V      P straight from the fragments, V rows through ldmatrix.trans
-// Weights are not normalised, so warps and splits simply add up; splits meet in scratch, and the last CTA to arrive sums
-// them in split order (no CTA waits for another).  The new token's key and value are read where the projections left them.
+// Weights are not normalised, so warps and splits simply add up: the splits of a cluster through distributed shared memory,
+// every CTA a slice of the outputs; clusters of a sequence meet in scratch, slice by slice, and the last CTA to arrive sums
+// them in order (no cluster waits for another).  The new token's key and value are read where the projections left them.
 // Before griddepcontrol.wait a CTA only reads its span and rows cached by earlier steps.
 #include "chunk_attention.h"
 #include "common.cuh"
@@ -19,15 +20,15 @@
 namespace tmb {
 namespace {
 
-constexpr int   kKeys = 16, kHeads = 16, kMaxStages = 4, kMaxWarps = 16, kMaxAllHeads = 64, kMaxSplits = 64;
+constexpr int   kKeys = 16, kHeads = 16, kMaxStages = 4, kMaxWarps = 16, kMaxAllHeads = 64, kMaxCluster = 4;
 constexpr float kLog2e = 1.4426950408889634f;
 
 struct StepParams {
     ChunkAttention a;
     MixerCall      c;
-    int            splits, head_blocks, items, kw, stages, hb;
-    float*         scratch;  // [sequence][split][heads][D]
-    int*           tickets;
+    int            splits, cluster, head_blocks, items, kw, stages, hb;  // splits: a multiple of cluster
+    float*         scratch;  // [sequence][cluster][heads][vdim]
+    int*           tickets;  // [sequence][slice]
 };
 
 __device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, int bytes)
@@ -54,6 +55,18 @@ __device__ __forceinline__ float sigmoid_log2(float x)  // sigmoid of x / log2(e
     float e;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-x));
     return __fdividef(1.f, 1.f + e);
+}
+__device__ __forceinline__ float load_cluster(uint32_t addr, uint32_t rank)  // shared memory of another CTA of the cluster
+{
+    float    y;
+    uint32_t there;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(there) : "r"(addr), "r"(rank));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(y) : "r"(there) : "memory");
+    return y;
+}
+__device__ __forceinline__ void cluster_sync()
+{
+    asm volatile("barrier.cluster.arrive.release.aligned;\nbarrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
 __device__ __forceinline__ void wait_pending(int groups)
 {
@@ -213,34 +226,55 @@ __global__ void __launch_bounds__(MAXT) chunk_step_kernel(const StepParams p)
 #pragma unroll
         for (int n = 0; n < D / 8; ++n) *reinterpret_cast<float2*>(rec + 8 * n + c2) = make_float2(o[n][2 * e], o[n][2 * e + 1]);
     }
-    __syncthreads();
-    auto of_warps = [&](int hh, int d) {  // head hh of all
-        const int in = hh % group, it = hh / group * p.head_blocks + in / kHeads;
-        float     y  = 0.f;
-        for (int x = 0; x < p.kw; ++x) y += all[((size_t)(x * p.items + it) * kHeads + in % kHeads) * D + d];
-        return y;
-    };
-    E* const out = static_cast<E*>(p.c.out) + (size_t)sp.tok0 * p.c.out_ld;
-    if (p.splits == 1) {
-        for (int x = tid; x < a.heads * a.vdim; x += threads) out[x] = from_f32<E>(of_warps(x / a.vdim, x % a.vdim));
+    const int  rank = (int)blockIdx.x % p.cluster, n = a.heads * a.vdim, x0 = rank * n / p.cluster, x1 = (rank + 1) * n / p.cluster;
+    E* const   out  = static_cast<E*>(p.c.out) + (size_t)sp.tok0 * p.c.out_ld;
+    const bool whole = p.splits == p.cluster;  // one cluster has all of the sequence
+    if (p.cluster > 1) {
+        cluster_sync();
     }
     else {
-        const size_t n    = (size_t)a.heads * a.vdim;
-        float*       recs = p.scratch + (size_t)blockIdx.y * p.splits * n;
-        for (int x = tid; x < (int)n; x += threads) __stcg(recs + blockIdx.x * n + x, of_warps(x / a.vdim, x % a.vdim));
+        __syncthreads();
+    }
+    float* const recs = p.scratch + (size_t)blockIdx.y * (p.splits / p.cluster) * n;
+    for (int x = x0 + tid; x < x1; x += threads) {
+        const int h = x / a.vdim, in = h % group, it = h / group * p.head_blocks + in / kHeads;
+        float     y = 0.f;
+        if (p.cluster > 1) {
+            float v[kMaxCluster];
+            for (int k = 0; k < p.kw; ++k) {
+                const uint32_t at = smem_u32(all + ((size_t)(k * p.items + it) * kHeads + in % kHeads) * D + x % a.vdim);
+#pragma unroll
+                for (int c = 0; c < kMaxCluster; ++c) v[c] = c < p.cluster ? load_cluster(at, c) : 0.f;
+#pragma unroll
+                for (int c = 0; c < kMaxCluster; ++c) y += v[c];
+            }
+        }
+        else {
+            for (int k = 0; k < p.kw; ++k) y += all[((size_t)(k * p.items + it) * kHeads + in % kHeads) * D + x % a.vdim];
+        }
+        if (whole) {
+            out[x] = from_f32<E>(y);
+        }
+        else {
+            __stcg(recs + (blockIdx.x / p.cluster) * n + x, y);
+        }
+    }
+    if (!whole) {
+        const int clusters = p.splits / p.cluster;
         __threadfence();
         __syncthreads();
         if (tid == 0) {
-            s_last = atomicAdd(p.tickets + blockIdx.y, 1) == p.splits - 1;
-            if (s_last) p.tickets[blockIdx.y] = 0;
+            int* ticket = p.tickets + blockIdx.y * p.cluster + rank;
+            s_last      = atomicAdd(ticket, 1) == clusters - 1;
+            if (s_last) *ticket = 0;
         }
         __syncthreads();
         if (s_last) {
             __threadfence();
-            for (int x = tid; x < (int)n; x += threads) {
+            for (int x = x0 + tid; x < x1; x += threads) {
                 float y = 0.f;
 #pragma unroll 8
-                for (int k = 0; k < p.splits; ++k) y += __ldcg(recs + k * n + x);
+                for (int k = 0; k < clusters; ++k) y += __ldcg(recs + (size_t)k * n + x);
                 out[x] = from_f32<E>(y);
             }
         }
@@ -255,6 +289,7 @@ __global__ void __launch_bounds__(MAXT) chunk_step_kernel(const StepParams p)
         }
         for (int d = a.heads * a.vdim + tid; d < p.c.out_pad; d += threads) out[d] = from_f32<E>(0.f);
     }
+    if (p.cluster > 1) cluster_sync();  // the others have read this CTA's results
 }
 
 struct StepPlan {
@@ -280,7 +315,17 @@ StepPlan plan_of(const tm_handle* h, const ChunkAttention& a)
 template<int D, int MAXT>
 cudaError_t launch(const StepParams& p, int batch, size_t smem, cudaStream_t st)
 {
-    return launch_kernel(chunk_step_kernel<D, MAXT>, dim3(p.splits, batch), dim3(p.items * p.kw * 32), smem, st, p.c.pdl, p);
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = dim3(p.splits, batch), cfg.blockDim = dim3(p.items * p.kw * 32), cfg.dynamicSmemBytes = smem, cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id                                         = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x                           = p.cluster;
+    attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+    attr[1].id                                         = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs                                          = attr;
+    cfg.numAttrs                                       = p.c.pdl ? 2 : 1;
+    return cudaLaunchKernelEx(&cfg, chunk_step_kernel<D, MAXT>, p);
 }
 
 cudaError_t prepare(int max_smem)
@@ -305,14 +350,15 @@ bool chunk_attention_step_supported(const tm_handle* h, const ChunkAttention& a,
 int chunk_attention_step(tm_handle* h, const ChunkAttention& a, const MixerCall& c, cudaStream_t st)
 {
     const StepPlan  pl = plan_of(h, a);
-    StepParams      p{a, c, 1, pl.head_blocks, pl.items, pl.kw, pl.stages, pl.hb, static_cast<float*>(h->attn_scratch), h->attn_counters};
-    // the bound on the visible keys is the host's; a split takes at least two tiles
+    StepParams      p{a, c, 1, 1, pl.head_blocks, pl.items, pl.kw, pl.stages, pl.hb, static_cast<float*>(h->attn_scratch), h->attn_counters};
+    // one wave of CTAs, a split with at least two tiles; the bound on the visible keys is the host's
     const long long keys = a.chunk > 0 ? std::min(a.chunk, c.max_context) : c.max_context, resident = std::max<long long>(1, h->max_smem / (long long)pl.smem);
-    long long       splits = std::min<long long>((resident * h->sm_count + c.batch - 1) / c.batch, std::max<long long>(1, keys / (2 * kKeys * pl.kw)));
-    splits = std::min<long long>(splits, kMaxSplits);
-    splits = std::min<long long>(splits, (long long)(h->attn_scratch_bytes / ((size_t)c.batch * a.heads * a.vdim * 4)));
-    if (c.batch >= h->sm_count || c.batch > (int)h->attn_counter_ints) splits = 1;
-    p.splits = (int)std::max<long long>(1, splits);
+    const long long splits = std::min(std::min(resident, 2ll) * h->sm_count / c.batch, keys / (2 * kKeys * pl.kw));
+    while (p.cluster < kMaxCluster && 2 * p.cluster <= splits) p.cluster *= 2;
+    long long clusters = std::max<long long>(1, splits / p.cluster);
+    clusters = std::min<long long>(clusters, (long long)(h->attn_scratch_bytes / ((size_t)c.batch * a.heads * a.vdim * 4)));
+    if (clusters < 1 || (long long)c.batch * p.cluster > (long long)h->attn_counter_ints) clusters = 1;
+    p.splits = (int)clusters * p.cluster;
     const bool        wide = pl.items * pl.kw > 8;
     const cudaError_t e = pl.D == 64 ? (wide ? launch<64, 512>(p, c.batch, pl.smem, st) : launch<64, 256>(p, c.batch, pl.smem, st)) :
                                        (wide ? launch<128, 512>(p, c.batch, pl.smem, st) : launch<128, 256>(p, c.batch, pl.smem, st));

@@ -70,22 +70,81 @@ __global__ void __launch_bounds__(128) linear_gates_kernel(const LinearParams p)
     for (int c = lane; c < p.record - 3 * DP; c += 32) rec[3 * DP + c] = c < d.vdim ? to_f32(row[d.v_col + h * d.vdim + c]) : 0.f;
 }
 
-// The sequential part.  CTA = (block of value columns, head, sequence).  Lanes of a group share four columns; lane `part`
+// The same where head sizes are multiples of four: a CTA per token, a thread takes four channels at a time
+template<typename E>
+__device__ __forceinline__ float4 load4(const E* p)
+{
+    if constexpr (sizeof(E) == 2) {
+        const uint2 w = *reinterpret_cast<const uint2*>(p);
+        return make_float4(bf16_lo(w.x), bf16_hi(w.x), bf16_lo(w.y), bf16_hi(w.y));
+    }
+    else {
+        return *reinterpret_cast<const float4*>(p);
+    }
+}
+template<typename E, int DP>
+__global__ void __launch_bounds__(256) linear_gates4_kernel(const LinearParams p)
+{
+    pdl_wait();
+    pdl_launch_dependents();
+    const GatedLinear& d = p.d;
+    const SeqSpan      s = p.c.spans[blockIdx.y];
+    if (!s.live || (int)blockIdx.x >= s.n) return;
+    const size_t tok = (size_t)s.tok0 + blockIdx.x;
+    const E*     row = static_cast<const E*>(p.c.proj) + tok * p.c.proj_ld;
+    const float* pre = p.decay_pre + tok * d.heads * d.dim;
+    const int    per = p.record / 4;
+    const float  inv_tau = 1.f / d.tau;
+    for (int x = threadIdx.x; x < d.heads * per; x += 256) {
+        const int h = x / per, i = 4 * (x - h * per), part = i < 3 * DP ? i / DP : 3, c = i - part * DP, at = h * d.dim + c;
+        float4    y = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (part == 3) {
+            y = load4(row + d.v_col + h * d.vdim + c);
+        }
+        else if (c < d.dim) {
+            if (part == 1) {
+                const float4 z = *reinterpret_cast<const float4*>(pre + at), b = *reinterpret_cast<const float4*>(d.bias + at);
+                y = make_float4(decay_of(z.x + b.x, inv_tau), decay_of(z.y + b.y, inv_tau), decay_of(z.z + b.z, inv_tau), decay_of(z.w + b.w, inv_tau));
+            }
+            else {
+                y = load4(row + (part == 0 ? d.q_col : d.k_col) + at);
+                if (part == 0) y.x *= d.scale, y.y *= d.scale, y.z *= d.scale, y.w *= d.scale;
+            }
+        }
+        *reinterpret_cast<float4*>(p.records + ((size_t)h * p.c.tokens + tok) * p.record + i) = y;
+    }
+}
+
+// The sequential part.  CTA = (block of value columns, head, sequence).  Lanes of a group share NC columns; lane `part`
 // holds rows [4 part, 4 part + 4) and [DP/2 + 4 part, ...) of each, in pairs.  Records of a head are contiguous, so one bulk
-// copy brings a chunk of tokens into a stage.  Tokens go in pairs: eight sums are exchanged together, while the next pair
-// is under way.
-template<int DP>
+// copy brings a chunk of tokens into a stage.  Tokens go in pairs: their sums are exchanged together, while the next pair is
+// under way and the operands of the one behind it are on their way from shared memory.
+// NC: columns of a lane group; four use the shared memory best, two spread a short batch over more SMs.
+template<int DP, int NC>
 struct LinearShape {
-    static constexpr int kThreads = 128, kLanes = DP / 8, kPerLane = 4;
-    static constexpr int kColumns = kThreads / kLanes * kPerLane;
+    static constexpr int kThreads = 128, kLanes = DP / 8;
+    static constexpr int kColumns = kThreads / kLanes * NC;
     static constexpr int kStages  = 3;
-    static constexpr int kBits    = kLanes >= 8 ? 3 : (kLanes == 4 ? 2 : 1);  // exchanges that halve the number of sums
+    static constexpr int kBits    = kLanes == 2 ? 1 : (kLanes == 4 || NC == 2 ? 2 : 3);  // exchanges that halve the number of sums
 };
 
-template<int DP>
-__global__ void __launch_bounds__(LinearShape<DP>::kThreads) linear_scan_kernel(const LinearParams p)
+// A store that the compiler need not order against loads from shared memory, as it has to with an ordinary pointer
+// (and no branch around it)
+__device__ __forceinline__ void store_global_if(bool on, float* p, float v)
 {
-    using S = LinearShape<DP>;
+    asm volatile(
+        "{\n"
+        ".reg .pred p;\n"
+        "setp.ne.b32 p, %2, 0;\n"
+        "@p st.global.f32 [%0], %1;\n"
+        "}\n" ::"l"(__cvta_generic_to_global(p)),
+        "f"(v), "r"((int)on));
+}
+
+template<int DP, int NC>
+__global__ void __launch_bounds__(128) linear_scan_kernel(const LinearParams p)
+{
+    using S = LinearShape<DP, NC>;
     extern __shared__ __align__(128) float sm[];
     __shared__ uint64_t full[S::kStages];
     const int tid = threadIdx.x;
@@ -114,7 +173,7 @@ __global__ void __launch_bounds__(LinearShape<DP>::kThreads) linear_scan_kernel(
     if (tid == 0) {
         for (int ch = 0; ch < min(S::kStages, chunks); ++ch) fetch(ch);
     }
-    constexpr int NC = S::kPerLane, NV = 2 * NC, kKeep = NV >> S::kBits;
+    constexpr int NV = 2 * NC, kKeep = NV >> S::kBits;
     const int     part = tid % S::kLanes, col0 = c0 + tid / S::kLanes * NC;
     float*        state = reinterpret_cast<float*>(s.slab + d.state_off) + (size_t)h * dim * vdim;
     auto          row_of = [&](int i) { return (i >> 1) * (DP / 2) + 4 * part + 2 * (i & 1); };  // first row of pair i
@@ -129,7 +188,7 @@ __global__ void __launch_bounds__(LinearShape<DP>::kThreads) linear_scan_kernel(
             st[c][i]        = pair_of(on && r < dim ? at[0] : 0.f, on && r + 1 < dim ? at[1] : 0.f);
         }
     }
-    // sums over the lanes of the group: a lane ends up with numbers [first, first + kKeep) of the eight (token, column)
+    // sums over the lanes of the group: a lane ends up with numbers [first, first + kKeep) of the pair's (token, column)
     int first = 0;
 #pragma unroll
     for (int level = 0; level < S::kBits; ++level) first += ((part >> level) & 1) * (NV >> (level + 1));
@@ -156,57 +215,75 @@ __global__ void __launch_bounds__(LinearShape<DP>::kThreads) linear_scan_kernel(
     bool   held_two = false, ok = true;
     auto store_outputs = [&]() {
         scatter_sums(sums);
-        if (held < 0 || part >= (1 << S::kBits)) return;
+        const bool mine = held >= 0 && part < (1 << S::kBits);
 #pragma unroll
         for (int i = 0; i < kKeep; ++i) {
             const int b = (first + i) / NC, c = (first + i) % NC;
-            if ((b == 0 || held_two) && col0 + c < vdim) o_out[(size_t)(held + b) * d.heads * vdim + c] = sums[i];
+            store_global_if(mine && (b == 0 || held_two) && col0 + c < vdim, o_out + (size_t)(max(held, 0) + b) * d.heads * vdim + c, sums[i]);
         }
     };
-    const int v_at = 3 * DP + (col0 < vdim ? col0 : 0);  // four columns; groups beyond the last write nothing
+    const int v_at = 3 * DP + (col0 < vdim ? col0 : 0);  // groups beyond the last column write nothing
+    struct Pair {
+        f32x2 q[2][4], a[2][4], k[2][4];
+        float v[2][NC];
+    };
     int ch = 0;
     for (; ch < chunks; ++ch) {
         ok           = mbar_wait(&full[ch % S::kStages], (ch / S::kStages) & 1, p.max_wait);
         const int nt = min(CH, s.n - ch * CH);
-#pragma unroll 2
-        for (int t = 0; t < nt; t += 2) {
-            const bool   two  = t + 1 < nt;
-            const float* rec  = sm + (size_t)((ch % S::kStages) * CH + t) * p.record;
-            const float* rec1 = two ? rec + p.record : rec;
-            auto vec = [&](const float* r, int which, f32x2 (&x)[4]) {
-#pragma unroll
-                for (int q = 0; q < 2; ++q) {
-                    const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(r + which * DP + q * (DP / 2) + 4 * part);
-                    x[2 * q] = w.x, x[2 * q + 1] = w.y;
-                }
-            };
-            f32x2  q[2][4], a[2][4], k[2][4];
-            float4 v[2];
-            vec(rec, 0, q[0]), vec(rec, 1, a[0]), vec(rec, 2, k[0]);
-            vec(rec1, 0, q[1]), vec(rec1, 1, a[1]), vec(rec1, 2, k[1]);
-            v[0] = *reinterpret_cast<const float4*>(rec + v_at), v[1] = *reinterpret_cast<const float4*>(rec1 + v_at);
-            store_outputs();
+        const float* const stage = sm + (size_t)(ch % S::kStages) * CH * p.record;
+        auto load = [&](int t, Pair& x) {
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
-                const float vv[4] = {v[j].x, v[j].y, v[j].z, v[j].w};
-                if (j == 0 || two) {
+                const float* rec = stage + (size_t)min(t + j, nt - 1) * p.record;
+                auto vec = [&](int which, f32x2 (&y)[4]) {
 #pragma unroll
-                    for (int c = 0; c < NC; ++c) {
-                        const f32x2 x = pair_of(vv[c], vv[c]);
-#pragma unroll
-                        for (int i = 0; i < 4; ++i) st[c][i] = fma2(a[j][i], st[c][i], mul2(k[j][i], x));
+                    for (int q = 0; q < 2; ++q) {
+                        const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(rec + which * DP + q * (DP / 2) + 4 * part);
+                        y[2 * q] = w.x, y[2 * q + 1] = w.y;
                     }
+                };
+                vec(0, x.q[j]), vec(1, x.a[j]), vec(2, x.k[j]);
+                if constexpr (NC == 4) {
+                    const float4 w = *reinterpret_cast<const float4*>(rec + v_at);
+                    x.v[j][0] = w.x, x.v[j][1] = w.y, x.v[j][2] = w.z, x.v[j][3] = w.w;
                 }
-#pragma unroll
-                for (int c = 0; c < NC; ++c) {
-                    f32x2 y = mul2(q[j][0], st[c][0]);
-#pragma unroll
-                    for (int i = 1; i < 4; ++i) y = fma2(q[j][i], st[c][i], y);
-                    const float2 f   = halves(y);
-                    sums[j * NC + c] = f.x + f.y;
+                else {
+                    const float2 w = *reinterpret_cast<const float2*>(rec + v_at);
+                    x.v[j][0] = w.x, x.v[j][1] = w.y;
                 }
             }
-            held = ch * CH + t, held_two = two;
+        };
+        auto token = [&](const Pair& x, int j) {
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                const f32x2 v = pair_of(x.v[j][c], x.v[j][c]);
+                f32x2       y[4];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) st[c][i] = fma2(x.a[j][i], st[c][i], mul2(x.k[j][i], v));
+#pragma unroll
+                for (int i = 0; i < 4; i += 2) y[i] = fma2(x.q[j][i + 1], st[c][i + 1], mul2(x.q[j][i], st[c][i]));
+                const float2 f = halves(y[0]), g = halves(y[2]);
+                sums[j * NC + c] = (f.x + f.y) + (g.x + g.y);
+            }
+        };
+        Pair now;
+        load(0, now);
+        int t = 0;
+#pragma unroll 2
+        for (; t + 1 < nt; t += 2) {
+            Pair next;
+            load(min(t + 2, nt - 1), next);
+            store_outputs();
+            token(now, 0);
+            token(now, 1);
+            held = ch * CH + t, held_two = true;
+            now  = next;
+        }
+        if (t < nt) {  // an odd last token
+            store_outputs();
+            token(now, 0);
+            held = ch * CH + t, held_two = false;
         }
         // everybody is through with the stage; one outcome for the whole CTA
         if (!__syncthreads_and(ok)) break;
@@ -410,16 +487,26 @@ __global__ void __launch_bounds__(256, 2) linear_step_kernel(const LinearParams 
     }
 }
 
-template<typename E, int DP>
-cudaError_t scan_launch(LinearParams p, cudaStream_t st)
+template<int DP, int NC>
+cudaError_t scan_kernel_launch(const LinearParams& p, cudaStream_t st)
 {
-    using S = LinearShape<DP>;
-    cudaError_t e = launch_kernel(linear_gates_kernel<E, DP>, dim3(p.c.max_n, (p.d.heads + 3) / 4, p.c.batch), dim3(128), 0, st, p.c.pdl, p);
-    if (e != cudaSuccess) return e;
-    p.chunk = std::max(2, std::min(16, 16384 / (p.record * 4) / 2 * 2));
+    using S           = LinearShape<DP, NC>;
     const size_t smem = (size_t)S::kStages * p.chunk * p.record * 4;
     const dim3   grid((p.d.vdim + S::kColumns - 1) / S::kColumns, p.d.heads, p.c.batch);
-    return launch_kernel(linear_scan_kernel<DP>, grid, dim3(S::kThreads), smem, st, p.c.pdl, p);
+    return launch_kernel(linear_scan_kernel<DP, NC>, grid, dim3(S::kThreads), smem, st, p.c.pdl, p);
+}
+
+template<typename E, int DP>
+cudaError_t scan_launch(LinearParams p, int sms, cudaStream_t st)
+{
+    const GatedLinear& d    = p.d;
+    const bool         quad = d.dim % 4 == 0 && d.vdim % 4 == 0 && p.c.proj_ld % 4 == 0 && d.q_col % 4 == 0 && d.k_col % 4 == 0 && d.v_col % 4 == 0;
+    cudaError_t        e = quad ? launch_kernel(linear_gates4_kernel<E, DP>, dim3(p.c.max_n, p.c.batch), dim3(256), 0, st, p.c.pdl, p) :
+                                  launch_kernel(linear_gates_kernel<E, DP>, dim3(p.c.max_n, (d.heads + 3) / 4, p.c.batch), dim3(128), 0, st, p.c.pdl, p);
+    if (e != cudaSuccess) return e;
+    p.chunk = std::max(2, std::min(16, 16384 / (p.record * 4) / 2 * 2));
+    const long long ctas = (long long)((p.d.vdim + LinearShape<DP, 4>::kColumns - 1) / LinearShape<DP, 4>::kColumns) * p.d.heads * p.c.batch;
+    return ctas < sms ? scan_kernel_launch<DP, 2>(p, st) : scan_kernel_launch<DP, 4>(p, st);
 }
 
 template<typename E, int DP>
@@ -430,14 +517,14 @@ cudaError_t step_launch(const LinearParams& p, cudaStream_t st)
 }
 
 template<typename E>
-cudaError_t dispatch(const LinearParams& p, bool step, cudaStream_t st)
+cudaError_t dispatch(const LinearParams& p, bool step, int sms, cudaStream_t st)
 {
     switch (padded_dim(p.d.dim)) {
-        case 16: return step ? step_launch<E, 16>(p, st) : scan_launch<E, 16>(p, st);
-        case 32: return step ? step_launch<E, 32>(p, st) : scan_launch<E, 32>(p, st);
-        case 64: return step ? step_launch<E, 64>(p, st) : scan_launch<E, 64>(p, st);
-        case 128: return step ? step_launch<E, 128>(p, st) : scan_launch<E, 128>(p, st);
-        default: return step ? step_launch<E, 256>(p, st) : scan_launch<E, 256>(p, st);
+        case 16: return step ? step_launch<E, 16>(p, st) : scan_launch<E, 16>(p, sms, st);
+        case 32: return step ? step_launch<E, 32>(p, st) : scan_launch<E, 32>(p, sms, st);
+        case 64: return step ? step_launch<E, 64>(p, st) : scan_launch<E, 64>(p, sms, st);
+        case 128: return step ? step_launch<E, 128>(p, st) : scan_launch<E, 128>(p, sms, st);
+        default: return step ? step_launch<E, 256>(p, st) : scan_launch<E, 256>(p, sms, st);
     }
 }
 
@@ -450,11 +537,13 @@ bool valid(const GatedLinear& d, const MixerCall& c)
 cudaError_t prepare(int)
 {
     constexpr int smem = 3 * 16384;  // at most: a chunk of several tokens fits 16 KB, and two tokens take no more
-    cudaError_t   e    = cudaFuncSetAttribute(linear_scan_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_scan_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_scan_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_scan_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(linear_scan_kernel<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t   e    = cudaSuccess;
+    for (const void* f : {(const void*)linear_scan_kernel<16, 2>, (const void*)linear_scan_kernel<32, 2>, (const void*)linear_scan_kernel<64, 2>,
+                          (const void*)linear_scan_kernel<128, 2>, (const void*)linear_scan_kernel<256, 2>, (const void*)linear_scan_kernel<16, 4>,
+                          (const void*)linear_scan_kernel<32, 4>, (const void*)linear_scan_kernel<64, 4>, (const void*)linear_scan_kernel<128, 4>,
+                          (const void*)linear_scan_kernel<256, 4>}) {
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    }
     return e;
 }
 const KernelPreparation g_prepare(prepare);
@@ -480,7 +569,7 @@ int gated_linear_prefill(tm_handle* h, const GatedLinear& d, const MixerCall& c,
     float* const       o       = scratch + (size_t)c.tokens * ((d.heads * d.dim + 3) / 4 * 4);
     float* const       records = o + (size_t)c.tokens * ((d.heads * d.vdim + 3) / 4 * 4);
     const LinearParams p{d, c, scratch, records, o, record_floats(d), 0, h->status, kMaxWaitCycles};
-    cudaError_t        e = c.f32 ? dispatch<float>(p, false, st) : dispatch<__nv_bfloat16>(p, false, st);
+    cudaError_t        e = c.f32 ? dispatch<float>(p, false, h->sm_count, st) : dispatch<__nv_bfloat16>(p, false, h->sm_count, st);
     const dim3         grid(c.tokens, (d.heads + 7) / 8);
     if (e == cudaSuccess) e = launch_kernel(c.f32 ? linear_finish_kernel<float> : linear_finish_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, c.pdl, p);
     if (e != cudaSuccess) {
@@ -495,7 +584,7 @@ int gated_linear_decode(tm_handle* h, const GatedLinear& d, const MixerCall& c, 
 {
     if (!valid(d, c)) return TM_ERR_UNSUPPORTED;
     const LinearParams p{d, c, nullptr, nullptr, nullptr, 0, 0, h->status, kMaxWaitCycles};
-    const cudaError_t  e = c.f32 ? dispatch<float>(p, true, st) : dispatch<__nv_bfloat16>(p, true, st);
+    const cudaError_t  e = c.f32 ? dispatch<float>(p, true, h->sm_count, st) : dispatch<__nv_bfloat16>(p, true, h->sm_count, st);
     if (e != cudaSuccess) {
         h->last_cuda_error = (int)e;
         return TM_ERR_CUDA;

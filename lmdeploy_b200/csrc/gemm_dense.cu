@@ -53,7 +53,7 @@ struct DenseTcParams {
     int           cut_ctas;    // > 0: CTAs that share the k blocks of all tiles evenly
     int           stages, tmem_columns;
     int           x2_tile;     // weight tiles from here on multiply the second operand
-    int           column_tiles;
+    int           column_tiles, half_box;
     DenseGroups   groups;
     float*        scratch;
     int*          tickets;
@@ -62,33 +62,44 @@ struct DenseTcParams {
     DenseEpilogue ep;
 };
 
-// What happens to 16 consecutive tokens of one output column (lane = column); `live` = tokens of the 16 that exist
-__device__ __forceinline__ void epilogue16(const DenseEpilogue& ep, const float (&y)[16], int t0, int live, int n, int n_out, float (&sq)[16])
+// kResidual: what 16 consecutive tokens of one output column add to and are gated by, as it lies in memory, requested ahead
+struct ResidualIn {
+    float         r[16];
+    __nv_bfloat16 gate[16];
+};
+__device__ __forceinline__ void residual_load(const DenseEpilogue& ep, int t0, int live, int n, int n_out, ResidualIn& in)
+{
+    const bool col = n < n_out;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) in.r[i] = i < live && col ? ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] : 0.f;
+    if (ep.gate) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            in.gate[i] = i < live && col ? static_cast<const __nv_bfloat16*>(ep.gate)[(size_t)(t0 + i) * ep.gate_ld + n] : __nv_bfloat16();
+        }
+    }
+}
+__device__ __forceinline__ void residual_add(const DenseEpilogue& ep, const float (&y)[16], const ResidualIn& in, float bias, int t0, int live, int n, int n_out,
+                                             float (&sq)[16])
 {
     using E        = __nv_bfloat16;
     const bool col = n < n_out;
-    if (ep.kind == DenseKind::kResidual) {
-        float r[16];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) r[i] = i < live && col ? ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] : 0.f;
-        float f[16];
-        if (ep.gate) {
-            const float b = col ? ep.gate_bias[n] : 0.f;
-#pragma unroll
-            for (int i = 0; i < 16; ++i) f[i] = i < live && col ? to_f32(static_cast<const E*>(ep.gate)[(size_t)(t0 + i) * ep.gate_ld + n]) + b : 0.f;
-#pragma unroll
-            for (int i = 0; i < 16; ++i) f[i] = __fdividef(ep.mult, 1.f + __expf(-f[i]));
-        }
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-            const bool on = i < live && col;
-            r[i]          = on ? r[i] + (ep.gate ? f[i] * y[i] : y[i]) : 0.f;
-            sq[i]         = r[i] * r[i];
-            if (on) ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] = r[i];
-            if (on && ep.cast) static_cast<E*>(ep.cast)[(size_t)(t0 + i) * ep.cast_ld + n] = from_f32<E>(r[i]);
-        }
-        return;
+    for (int i = 0; i < 16; ++i) {
+        const bool  on = i < live && col;
+        const float f  = ep.gate ? __fdividef(ep.mult, 1.f + __expf(-(to_f32(in.gate[i]) + bias))) : 1.f;
+        const float r  = on ? in.r[i] + f * y[i] : 0.f;
+        sq[i]          = r * r;
+        if (on) ep.residual[(size_t)(t0 + i) * ep.residual_ld + n] = r;
+        if (on && ep.cast) static_cast<E*>(ep.cast)[(size_t)(t0 + i) * ep.cast_ld + n] = from_f32<E>(r);
     }
+}
+
+// What happens to 16 consecutive tokens of one output column (lane = column); `live` = tokens of the 16 that exist
+__device__ __forceinline__ void epilogue16(const DenseEpilogue& ep, const float (&y)[16], int t0, int live, int n, int n_out)
+{
+    using E        = __nv_bfloat16;
+    const bool col = n < n_out;
     if (ep.kind == DenseKind::kF32) {
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
@@ -181,7 +192,7 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
     const int cut_ctas = GROUPS && p.cut_ctas > 0 ? max(1, min(p.cut_ctas, (int)min((long long)tiles * p.k_blocks / 4, 1ll << 20))) : p.cut_ctas;
     // tile -> weight tile, first row of its tokens, how many there are, first weight row, token tile (the key of `scale`)
     struct Place {
-        int ct, t0, rows, w_row, tt;
+        int ct, t0, rows, w_row, tt, height;  // height: token columns of the tile's products
     };
     auto place = [&](int tile) {
         Place q;
@@ -193,11 +204,12 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
             }
             const int begin = p.groups.offsets[lo], n = p.groups.offsets[lo + 1] - begin, tts = (n + NT - 1) / NT, in = tile - first_tile[lo];
             q.ct = in / tts, q.tt = in - q.ct * tts;
-            q.t0 = begin + q.tt * NT, q.rows = min(NT, n - q.tt * NT), q.w_row = lo * p.n_out + q.ct * kDenseTile;
+            q.height = ((n + tts - 1) / tts + 15) / 16 * 16;  // the group's tiles are equally high
+            q.t0 = begin + q.tt * q.height, q.rows = min(q.height, n - q.tt * q.height), q.w_row = lo * p.n_out + q.ct * kDenseTile;
         }
         else {
             q.ct = tile / p.token_tiles, q.tt = tile - q.ct * p.token_tiles;
-            q.t0 = q.tt * NT, q.rows = min(NT, p.tokens - q.t0), q.w_row = q.ct * kDenseTile;
+            q.t0 = q.tt * NT, q.rows = min(NT, p.tokens - q.t0), q.w_row = q.ct * kDenseTile, q.height = NT;
         }
         return q;
     };
@@ -223,12 +235,14 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
         if (lane == 0) {
             int  issued = 0;
             bool ok = true, waited = false;
+            // groups: a low tile's rows come in a box of half the height (one copy either way: their issue rate counts)
+            auto low    = [&](const Place& q) { return GROUPS && q.height <= p.half_box; };
             auto load_w = [&](int kb, const Place& q, int s) {
-                mbar_arrive_expect_tx(&sh->full[s], stage_b);
+                mbar_arrive_expect_tx(&sh->full[s], low(q) ? w_bytes + (uint32_t)p.half_box * 128 : stage_b);
                 tma_load_2d(base + s * stage_b, &w_map, kb * kKBlock, q.w_row, &sh->full[s]);
             };
             auto load_x = [&](int kb, const Place& q, int s) {
-                tma_load_2d(base + s * stage_b + w_bytes, q.ct >= p.x2_tile ? &x2_map : &x_map, kb * kKBlock, q.t0, &sh->full[s]);
+                tma_load_2d(base + s * stage_b + w_bytes, low(q) || q.ct >= p.x2_tile ? &x2_map : &x_map, kb * kKBlock, q.t0, &sh->full[s]);
             };
             int tile, kb0, kb1;
             for (int seg = 0; ok && segment(seg, tile, kb0, kb1); ++seg) {
@@ -276,12 +290,13 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
         pdl_wait();
         pdl_launch_dependents();
         if (lane == 0) {
-            const uint32_t idesc = umma_idesc_bf16(kDenseTile, NT);
+            uint32_t       idesc = umma_idesc_bf16(kDenseTile, NT);
             int            it = 0, local = 0;
             bool           ok = true;
             int            tile, kb0, kb1;
             for (; ok && segment(local, tile, kb0, kb1); ++local) {
                 const int a = local & 1;
+                if (GROUPS) idesc = umma_idesc_bf16(kDenseTile, place(tile).height);
                 if (local >= 2 && !mbar_wait(&sh->acc_empty[a], ((local >> 1) - 1) & 1, p.max_wait)) ok = false;
                 tcgen05_after_sync();
                 for (int kb = kb0; kb < kb1 && ok; ++kb, ++it) {
@@ -331,6 +346,10 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                 named_bar_sync(kEpiBar, 128);
                 scaled_tile = tt;
             }
+            const bool  adds = p.ep.kind == DenseKind::kResidual;
+            const float bias = adds && p.ep.gate && n < p.n_out ? p.ep.gate_bias[n] : 0.f;
+            ResidualIn  in;
+            if (adds && kb1 - kb0 == p.k_blocks) residual_load(p.ep, t0, min(16, rows), n, p.n_out, in);
             int okw = 1;
             if (lane == 0) okw = mbar_wait(&sh->acc_full[a], (local >> 1) & 1, p.max_wait) ? 1 : 0;
             okw = __shfl_sync(0xffffffffu, okw, 0);
@@ -384,7 +403,8 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
                 if (finish) __threadfence();
             }
             if (finish) {
-                const bool sums = p.ep.kind == DenseKind::kResidual && p.ep.ssq_out;
+                const bool sums = adds && p.ep.ssq_out;
+                if (adds && kb1 - kb0 < p.k_blocks) residual_load(p.ep, t0, min(16, rows), n, p.n_out, in);
                 for (int c0 = 0; c0 < rows; c0 += 16) {
                     float     v[16], sq[16];
                     const int live = min(16, rows - c0);
@@ -415,7 +435,15 @@ dense_tc_kernel(const DenseTcParams p, const __grid_constant__ CUtensorMap w_map
 #pragma unroll
                         for (int i = 0; i < 16; ++i) v[i] *= i < live ? sh->scale[c0 + i] : 0.f;
                     }
-                    epilogue16(p.ep, v, t0 + c0, live, n, p.n_out, sq);
+                    if (adds) {
+                        ResidualIn next;
+                        if (c0 + 16 < rows) residual_load(p.ep, t0 + c0 + 16, min(16, rows - c0 - 16), n, p.n_out, next);
+                        residual_add(p.ep, v, in, bias, t0 + c0, live, n, p.n_out, sq);
+                        in = next;
+                    }
+                    else {
+                        epilogue16(p.ep, v, t0 + c0, live, n, p.n_out);
+                    }
                     if (sums) {
 #pragma unroll
                         for (int i = 0; i < 16; ++i) {
@@ -598,6 +626,7 @@ int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
     p.groups           = g.groups;
     p.x2_tile          = g.x2 ? g.x2_from / kDenseTile : 1 << 30;
     p.column_tiles     = (g.n_out + kDenseTile - 1) / kDenseTile;
+    p.half_box         = plan.token_tile / 2 / 16 * 16;
     p.token_tile    = plan.token_tile;
     p.token_tiles   = (g.tokens + p.token_tile - 1) / p.token_tile;
     p.tiles         = (g.n_out + kDenseTile - 1) / kDenseTile * p.token_tiles;
@@ -625,7 +654,8 @@ int dense_tc(tm_handle* h, const DenseGemm& g, cudaStream_t st, bool pdl)
     CUtensorMap w_map, x_map, x2_map;
     if (!encode_rows(encode, &w_map, g.w, g.n_out * std::max(1, g.groups.count), g.k, g.ldw, kDenseTile)) return TM_ERR_CUDA;
     if (!encode_rows(encode, &x_map, g.x, g.tokens, g.k, g.ldx, p.token_tile)) return TM_ERR_CUDA;
-    if (!encode_rows(encode, &x2_map, g.x2 ? g.x2 : g.x, g.tokens, g.k, g.ldx, p.token_tile)) return TM_ERR_CUDA;
+    // the second operand, or the half-height boxes of the groups
+    if (!encode_rows(encode, &x2_map, g.x2 ? g.x2 : g.x, g.tokens, g.k, g.ldx, grouped ? std::max(16, p.half_box) : p.token_tile)) return TM_ERR_CUDA;
     const size_t smem = 1024 + (size_t)p.stages * stage_b + shared;
     const dim3   grid(grid_ctas);
     const cudaError_t e = grouped ? launch_kernel(dense_tc_kernel<true>, grid, dim3(kThreads), smem, st, pdl, p, w_map, x_map, x2_map) :

@@ -10,7 +10,7 @@ namespace tmb {
 namespace {
 
 constexpr int kRouteWarps  = 8;
-constexpr int kSmallTokens = 64;  // up to here every CTA routes all tokens itself: one launch instead of two
+constexpr int kSmallTokens = 8;   // up to here every CTA routes all tokens itself: one launch instead of two
 
 struct DispatchParams {
     MoeRouter    r;
