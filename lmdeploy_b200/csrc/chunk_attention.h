@@ -11,6 +11,10 @@ __host__ __device__ __forceinline__ int chunk_first(int i, int chunk)
     return chunk > 0 ? i - i % chunk : 0;
 }
 
+// The 16-bit kernels hold a weight in fp16 times this, so that weights down to 2^-26 keep all their digits; outputs are
+// divided by it at the end.
+constexpr float kWeightScale = 4096.f;
+
 struct ChunkKernelParams {
     ChunkAttention a;
     MixerCall      c;

@@ -50,11 +50,11 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ float sigmoid_log2(float x)  // sigmoid of x / log2(e)
+__device__ __forceinline__ float scaled_sigmoid_log2(float x)  // sigmoid of x / log2(e), times kWeightScale
 {
     float e;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-x));
-    return __fdividef(1.f, 1.f + e);
+    return __fdividef(kWeightScale, 1.f + e);
 }
 __device__ __forceinline__ float load_cluster(uint32_t addr, uint32_t rank)  // shared memory of another CTA of the cluster
 {
@@ -189,8 +189,8 @@ __global__ void __launch_bounds__(MAXT) chunk_step_kernel(const StepParams p)
             for (int e = 0; e < 2; ++e) {
                 if (r + 8 * e >= heads) continue;
                 const int   idx = b * TK + kb * kKeys + 8 * t + c2;
-                const float x = idx < total ? sigmoid_log2(fmaf(s[t][2 * e], scale, bias[e])) : 0.f;
-                const float y = idx + 1 < total ? sigmoid_log2(fmaf(s[t][2 * e + 1], scale, bias[e])) : 0.f;
+                const float x = idx < total ? scaled_sigmoid_log2(fmaf(s[t][2 * e], scale, bias[e])) : 0.f;
+                const float y = idx + 1 < total ? scaled_sigmoid_log2(fmaf(s[t][2 * e + 1], scale, bias[e])) : 0.f;
                 *reinterpret_cast<__half2*>(w + (h0 + r + 8 * e) * w_ld + kb * kKeys + 8 * t + c2) = __floats2half2_rn(x, y);
             }
         }
@@ -252,6 +252,7 @@ __global__ void __launch_bounds__(MAXT) chunk_step_kernel(const StepParams p)
         else {
             for (int k = 0; k < p.kw; ++k) y += all[((size_t)(k * p.items + it) * kHeads + in % kHeads) * D + x % a.vdim];
         }
+        y *= 1.f / kWeightScale;
         if (whole) {
             out[x] = from_f32<E>(y);
         }

@@ -9,8 +9,8 @@
 //   chunk_mix_kernel      warp = 64 pairs of a query at a time: [heads x heads] times [heads x pairs] by mma.m16n8k16 with
 //                         fragments straight from and to memory, in place; the mixed weights are bf16
 //   chunk_values_kernel   CTA = (head, tile): O = P V (tcgen05)
-// fp16 holds a weight (at most 1) to 2^-12, finer than the bf16 operand of the last product, and the mixing matrix, whose
-// elements are bf16 weights, exactly unless they are tiny.  Every barrier wait is bounded.
+// fp16 holds a weight (times a power of two, kWeightScale) to 2^-12, finer than the bf16 operand of the last product, and the
+// mixing matrix, whose elements are bf16 weights, exactly unless they are tiny.  Every barrier wait is bounded.
 #include "chunk_attention.h"
 #include "tcgen05.cuh"
 #include "tm_b200.h"
@@ -63,11 +63,11 @@ __device__ __forceinline__ void cp_async16z(uint32_t dst, const void* src, int b
 {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
 }
-__device__ __forceinline__ float sigmoid_log2(float x)  // sigmoid of x / log2(e)
+__device__ __forceinline__ float scaled_sigmoid_log2(float x)  // sigmoid of x / log2(e), times kWeightScale
 {
     float e, y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-x));
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + e));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(fmaf(e, 1.f / kWeightScale, 1.f / kWeightScale)));
     return y;
 }
 // rows [0, count) of [row][width] at src into a swizzled tile of ROWS rows and D columns, zeros elsewhere
@@ -166,7 +166,8 @@ __global__ void __launch_bounds__(kThreads, 2) chunk_scores_kernel(const ChunkTc
             const int key0 = ti.base + t * kBN;
             uint32_t  w[32];
             auto pair = [&](uint32_t x, uint32_t y) {
-                const __half2 v = __floats2half2_rn(sigmoid_log2(fmaf(__uint_as_float(x), scale, bias)), sigmoid_log2(fmaf(__uint_as_float(y), scale, bias)));
+                const __half2 v = __floats2half2_rn(scaled_sigmoid_log2(fmaf(__uint_as_float(x), scale, bias)),
+                                                    scaled_sigmoid_log2(fmaf(__uint_as_float(y), scale, bias)));
                 return *reinterpret_cast<const uint32_t*>(&v);
             };
 #pragma unroll
@@ -230,7 +231,7 @@ __device__ __forceinline__ void mma_f16(float (&d)[4], const uint32_t (&a)[4], u
 // 8 n + t of the warp's 64, so that a lane's operand halves of all products are 8 consecutive pairs of one head, and a
 // lane's results 16 consecutive pairs.
 template<int HB>
-__global__ void __launch_bounds__(256) chunk_mix_kernel(const ChunkTcParams p)
+__global__ void __launch_bounds__(256, HB <= 2 ? 2 : 1) chunk_mix_kernel(const ChunkTcParams p)
 {
     pdl_wait();
     pdl_launch_dependents();
@@ -373,7 +374,9 @@ __global__ void __launch_bounds__(kThreads, 2) chunk_values_kernel(const ChunkTc
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 if (!live || 32 * c + 8 * i >= a.vdim) continue;
-                auto two = [&](int j) { return pack_bf16(__uint_as_float(o[8 * i + j]), __uint_as_float(o[8 * i + j + 1])); };
+                auto two = [&](int j) {
+                    return pack_bf16(__uint_as_float(o[8 * i + j]) * (1.f / kWeightScale), __uint_as_float(o[8 * i + j + 1]) * (1.f / kWeightScale));
+                };
                 *reinterpret_cast<uint4*>(out + h * a.vdim + 32 * c + 8 * i) = make_uint4(two(0), two(2), two(4), two(6));
             }
         }

@@ -117,6 +117,16 @@ def test_chunk_attention_whole_portions_and_decoding(dtype, shape):
 
 
 @both
+@pytest.mark.parametrize("bias", [-15.0, 6.0])
+def test_weights_that_are_tiny_or_all_but_one(dtype, bias):
+    a = Attention(dtype, 8, 2, 64, 64, scale=0.1, size=90, bias=bias)
+    x = random_inputs(a, 150)
+    want = a.oracle(*x)
+    for sizes in ((150,), (40, 1, 1)):
+        assert worst(run_in(a, x, sizes), want) <= TOL[dtype], sizes
+
+
+@both
 @pytest.mark.parametrize("dims", [(16, 16), (64, 64), (128, 128), (20, 12)])
 @pytest.mark.parametrize("size", [1, 32, 100, 130, 0])
 def test_one_key_stands_out_on_either_side_of_every_edge(dtype, dims, size):
